@@ -114,6 +114,9 @@ class GatedAttentionMixer(Mixer):
     pair m by j * rot_base^(-2m/vdim)) before it is cached, and a head's output at position i is turned back by i.
     ``weights`` "sigmoid": the weight of a visible key is sigmoid(score * scale + b_head) with a learned number per head
     (``score_bias``), not normalised over the keys.
+    ``value_norm``: every value head is divided by its root mean square over ``vdim`` (``eps`` inside the root) and cached so.
+    ``head_scales``: scores are multiplied by a learned number per query head as well as by ``scale``.
+    ``softcap`` > 0: scores, scaled, then become softcap * tanh(score / softcap).
 
     q, k, v and the head gates are one product; convolution, rotation, unit norm and the cache write are one kernel;
     angles, norms, scores and softmax are float32."""
@@ -128,7 +131,7 @@ class GatedAttentionMixer(Mixer):
                  rot_dims: int = 0, conv: int = 0, qk_norm: bool = False, eps: float = 1e-6, mask: str = "full", mask_size: int = 0,
                  sink: bool = False, conv_group: int = -1, conv_slot: int = -1, norm_weights: bool = False, temp_coef: float = 0.0,
                  temp_every: int = 1, gate: str = "head", norm_scope: str = "head", rot_pairs: str = "halves", rotate_values: bool = False,
-                 weights: str = "softmax"):
+                 weights: str = "softmax", value_norm: bool = False, head_scales: bool = False, softcap: float = 0.0):
         if heads % kv_heads:
             raise ValueError("Invalid GQA head ratio")
         if mask not in self.MASKS or (mask != "full" and mask_size <= 0):
@@ -160,7 +163,12 @@ class GatedAttentionMixer(Mixer):
             raise ValueError("values turn in pairs: vdim must be even")
         if weights == "sigmoid" and self.sink:
             raise ValueError("a sink belongs to a softmax")
-        self.score_bias = None
+        self.value_norm, self.has_head_scales, self.softcap = bool(value_norm), bool(head_scales), float(softcap)
+        if self.value_norm and self.wide_prepare:
+            raise ValueError("the value norm goes with neither a norm over the whole projection, nor neighbouring pairs, nor turned values")
+        if self.softcap < 0.0 or ((self.softcap > 0.0 or self.has_head_scales) and weights == "sigmoid"):
+            raise ValueError("softcap and head scales belong to a softmax; softcap is not negative")
+        self.score_bias = self.head_scales = None
         self._inv_freq_v = {}
         if self.temp_every < 1:
             raise ValueError("temp_every must be positive")
@@ -203,6 +211,8 @@ class GatedAttentionMixer(Mixer):
             shapes["k_norm.weight"] = ((self.kv_heads * self.dim if every else self.dim,), "vector")
         if self.weights == "sigmoid":
             shapes["score_bias"] = ((self.heads,), "vector")
+        if self.has_head_scales:
+            shapes["head_scales"] = ((self.heads,), "vector")
         return shapes
 
     def bind(self, tensors: dict) -> None:
@@ -251,6 +261,8 @@ class GatedAttentionMixer(Mixer):
             more.update(q_weight=self.q_norm_weight, k_weight=self.k_norm_weight)
         if self.temp_coef != 0.0:
             more.update(temp=(self.temp_coef, self.temp_every))
+        if self.value_norm:
+            more.update(value_norm=True)
         turned = self.value_inverse_frequencies(projected.device) if self.rotate_values else None
         if self.wide_prepare:
             queries = ops.qkv_norm_rope_cache(
@@ -268,8 +280,9 @@ class GatedAttentionMixer(Mixer):
             mixed = ops.paged_attention(queries, k_cache, v_cache, group.block_table, ctx, self.heads, self.kv_heads, self.head,
                                         group.page_size, self.scale, visibility, weights="sigmoid", head_bias=self.score_bias)
         else:
+            scores = {"softcap": self.softcap, "head_scales": self.head_scales} if self.softcap > 0.0 or self.has_head_scales else {}
             mixed = ops.paged_attention(queries, k_cache, v_cache, group.block_table, ctx, self.heads, self.kv_heads, self.head,
-                                        group.page_size, self.scale, visibility, sink=self.sink)
+                                        group.page_size, self.scale, visibility, sink=self.sink, **scores)
         head = self.head
         if self.rotate_values:
             # every head's sum turned back by the query's position; the padding of the kernels' head size goes on the way

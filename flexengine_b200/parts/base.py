@@ -46,6 +46,7 @@ Head:            ``forward(ctx, h) -> logits``: float32 [rows, vocab] from the f
 Junction:        ``forward(ctx, residual, pending, origin) -> residual``: rewrites the residual stream between two
                  layers (what the block before left ``pending`` is settled first); ``origin`` is the embedding's
                  output of this step, untouched.  A run entry names the junction that runs before its layer.
+                 It may return (residual, pending) instead, with something still to be put into the stream.
 """
 from __future__ import annotations
 

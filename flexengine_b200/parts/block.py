@@ -217,7 +217,8 @@ class HyperGatedBlock:
 
 class SandwichBlock:
     """Norms on both sides of every sublayer:
-        x <- x + norm1b(mixer(norm1(x)));  x <- x + norm2b(feed_forward(norm2(x)))   (the second where the layer has one).
+        x <- x + m norm1b(mixer(norm1(x)));  x <- x + m norm2b(feed_forward(norm2(x)))   (the second where the layer has one),
+    with a constant m = ``residual_scale`` (``block_params``; 1 unless given, and only for norms whose ``after`` takes a scale).
     A sublayer's output is not normed and added at once: it is handed on as ``pending`` (``PostNormed``), and the kernel
     of the norm that reads the stream next norms it, adds it and norms the sum (the next sublayer's, the next layer's,
     a junction's, or the model's final norm)."""
@@ -227,6 +228,7 @@ class SandwichBlock:
         self.norm1b = build_part("norm", layer_spec.norm)
         self.mixer = build_part("mixer", layer_spec.mixer)
         self.feed_forward = build_part("feed_forward", layer_spec.feed_forward) if layer_spec.feed_forward is not None else None
+        self.residual_scale = float(dict(layer_spec.block_params).get("residual_scale", 1.0))
         self.part_names = ("norm1", "mixer", "norm1b")
         if self.feed_forward is not None:
             self.norm2 = build_part("norm", layer_spec.norm)
@@ -236,10 +238,10 @@ class SandwichBlock:
     def parts(self) -> dict:
         return {name: getattr(self, name) for name in self.part_names}
 
-    @staticmethod
-    def _post(norm, out):
+    def _post(self, norm, out):
         """A sublayer may return (rows, bias still to add): the norm's kernel adds it."""
-        return norm.after(*out) if isinstance(out, tuple) else norm.after(out)
+        more = {"scale": self.residual_scale} if self.residual_scale != 1.0 else {}
+        return norm.after(*out, **more) if isinstance(out, tuple) else norm.after(out, **more)
 
     def forward(self, ctx, residual, pending, entry):
         h = self.norm1.forward(ctx, residual, pending)

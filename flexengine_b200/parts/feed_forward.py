@@ -1,4 +1,4 @@
-"""Feed-forwards: the dense gated one, down( act(gate(h)) * up(h) ), act = silu (SwiGLU) or the tanh form of GELU; the dense
+"""Feed-forwards: the dense gated one, down( act(gate(h)) * up(h) ), act = silu (SwiGLU), the tanh form of GELU or relu; the dense
 one without a gate, down( act(up(h)) ), act = xIELU or the square of relu; and the routed one (a mixture of experts of either form).
 
 Formula: tests/unit/test_synthetic_qwen.py:30-36 of the reference (its product code
@@ -13,7 +13,7 @@ from .base import FeedForward, register_feed_forward
 class SwiGLU(FeedForward):
     takes_prenormed = True
 
-    ACTIVATIONS = ("silu", "gelu_tanh")
+    ACTIVATIONS = ("silu", "gelu_tanh", "relu")
 
     def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "silu", bias: bool = False):
         self.hidden_size = int(hidden_size)
@@ -63,9 +63,9 @@ class ActivatedMlp(FeedForward):
     """down( act(up(h)) ), one matrix up, one down, no gate.  ``activation``:
     "xielu": two-sided, with two learned numbers p, q (``act``): z > 0: softplus(p) z^2 + z/2;
              z <= 0: (1/2 + softplus(q)) (exp(z) - 1 - z) + z/2;
-    "relu2": the square of relu(z)."""
+    "relu2": the square of relu(z);  "gelu": the exact form, z/2 (1 + erf(z / sqrt(2)))."""
 
-    ACTIVATIONS = ("xielu", "relu2")
+    ACTIVATIONS = ("xielu", "relu2", "gelu")
     takes_prenormed = False
 
     def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "xielu"):
@@ -103,15 +103,16 @@ class RoutedExperts(FeedForward):
     rows (``ops.routed_experts``): no count ever comes back to the host, so the step can be a CUDA graph."""
 
     ROUTERS = ("softmax_all", "softmax_chosen")
-    ACTIVATIONS = ("silu", "clamped", "relu2")
+    ACTIVATIONS = ("silu", "clamped", "relu2", "gelu")
+    SINGLE = ("relu2", "gelu")            # experts (and a shared one) without a gate: one matrix up, one down
 
     def __init__(self, hidden_size: int, experts: int, top: int, expert_size: int, scale: float = 1.0, shared_size: int = 0,
                  router: str = "softmax_all", activation: str = "silu", limit: float = 0.0, identity: int = 0,
                  correction: bool = False, groups: int = 1, keep: int = 1):
         """``router`` "softmax_all": as above; "softmax_chosen": the ``top`` largest logits are chosen and the weights are
-        the softmax over the chosen logits only.  ``activation`` "silu": as above; "clamped": with g = min(gate h, limit)
-        and u = clamp(up h, -limit, limit) an expert is down( g * sigmoid(1.702 g) * (u + 1) ); "relu2": an expert has no
-        gate and is down( relu(up h)^2 ).
+        the softmax over the chosen logits only (the same as the softmax over all, divided by the sum of the chosen shares).  ``activation`` "silu": as above; "clamped": with g = min(gate h, limit)
+        and u = clamp(up h, -limit, limit) an expert is down( g * sigmoid(1.702 g) * (u + 1) ); "relu2", "gelu": an expert (and
+        the shared one) has no gate and is down( act(up h) ), act the square of relu or the exact GELU.
         ``identity``: the router has that many further outputs, after the experts', that stand for experts which return
         their input (times the weight); they have no tensors.  ``correction``: a learned number per router output is added
         to the scores for the choice only; the weights are the uncorrected scores.  ``groups``, ``keep``: the router's
@@ -130,22 +131,24 @@ class RoutedExperts(FeedForward):
             raise ValueError("the groups must share the router's outputs out equally, and 1 <= keep <= groups")
         if (self.correction or self.groups > 1) and router != "softmax_all":
             raise ValueError("a correction and groups go with the softmax over all router outputs")
-        if self.shared_size and activation == "relu2":
-            raise ValueError("the shared expert is a gated one")
+        self.single = activation in self.SINGLE
         self.router_weight = self.router_correction = self.experts_gate_up_weight = self.experts_up_weight = self.experts_down_weight = None
-        self.shared_gate_up_weight = self.shared_down_weight = None
+        self.shared_gate_up_weight = self.shared_up_weight = self.shared_down_weight = None
 
     def parameter_shapes(self) -> dict:
         h, e, f = self.hidden_size, self.experts, self.expert_size
         shapes = {"router.weight": ((e + self.identity, h), "float32"), "experts.down.weight": ((e * h, f), "matrix")}
-        if self.activation == "relu2":
+        if self.single:
             shapes["experts.up.weight"] = ((e * f, h), "matrix")
         else:
             shapes["experts.gate_up.weight"] = ((e * 2 * f, h), "matrix")
         if self.correction:
             shapes["router.correction"] = ((e + self.identity,), "vector")
         if self.shared_size:
-            shapes["shared.gate_up.weight"] = ((2 * self.shared_size, h), "matrix")
+            if self.single:
+                shapes["shared.up.weight"] = ((self.shared_size, h), "matrix")
+            else:
+                shapes["shared.gate_up.weight"] = ((2 * self.shared_size, h), "matrix")
             shapes["shared.down.weight"] = ((h, self.shared_size), "matrix")
         return shapes
 
@@ -157,13 +160,15 @@ class RoutedExperts(FeedForward):
         e, f, d = self.experts, self.expert_size, self.hidden_size
         logits = ops.linear(h, self.router_weight, None, out_float32=True)
         shared = None
-        if self.shared_size:
+        if self.shared_size and self.single:
+            shared = ops.linear(ops.linear_activated(h, self.shared_up_weight, self.activation), self.shared_down_weight)
+        elif self.shared_size:
             shared = ops.linear(ops.linear_swiglu(h, self.shared_gate_up_weight, self.shared_size), self.shared_down_weight)
         down = self.experts_down_weight.view(e, d, f)
-        if self.activation == "relu2" or self.identity or self.correction or self.groups > 1:
+        if self.single or self.identity or self.correction or self.groups > 1:
             chosen, weights = ops.route_top(logits, self.top, self.scale, over_chosen=self.router == "softmax_chosen",
                                             correction=self.router_correction, groups=(self.groups, self.keep))
-            first = self.experts_up_weight.view(e, f, d) if self.activation == "relu2" else self.experts_gate_up_weight.view(e, 2 * f, d)
+            first = self.experts_up_weight.view(e, f, d) if self.single else self.experts_gate_up_weight.view(e, 2 * f, d)
             return ops.routed_experts(h, chosen, weights, first, down, shared, activation=self.activation, limit=self.limit,
                                       identity=self.identity)
         gate_up = self.experts_gate_up_weight.view(e, 2 * f, d)

@@ -93,7 +93,8 @@ class DecoderModel:
         for at, entry in enumerate(run):
             block = self.blocks[entry.layer]
             if entry.before >= 0:
-                residual, pending = self.junctions[entry.before].forward(ctx, residual, pending, origin), None
+                joined = self.junctions[entry.before].forward(ctx, residual, pending, origin)
+                residual, pending = joined if isinstance(joined, tuple) else (joined, None)
             # a block that can make use of it is told which norm reads the residual after it
             after = self.blocks[run[at + 1].layer] if at + 1 < len(run) else None
             if after is not None and getattr(after, "takes_prenormed", False) and self._knows_next_norm(block):

@@ -14,13 +14,16 @@ from .base import Norm, register_norm
 
 class PostNormed:
     """A branch's output on its way into the residual stream through a norm of its own: the stream receives
-    w * (y + bias) / sqrt(mean((y + bias)^2) + eps).  The kernel of the norm that reads the stream next does it (the
+    scale * w * (y + bias) / sqrt(mean((y + bias)^2) + eps), or, with ``norm_bias`` b (a layer norm), scale * (w * z + b) with
+    z = (y + bias - mean) / sqrt(variance + eps).  The kernel of the norm that reads the stream next does it (the
     ``pending`` of this framework: a branch output is not added at once).  ``y`` is float32 or in the compute dtype,
-    ``bias`` (float32, may be None) what the branch's last product has yet to add."""
-    __slots__ = ("y", "weight", "eps", "bias")
+    ``bias`` (float32, may be None) what the branch's last product has yet to add.  ``plus`` (float32 rows like the
+    stream's, may be None) is added to the stream as well; ``y`` may then be None."""
+    __slots__ = ("y", "weight", "eps", "bias", "norm_bias", "scale", "plus")
 
-    def __init__(self, y, weight, eps, bias=None):
+    def __init__(self, y, weight, eps, bias=None, norm_bias=None, scale=1.0, plus=None):
         self.y, self.weight, self.eps, self.bias = y, weight, float(eps), bias
+        self.norm_bias, self.scale, self.plus = norm_bias, float(scale), plus
 
 
 class RMSNorm(Norm):
@@ -45,6 +48,8 @@ class RMSNorm(Norm):
         if isinstance(delta, PostNormed):
             # the branch before ends in a norm of its own (a layer with norms on both sides of a sublayer): one kernel
             # norms the branch's output, adds it to the stream and norms the sum
+            if delta.norm_bias is not None or delta.scale != 1.0 or delta.plus is not None:
+                raise ValueError("this norm follows a plain RMS norm of a branch: no norm bias, no scale, nothing else to add")
             return ctx.ops.add_rmsnorm(residual, delta.y, self.weight, self.eps, ctx.dtype, rows,
                                        post=(delta.weight, delta.eps, delta.bias))
         return ctx.ops.add_rmsnorm(residual, delta, self.weight, self.eps, ctx.dtype, rows, upcoming=upcoming)
@@ -61,6 +66,31 @@ class RMSNorm(Norm):
                 and ctx.num_tokens <= ops.FUSED_NORM_MAX_ROWS and type(self).forward is RMSNorm.forward):
             return (residual, self.weight, self.eps)
         return None
+
+
+class LayerNorm(Norm):
+    """y = w * (x - mean) / sqrt(variance + eps) + b, the variance the mean of the squared deviations; all float32.  What is
+    pending goes into the stream in the same kernel: a branch that ends in a norm of this kind (``after``; times ``scale``),
+    a plain branch output, and rows that a junction adds."""
+
+    def __init__(self, hidden_size: int, eps: float):
+        self.hidden_size, self.eps = int(hidden_size), float(eps)
+        self.weight = self.bias = None
+
+    def parameter_shapes(self) -> dict:
+        return {"weight": ((self.hidden_size,), "vector"), "bias": ((self.hidden_size,), "vector")}
+
+    def forward(self, ctx, residual, delta, rows=None):
+        post = plus = None
+        if isinstance(delta, PostNormed):
+            if delta.y is not None and delta.norm_bias is None:
+                raise ValueError("a layer norm follows a branch that ends in a layer norm, or a plain branch")
+            post = (delta.weight, delta.norm_bias, delta.eps, delta.scale, delta.bias) if delta.y is not None else None
+            delta, plus = delta.y, delta.plus
+        return ctx.ops.add_layernorm(residual, delta, self.weight, self.bias, self.eps, ctx.dtype, rows, post=post, plus=plus)
+
+    def after(self, y, bias=None, scale=1.0) -> PostNormed:
+        return PostNormed(y, self.weight, self.eps, bias, norm_bias=self.bias, scale=scale)
 
 
 class GroupRMSNorm(Norm):
@@ -103,5 +133,6 @@ class StreamRMSNorm(Norm):
 
 
 register_norm("rmsnorm", RMSNorm)
+register_norm("layernorm", LayerNorm)
 register_norm("stream_rmsnorm", StreamRMSNorm)
 register_norm("group_rmsnorm", GroupRMSNorm)

@@ -51,6 +51,29 @@ def add_rmsnorm(residual, delta, weight, eps, out_dtype, rows=None, upcoming=Non
     return (x * torch.rsqrt(variance + eps) * weight.float()).to(out_dtype)
 
 
+def _layer_normed(x, weight, bias, eps):
+    centred = x - x.mean(dim=-1, keepdim=True)
+    return centred * torch.rsqrt(centred.pow(2).mean(dim=-1, keepdim=True) + eps) * weight.float() + bias.float()
+
+
+def add_layernorm(residual, delta, weight, bias, eps, out_dtype, rows=None, post=None, plus=None):
+    """residual += delta (through a layer norm of its own with ``post`` = (weight, bias, eps, scale, bias still to add)) +
+    ``plus``, then the layer norm of the sum; with ``rows`` only those rows are read and nothing is written."""
+    pick = (lambda t: t) if rows is None else (lambda t: t[rows.long()])
+    x = pick(residual)
+    if delta is not None:
+        y = pick(delta).float()
+        if post is not None:
+            p_weight, p_bias, p_eps, p_scale, y_bias = post
+            y = p_scale * _layer_normed(y if y_bias is None else y + y_bias.float(), p_weight, p_bias, p_eps)
+        x = x + y
+    if plus is not None:
+        x = x + pick(plus)
+    if rows is None:
+        residual.copy_(x)
+    return _layer_normed(x, weight, bias, eps).to(out_dtype)
+
+
 def residual_concat(residual, delta, extra, out_dtype, post=None):
     """residual += delta (through its own norm with ``post``), then [residual | extra] in ``out_dtype``."""
     if delta is not None:
@@ -89,6 +112,8 @@ def gated_activation(gate_up, intermediate, activation, bias=None, out_dtype=Non
         g, u = g + bias[:intermediate].float(), u + bias[intermediate:].float()
     if activation == "silu":
         a = g / (1.0 + torch.exp(-g))
+    elif activation == "relu":
+        a = torch.relu(g)
     elif activation == "gelu_tanh":
         a = 0.5 * g * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (g + 0.044715 * g * g * g)))
     else:
@@ -135,8 +160,9 @@ def qkv_projection(h, w, bias, positions, inv_freq, rot, slot_mapping, k_cache, 
 
 
 def paged_attention(qkv, k_cache, v_cache, block_table, ctx, nq, nkv, d, page_size, scale, window, upcoming=None, sink=False,
-                    weights="softmax", head_bias=None):
-    """``window`` > 0: the last ``window`` keys; < 0: the earlier keys of the query's chunk of -window positions.
+                    weights="softmax", head_bias=None, softcap=0.0, head_scales=None):
+    """``head_scales`` (one number per query head) multiplies the scores as ``scale`` does; ``softcap`` > 0: they then become
+    softcap * tanh(score / softcap).  ``window`` > 0: the last ``window`` keys; < 0: the earlier keys of the query's chunk of -window positions.
     ``sink``: 1 is added to the softmax's denominator.  ``weights`` "sigmoid": a visible key weighs
     sigmoid(score + head_bias[head]), not normalised over the keys."""
     T = qkv.shape[0]
@@ -165,6 +191,10 @@ def paged_attention(qkv, k_cache, v_cache, block_table, ctx, nq, nkv, d, page_si
         kh = k.repeat_interleave(ratio, dim=1)
         vh = v.repeat_interleave(ratio, dim=1)
         scores = torch.einsum("qhd,thd->hqt", q, kh) * scale
+        if head_scales is not None:
+            scores = scores * head_scales.float()[:, None, None]
+        if softcap > 0.0:
+            scores = softcap * torch.tanh(scores / softcap)
         scores = scores.masked_fill(~visible[None], float("-inf"))
         if weights == "sigmoid":
             w = torch.sigmoid(scores if head_bias is None else scores + head_bias.float()[:, None, None])
@@ -229,7 +259,7 @@ def token_shift(h, mu, kept, state_slots, cu_q, token_request):
 
 def qkv_conv_rope_norm_cache(projected, conv, history, taps, state_slots, cu_q, token_request, positions, inv_freq, rot_dims,
                              qk_norm, eps, slot_mapping, k_cache, v_cache, heads, kv_heads, dim, vdim, head, page_size,
-                             q_weight=None, k_weight=None, temp=None):
+                             q_weight=None, k_weight=None, temp=None, value_norm=False):
     """projected [T, >= channels] holds q | k | v.  A causal convolution of ``taps`` taps over time per channel (``conv``
     [taps, channels]; ``history`` [seats, (taps - 1) channels] holds every request's last taps - 1 projected rows and is
     brought up to date), rotation of the first ``rot_dims`` entries of the query and key heads, their unit norm, keys and
@@ -265,6 +295,8 @@ def qkv_conv_rope_norm_cache(projected, conv, history, taps, state_slots, cu_q, 
     if qk_norm:
         q = q * torch.rsqrt(q.pow(2).mean(dim=-1, keepdim=True) + eps)
         k = k * torch.rsqrt(k.pow(2).mean(dim=-1, keepdim=True) + eps)
+    if value_norm:
+        v = v * torch.rsqrt(v.pow(2).mean(dim=-1, keepdim=True) + eps)
     if q_weight is not None:
         q, k = q * q_weight.float(), k * k_weight.float()
     if temp is not None:
@@ -401,15 +433,105 @@ def retention_scan(qk, values, decay, state, state_slots, cu_q, heads, dim, vdim
     return out.view(T, heads * vdim)
 
 
+def activate_rows(projected, columns, activation, scales):
+    """float32 [T, columns]: silu of the first ``columns`` columns, runs of them times a factor each, the rest times 1."""
+    assert activation == "silu"
+    x = projected[:, :columns].float()
+    y = x / (1.0 + torch.exp(-x))
+    at = 0
+    for count, factor in scales:
+        y[:, at:at + count] *= factor
+        at += count
+    return y
+
+
 def retention_decode(projected, heads, dim, vdim, positions, inv_freq, rot_dims, key_scale, decay, state, state_slots, eps, out_dtype,
-                     scale=1.0, into=None):
-    """One token a request: rotation, recurrence, head norm and gate (the three references above, one after the other)."""
+                     scale=1.0, into=None, activation=None, raw=False):
+    """One token a request: rotation or activation, recurrence, then head norm and gate unless ``raw`` (the references above,
+    one after the other)."""
     R = projected.shape[0]
+    if raw:
+        cu = torch.arange(R + 1, dtype=torch.int32, device=projected.device)
+        if activation is not None:
+            rows = activate_rows(projected, 2 * heads * dim + heads * vdim, activation, ((heads * dim, 1.0), (heads * dim, key_scale)))
+            qk, values = rows[:, :2 * heads * dim], rows[:, 2 * heads * dim:]
+        else:
+            qk = rotate_heads(projected, 2 * heads, dim, positions, inv_freq, rot_dims, ((heads, 1.0), (heads, key_scale)))
+            values = projected[:, 2 * heads * dim:2 * heads * dim + heads * vdim]
+        return retention_scan(qk, values, decay, state, state_slots, cu, heads, dim, vdim)
     qk = rotate_heads(projected, 2 * heads, dim, positions, inv_freq, rot_dims, ((heads, 1.0), (heads, key_scale)))
     at = 2 * heads * dim
     cu = torch.arange(R + 1, dtype=torch.int32, device=projected.device)
     o = retention_scan(qk, projected[:, at:at + heads * vdim], decay, state, state_slots, cu, heads, dim, vdim)
     return head_rmsnorm_gate(o, None, projected[:, at + heads * vdim:at + 2 * heads * vdim], eps, heads, out_dtype, scale=scale, into=into)
+
+
+# ---- the gated delta rule ------------------------------------------------------------------------------
+def delta_prepare(projected, conv, state, history_at, state_slots, cu_q, token_request, a_log, dt_bias, unit_eps, query_scale,
+                  heads, kv_heads, dim, vdim):
+    """projected float32 [T, q | k | v | g | b | a].  Convolution (``conv`` [taps, channels]; the last taps - 1 rows of a request
+    in state[seat, history_at:], brought up to date) and silu of q | k | v, q and k unit vectors per head, q times
+    ``query_scale``: float32 [T, channels]; and float32 [T, 2 heads]: the decays, then the step sizes."""
+    T = projected.shape[0]
+    taps, C = conv.shape
+    u = projected[:, :C].float()
+    y = torch.zeros(T, C, dtype=torch.float32, device=projected.device)
+    cu, seats = cu_q.tolist(), state_slots.tolist()
+    back = taps - 1
+    for r in range(len(seats)):
+        a, b = cu[r], cu[r + 1]
+        past = torch.zeros(back, C, dtype=torch.float32, device=projected.device)
+        if seats[r] >= 0 and back:
+            past = state[seats[r], history_at:history_at + back * C].view(back, C).clone()
+        rows = torch.cat([past, u[a:b]])
+        for j in range(taps):
+            y[a:b] += conv[j] * rows[j:j + b - a]
+        if seats[r] >= 0 and back:
+            state[seats[r], history_at:history_at + back * C] = rows[rows.shape[0] - back:].reshape(-1)
+    y = y / (1.0 + torch.exp(-y))
+    n = kv_heads * dim
+    qk = y[:, :2 * n].view(T, 2 * kv_heads, dim)
+    qk = qk * torch.rsqrt(qk.pow(2).sum(dim=-1, keepdim=True) + unit_eps)
+    qk[:, :kv_heads] *= query_scale
+    out = torch.cat([qk.reshape(T, 2 * n), y[:, 2 * n:]], dim=-1)
+    at = C + heads * vdim
+    z = projected[:, at + heads:at + 2 * heads].float() + dt_bias.float()
+    decay = torch.exp(-torch.exp(a_log.float()) * torch.nn.functional.softplus(z))
+    return out, torch.cat([decay, torch.sigmoid(projected[:, at:at + heads].float())], dim=-1)
+
+
+def delta_scan(qkv, gates, state, state_slots, cu_q, heads, kv_heads, dim, vdim, max_q_len=0):
+    """S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, per request and head; S in state[seat, : heads dim vdim]."""
+    T, n = qkv.shape[0], kv_heads * dim
+    group = heads // kv_heads
+    q = qkv[:, :n].view(T, kv_heads, dim).repeat_interleave(group, dim=1)
+    k = qkv[:, n:2 * n].view(T, kv_heads, dim).repeat_interleave(group, dim=1)
+    v = qkv[:, 2 * n:].view(T, heads, vdim)
+    out = torch.zeros(T, heads, vdim, dtype=torch.float32, device=qkv.device)
+    cu, seats = cu_q.tolist(), state_slots.tolist()
+    m = heads * dim * vdim
+    for r in range(len(seats)):
+        S = state[seats[r], :m].view(heads, dim, vdim).clone() if seats[r] >= 0 else torch.zeros(heads, dim, vdim, device=qkv.device)
+        for t in range(cu[r], cu[r + 1]):
+            S = gates[t, :heads, None, None] * S
+            u = gates[t, heads:, None] * (v[t] - torch.einsum("hdv,hd->hv", S, k[t]))
+            S = S + k[t][:, :, None] * u[:, None, :]
+            out[t] = torch.einsum("hdv,hd->hv", S, q[t])
+        if seats[r] >= 0:
+            state[seats[r], :m] = S.reshape(-1)
+    return out.view(T, heads * vdim)
+
+
+def delta_decode(projected, conv, state, history_at, state_slots, a_log, dt_bias, norm_weight, eps, unit_eps, query_scale,
+                 heads, kv_heads, dim, vdim, out_dtype):
+    """One token a request: the two references above, then the head norm and the gate."""
+    R = projected.shape[0]
+    cu = torch.arange(R + 1, dtype=torch.int32, device=projected.device)
+    qkv, gates = delta_prepare(projected, conv, state, history_at, state_slots, cu, torch.arange(R), a_log, dt_bias, unit_eps, query_scale,
+                               heads, kv_heads, dim, vdim)
+    o = delta_scan(qkv, gates, state, state_slots, cu, heads, kv_heads, dim, vdim)
+    C = conv.shape[1]
+    return head_rmsnorm_gate(o, norm_weight.repeat(heads), projected[:, C:C + heads * vdim], eps, heads, out_dtype)
 
 
 def mingru_scan(zxg, bias, state, state_slots, cu_q, width, out_dtype, max_q_len=0):
@@ -513,6 +635,8 @@ def activation(x, kind, params=None):
         y = torch.where(z > 0, ap * z * z + 0.5 * z, an * (torch.exp(torch.clamp(z, max=0.0)) - 1.0 - z) + 0.5 * z)
     elif kind == "relu2":
         y = torch.relu(z) ** 2
+    elif kind == "gelu":
+        y = 0.5 * z * (1.0 + torch.erf(z * math.sqrt(0.5)))
     else:
         raise ValueError(kind)
     return y.to(x.dtype)
@@ -541,14 +665,14 @@ def wkv_recurrence(r, k, v, decay_logits, w0, u, state, state_slots, cu_q, heads
     return out.view(T, heads * dim)
 
 
-def head_rmsnorm_gate(out, weight, g, eps, heads, out_dtype, scale=1.0, into=None):
+def head_rmsnorm_gate(out, weight, g, eps, heads, out_dtype, scale=1.0, into=None, gate="silu"):
     T, inner = out.shape
     x = out.float().view(T, heads, inner // heads)
     x = (x * torch.rsqrt(x.pow(2).mean(dim=-1, keepdim=True) + eps)).reshape(T, inner)
     if weight is not None:
         x = x * weight.float()
     gf = g.float()
-    rows = (x * (gf / (1.0 + torch.exp(-gf))) * scale).to(out_dtype)
+    rows = (x * (gf / (1.0 + torch.exp(-gf)) if gate == "silu" else torch.sigmoid(gf)) * scale).to(out_dtype)
     if into is None:
         return rows
     into.copy_(rows)
@@ -623,7 +747,7 @@ def route_top(logits, top, scale, over_chosen=False, correction=None, groups=(1,
 
 
 def routed_experts(h, chosen, weights, gate_up, down, shared=None, activation="silu", limit=0.0, identity=0):
-    """``activation`` "relu2": ``gate_up`` is [experts, F, H], an expert is down(relu(up h)^2).  ``identity``: choices from
+    """``activation`` "relu2" or "gelu": ``gate_up`` is [experts, F, H], an expert is down(act(up h)).  ``identity``: choices from
     ``experts`` on stand for experts that return their input."""
     T, D = h.shape
     f = down.shape[2]
@@ -638,8 +762,9 @@ def routed_experts(h, chosen, weights, gate_up, down, shared=None, activation="s
                     total[rows] += weights[rows, slot, None] * hf[rows]
                 continue
             gu = hf[rows] @ gate_up[e].float().T
-            if activation == "relu2":
-                act = (torch.relu(gu) ** 2).to(h.dtype).float()
+            if activation in ("relu2", "gelu"):
+                z = torch.relu(gu) ** 2 if activation == "relu2" else 0.5 * gu * (1.0 + torch.erf(gu * math.sqrt(0.5)))
+                act = z.to(h.dtype).float()
                 total[rows] += weights[rows, slot, None] * (act @ down[e].float().T)
                 continue
             g, u = gu[:, :f], gu[:, f:]
