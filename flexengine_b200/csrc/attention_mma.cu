@@ -7,8 +7,9 @@
 // head h reads key/value head h / (nq / nkv).  ``sink``: the softmax starts as if a key of score 0 and value 0 had been
 // seen (running maximum 0, running sum 1), which adds 1 to its denominator; of the blocks and warps that share a row's
 // keys, the first one does.  ``mode`` carries the sink in bit 0; bit 1 asks for sigmoid weights instead of a softmax: a
-// visible key weighs sigmoid(score + head_bias[head]), nothing is normalised over the keys, and the parts of a row that
-// blocks and warps share are plainly added.
+// visible key weighs sigmoid(score + per_head[head]), nothing is normalised over the keys, and the parts of a row that
+// blocks and warps share are plainly added.  Bit 2: scores are multiplied by per_head[head] (null: by 1) and, with softcap > 0,
+// become softcap * tanh(score / softcap), before the softmax.
 //
 // Both kernels walk the keys in tiles of 32 aligned to position 0.  A tile's keys and values are
 // gathered page by page with 16-byte asynchronous copies (cp.async) into a ring of shared-memory
@@ -120,15 +121,24 @@ __device__ __forceinline__ void copy_rows(bf16* ks, bf16* vs, const KvSource& sr
     }
 }
 
+// The factor that takes a raw score to log2(e) * 2 * score * scale / cap, from the scale and the cap in log2 units.
+__device__ __forceinline__ float score_map_unit(float scale_log2, float cap_log2) {
+    return 2.f * scale_log2 * 1.4426950408889634f / cap_log2;
+}
+
 // One warp, KEYS keys (32, or 16 when two warps share a tile): s = Q K^T, mask (only where ``masked``), online
 // softmax in float with the running maximum kept in log2 units, o += P V.  ``ks``/``vs`` point at the first row.
 // pos0/pos1 and lo0/lo1: last and first visible key of the queries in rows g and g + 8.
 // UPPER = false: rows 8..15 of the tile are padding and their softmax is skipped.
+// mapped: the scores of the two rows are taken through a map of their own first: times bias0 / bias1 (the scale in log2 units and
+// the head's number in one), or, with cap_log2 > 0, squashed: cap tanh(score / cap) in log2 units, bias0 / bias1 being
+// the factors of the exponential in tanh(z) = 1 - 2 / (1 + e^(2z)).
 template <int DMAX, bool UPPER, int KEYS = TK>
 __device__ __forceinline__ void compute_tile(const bf16* ks, const bf16* vs, const unsigned (*qfrag)[4],
                                              float (*o)[4], float* m, float* l, int first_key, int d,
                                              float scale_log2, int pos0, int pos1, int lo0, int lo1, bool masked,
-                                             bool sigmoid = false, float bias0 = 0.f, float bias1 = 0.f) {
+                                             bool sigmoid = false, float bias0 = 0.f, float bias1 = 0.f,
+                                             bool mapped = false, float cap_log2 = 0.f) {
     const int lane = threadIdx.x & 31, t = lane & 3;
     const int mat = lane >> 3, mrow = lane & 7;
     float s[KEYS / 8][4];
@@ -149,6 +159,17 @@ __device__ __forceinline__ void compute_tile(const bf16* ks, const bf16* vs, con
                 }
             }
         }
+    }
+    if (mapped) {                                     // before the mask: a masked score is -inf and stays so
+#pragma unroll
+        for (int j = 0; j < KEYS / 8; ++j) {
+#pragma unroll
+            for (int e = 0; e < (UPPER ? 4 : 2); ++e) {
+                const float z = s[j][e] * (e < 2 ? bias0 : bias1);
+                s[j][e] = cap_log2 > 0.f ? fmaf(-2.f * cap_log2, rcp(1.f + ex2(z)), cap_log2) : z;
+            }
+        }
+        scale_log2 = 1.f;
     }
     if (masked) {
 #pragma unroll
@@ -285,7 +306,7 @@ paged_decode_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __rest
                     const bf16* __restrict__ vc, const int* __restrict__ block_table, int bt_stride,
                     const int* __restrict__ cu_q, const int* __restrict__ q_start, int nq, int nkv, int d, int ps,
                     int num_pages, float scale_log2, int window, int mode, int* __restrict__ status,
-                    const float* __restrict__ head_bias) {
+                    const float* __restrict__ per_head, float cap_log2) {
     griddep_wait();
     griddep_launch_dependents();
     const bool sink = mode & 1, sigmoid = mode & 2;
@@ -343,10 +364,16 @@ paged_decode_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __rest
         // parts up unweighted and divide a block's part by 1
         m[0] = m[1] = 0.f;
         if (warp == 0 && t == 0) l[0] = l[1] = 1.f;
-        if (head_bias) {
-            if (g < G) bias0 = head_bias[kvh * G + g] * 1.4426950408889634f;
-            if (UPPER && g + 8 < G) bias1 = head_bias[kvh * G + g + 8] * 1.4426950408889634f;
+        if (per_head) {
+            if (g < G) bias0 = per_head[kvh * G + g] * 1.4426950408889634f;
+            if (UPPER && g + 8 < G) bias1 = per_head[kvh * G + g + 8] * 1.4426950408889634f;
         }
+    }
+    const bool mapped = mode & 4;
+    if (mapped) {
+        const float unit = cap_log2 > 0.f ? score_map_unit(scale_log2, cap_log2) : scale_log2;
+        bias0 = g < G ? unit * (per_head ? per_head[kvh * G + g] : 1.f) : 0.f;
+        bias1 = (UPPER && g + 8 < G) ? unit * (per_head ? per_head[kvh * G + g + 8] : 1.f) : 0.f;
     }
 
     for (int it = 0; it < n_tiles; ++it) {
@@ -366,7 +393,7 @@ paged_decode_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __rest
         const bf16* sp = smem + (it % STAGES) * 2 * TILE + warp * DECODE_KEYS * pitch<DMAX>();
         const int first = (t_begin + it) * TK + warp * DECODE_KEYS;
         compute_tile<DMAX, UPPER, DECODE_KEYS>(sp, sp + TILE, qfrag, o, m, l, first, d, scale_log2, pos, pos, lo, lo,
-                                               first + DECODE_KEYS - 1 > pos || first < lo, sigmoid, bias0, bias1);
+                                               first + DECODE_KEYS - 1 > pos || first < lo, sigmoid, bias0, bias1, mapped, cap_log2);
     }
     cp_async_wait<0>();
 #pragma unroll
@@ -565,7 +592,7 @@ paged_prefill_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __res
                      const bf16* __restrict__ kc, const bf16* __restrict__ vc, const int* __restrict__ block_table,
                      int bt_stride, const int* __restrict__ cu_q, const int* __restrict__ q_start, int nq, int nkv,
                      int d, int ps, int num_pages, float scale_log2, int window, int mode, int* __restrict__ status,
-                     const float* __restrict__ head_bias) {
+                     const float* __restrict__ per_head, float cap_log2) {
     griddep_wait();
     griddep_launch_dependents();
     const bool sink = mode & 1, sigmoid = mode & 2;
@@ -616,8 +643,14 @@ paged_prefill_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __res
         m[0] = m[1] = 0.f;
         if (t == 0) l[0] = l[1] = 1.f;              // the four threads of a row add their sums up later
     }
-    const float bias0 = (sigmoid && head_bias) ? head_bias[head0] * 1.4426950408889634f : 0.f;
-    const float bias1 = (sigmoid && head_bias) ? head_bias[head1] * 1.4426950408889634f : 0.f;
+    float bias0 = (sigmoid && per_head) ? per_head[head0] * 1.4426950408889634f : 0.f;
+    float bias1 = (sigmoid && per_head) ? per_head[head1] * 1.4426950408889634f : 0.f;
+    const bool mapped = mode & 4;
+    if (mapped) {
+        const float unit = cap_log2 > 0.f ? score_map_unit(scale_log2, cap_log2) : scale_log2;
+        bias0 = unit * (per_head ? per_head[head0] : 1.f);
+        bias1 = unit * (per_head ? per_head[head1] : 1.f);
+    }
 
     // this warp's rows: the first and last position any of them has, and the widest window edge
     const int w_first = m_block + warp * 16, w_last = min(rows - 1, w_first + 15);
@@ -641,7 +674,7 @@ paged_prefill_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __res
                 // rows differ in what they see only near the diagonal and the window edge
                 const bool masked = first + TK - 1 > w_pos_min || first < w_lo_max || !(v0 && v1);
                 compute_tile<DMAX, true>(st + sub * TK * pitch<DMAX>(), st + STAGE + sub * TK * pitch<DMAX>(), qfrag, o, m,
-                                         l, first, d, scale_log2, pos0, pos1, lo0, lo1, masked, sigmoid, bias0, bias1);
+                                         l, first, d, scale_log2, pos0, pos1, lo0, lo1, masked, sigmoid, bias0, bias1, mapped, cap_log2);
             }
         }
         // offsets of stage it + 2 go where those of stage ``it`` were: all copies of stage ``it``'s
@@ -713,7 +746,7 @@ extern "C" int fe_paged_decode_mma_upcoming(const void* q, long long q_stride, v
                                             const void* kc, const void* vc, const int* block_table, int bt_stride,
                                             const int* cu_q, const int* q_start, int requests, int nq, int nkv, int d, int ps,
                                             int num_pages, float scale, int window, int sink, int splits, const void* upcoming,
-                                            long long upcoming_bytes, int* status, const float* head_bias, cudaStream_t stream) {
+                                            long long upcoming_bytes, int* status, const float* per_head, float softcap, cudaStream_t stream) {
     if (check_common("paged_decode", nq, nkv, d, ps, num_pages, window, q_stride, out_stride)) return 1;
     FE_REQUIRE(nq / nkv <= 16, "paged_decode: %d query heads per key/value head; this kernel takes up to 16", nq / nkv);
     FE_REQUIRE(splits >= 1 && splits <= MAX_SPLITS_SHARED && requests >= 0,
@@ -729,7 +762,7 @@ extern "C" int fe_paged_decode_mma_upcoming(const void* q, long long q_stride, v
         if (allow_smem(paged_decode_kernel<DMAX, UPPER>, decode_smem<DMAX>(), "paged_decode")) return 1;          \
         fe::launch(paged_decode_kernel<DMAX, UPPER>, grid, DECODE_WARPS * 32, decode_smem<DMAX>(), stream,                               \
             (const bf16*)q, q_stride, (bf16*)out, out_stride, part_o, part_lse, (const bf16*)kc, (const bf16*)vc, \
-            block_table, bt_stride, cu_q, q_start, nq, nkv, d, ps, num_pages, scale_log2, window, sink, status, head_bias);  \
+            block_table, bt_stride, cu_q, q_start, nq, nkv, d, ps, num_pages, scale_log2, window, sink, status, per_head, softcap * LOG2E);  \
     } while (0)
     const bool upper = nq / nkv > 8;
     if (d <= 64) { if (upper) FE_DECODE(64, true); else FE_DECODE(64, false); }
@@ -804,7 +837,7 @@ extern "C" int fe_paged_decode_cluster(const void* q, long long q_stride, void* 
                                        const void* kc, const void* vc, const int* block_table, int bt_stride,
                                        const int* cu_q, const int* q_start, int requests, int nq, int nkv, int d, int ps,
                                        int num_pages, float scale, int window, int sink, int splits, int* status,
-                                       const float* head_bias, cudaStream_t stream) {
+                                       const float* per_head, float softcap, cudaStream_t stream) {
     if (check_common("paged_decode", nq, nkv, d, ps, num_pages, window, q_stride, out_stride)) return 1;
     FE_REQUIRE(nq / nkv <= 16, "paged_decode: %d query heads per key/value head; this kernel takes up to 16", nq / nkv);
     FE_REQUIRE(splits >= 1 && splits <= CLUSTER_MAX_SPLITS && requests >= 0,
@@ -843,7 +876,7 @@ extern "C" int fe_paged_decode_cluster(const void* q, long long q_stride, void* 
         cfg.dynamicSmemBytes = decode_smem<DMAX>(STAGES);                                                              \
         const cudaError_t err = cudaLaunchKernelEx(&cfg, kernel, (const bf16*)q, q_stride, (bf16*)out, out_stride,     \
             (float*)nullptr, (float*)nullptr, (const bf16*)kc, (const bf16*)vc, block_table, bt_stride, cu_q, q_start, \
-            nq, nkv, d, ps, num_pages, scale_log2, window, sink, status, head_bias);                                   \
+            nq, nkv, d, ps, num_pages, scale_log2, window, sink, status, per_head, softcap * LOG2E);                                   \
         FE_REQUIRE(err == cudaSuccess, "paged_decode (cluster of %d): %s", splits, cudaGetErrorString(err));           \
     } while (0)
     const bool upper = nq / nkv > 8;
@@ -861,14 +894,14 @@ extern "C" int fe_paged_decode_mma(const void* q, long long q_stride, void* out,
                                    int num_pages, float scale, int window, int splits, int* status,
                                    cudaStream_t stream) {
     return fe_paged_decode_mma_upcoming(q, q_stride, out, out_stride, scratch, kc, vc, block_table, bt_stride, cu_q, q_start,
-                                        requests, nq, nkv, d, ps, num_pages, scale, window, 0, splits, nullptr, 0, status, nullptr, stream);
+                                        requests, nq, nkv, d, ps, num_pages, scale, window, 0, splits, nullptr, 0, status, nullptr, 0.f, stream);
 }
 
 extern "C" int fe_paged_prefill_mma(const void* q, long long q_stride, void* out, long long out_stride,
                                     const void* kc, const void* vc, const int* block_table, int bt_stride,
                                     const int* cu_q, const int* q_start, int requests, int max_q_len, int nq, int nkv,
                                     int d, int ps, int num_pages, float scale, int window, int sink, int* status,
-                                    const float* head_bias, cudaStream_t stream) {
+                                    const float* per_head, float softcap, cudaStream_t stream) {
     if (check_common("paged_prefill", nq, nkv, d, ps, num_pages, window, q_stride, out_stride)) return 1;
     FE_REQUIRE(requests >= 0 && max_q_len >= 0, "paged_prefill: bad request count or length");
     if (requests == 0 || max_q_len == 0) return 0;
@@ -882,7 +915,7 @@ extern "C" int fe_paged_prefill_mma(const void* q, long long q_stride, void* out
         if (allow_smem(paged_prefill_kernel<DMAX>, prefill_smem<DMAX>(), "paged_prefill")) return 1;           \
         fe::launch(paged_prefill_kernel<DMAX>, grid, PREFILL_WARPS * 32, prefill_smem<DMAX>(), stream,                 \
             (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kc, (const bf16*)vc, block_table,  \
-            bt_stride, cu_q, q_start, nq, nkv, d, ps, num_pages, scale_log2, window, sink, status, head_bias); \
+            bt_stride, cu_q, q_start, nq, nkv, d, ps, num_pages, scale_log2, window, sink, status, per_head, softcap * LOG2E); \
     } while (0)
     if (d <= 64) FE_PREFILL(64);
     else if (d <= 128) FE_PREFILL(128);

@@ -7,7 +7,8 @@
 // (and t > p - window when window > 0; t in the chunk of -window positions that holds p when window < 0)
 // (paged.py:31-32).  ``sink``: the softmax starts as if a key of score 0 and value 0 had been seen, which adds
 // 1 to its denominator.  ``mode`` bit 1 (bit 0 is the sink): no softmax; the weight of a visible key is
-// sigmoid(score + head_bias[h]), not normalised over the keys.  Query head h reads key/value head
+// sigmoid(score + per_head[h]), not normalised over the keys.  Bit 2: scores are multiplied by per_head[h] (null: by 1) and, with
+// softcap > 0, become softcap * tanh(score / softcap).  Query head h reads key/value head
 // h / (nq / nkv) (paged.py:29-30).  Because the blocks are aligned to position 0 and taken in
 // order, the result for a query does not depend on how its request was cut into steps.
 //
@@ -26,7 +27,7 @@ __global__ void paged_attention_simt_kernel(const T* __restrict__ q, long long q
                                             int bt_stride, const int* __restrict__ cu_q,
                                             const int* __restrict__ q_start, const int* __restrict__ token_req,
                                             int T_tokens, int nq, int nkv, int d, int ps, int num_pages, float scale,
-                                            int window, int mode, const float* __restrict__ head_bias, int* __restrict__ status) {
+                                            int window, int mode, const float* __restrict__ per_head, float softcap, int* __restrict__ status) {
     griddep_wait();
     griddep_launch_dependents();
     extern __shared__ float q_smem[];
@@ -44,7 +45,9 @@ __global__ void paged_attention_simt_kernel(const T* __restrict__ q, long long q
     __syncwarp();
 
     const bool sink = mode & 1, sigmoid = mode & 2;
-    const float bias = (sigmoid && head_bias) ? head_bias[h] : 0.f;
+    const float bias = (sigmoid && per_head) ? per_head[h] : 0.f;
+    if ((mode & 4) && per_head) scale *= per_head[h];
+    const float cap = mode & 4 ? softcap : 0.f;
     float m = sink ? 0.f : -CUDART_INF_F, l = sink ? 1.f : 0.f;
     float acc[DPL];
 #pragma unroll
@@ -73,6 +76,7 @@ __global__ void paged_attention_simt_kernel(const T* __restrict__ q, long long q
                     for (int e = 0; e < 8; ++e) dot = fmaf(qs[j + e], kv[e], dot);
                 }
                 s = dot * scale;
+                if (cap > 0.f) s = cap * tanhf(s / cap);
             }
         }
         float p;
@@ -117,7 +121,7 @@ template <typename T>
 static int launch_simt(const void* q, long long q_stride, void* out, long long out_stride, const void* kc,
                        const void* vc, const int* block_table, int bt_stride, const int* cu_q, const int* q_start,
                        const int* token_req, int T_tokens, int nq, int nkv, int d, int ps, int num_pages,
-                       float scale, int window, int sink, const float* head_bias, int* status, cudaStream_t stream) {
+                       float scale, int window, int sink, const float* per_head, float softcap, int* status, cudaStream_t stream) {
     const int warps = 4;
     const long long total = (long long)T_tokens * nq;
     const int blocks = (int)((total + warps - 1) / warps);
@@ -125,7 +129,7 @@ static int launch_simt(const void* q, long long q_stride, void* out, long long o
 #define FE_LAUNCH_SIMT(DPL)                                                                                      \
     fe::launch(paged_attention_simt_kernel<T, DPL>, blocks, warps * 32, smem, stream,                                    \
         (const T*)q, q_stride, (T*)out, out_stride, (const T*)kc, (const T*)vc, block_table, bt_stride, cu_q,   \
-        q_start, token_req, T_tokens, nq, nkv, d, ps, num_pages, scale, window, sink, head_bias, status)
+        q_start, token_req, T_tokens, nq, nkv, d, ps, num_pages, scale, window, sink, per_head, softcap, status)
     if (d <= 32) FE_LAUNCH_SIMT(1);
     else if (d <= 64) FE_LAUNCH_SIMT(2);
     else if (d <= 128) FE_LAUNCH_SIMT(4);
@@ -140,7 +144,7 @@ extern "C" int fe_paged_attention_simt(const void* q, long long q_stride, void* 
                                        const void* kc, const void* vc, const int* block_table, int bt_stride,
                                        const int* cu_q, const int* q_start, const int* token_req, int T_tokens,
                                        int nq, int nkv, int d, int ps, int num_pages, float scale, int window,
-                                       int sink, int dtype, int* status, const float* head_bias, cudaStream_t stream) {
+                                       int sink, int dtype, int* status, const float* per_head, float softcap, cudaStream_t stream) {
     FE_REQUIRE(T_tokens >= 0 && nq > 0 && nkv > 0 && nq % nkv == 0, "paged_attention: bad head counts %d/%d", nq, nkv);
     FE_REQUIRE(d >= 16 && d <= 1024 && d % 16 == 0, "paged_attention: head size %d is not a multiple of 16 in [16, 1024]", d);
     FE_REQUIRE(ps > 0 && num_pages > 0, "paged_attention: bad page size or page count");
@@ -148,9 +152,9 @@ extern "C" int fe_paged_attention_simt(const void* q, long long q_stride, void* 
     if (T_tokens == 0) return 0;
     if (dtype == FE_F32)
         return launch_simt<float>(q, q_stride, out, out_stride, kc, vc, block_table, bt_stride, cu_q, q_start,
-                                  token_req, T_tokens, nq, nkv, d, ps, num_pages, scale, window, sink, head_bias, status, stream);
+                                  token_req, T_tokens, nq, nkv, d, ps, num_pages, scale, window, sink, per_head, softcap, status, stream);
     if (dtype == FE_BF16)
         return launch_simt<bf16>(q, q_stride, out, out_stride, kc, vc, block_table, bt_stride, cu_q, q_start,
-                                 token_req, T_tokens, nq, nkv, d, ps, num_pages, scale, window, sink, head_bias, status, stream);
+                                 token_req, T_tokens, nq, nkv, d, ps, num_pages, scale, window, sink, per_head, softcap, status, stream);
     FE_REQUIRE(false, "paged_attention: unknown dtype %d", dtype);
 }

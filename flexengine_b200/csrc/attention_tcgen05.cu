@@ -261,6 +261,23 @@ __device__ __forceinline__ void row_sigmoid(const unsigned* r, unsigned p_addr, 
     }
 }
 
+// Scores through a map before the softmax: s <- s * unit, or with cap_log2 > 0 s <- cap tanh(score / cap) in log2 units, ``unit``
+// then being the factor of the exponential in tanh(z) = 1 - 2 / (1 + e^(2z)).
+__device__ __forceinline__ void row_map(unsigned* r, float unit, float cap_log2) {
+    if (cap_log2 > 0.f) {
+        const float2 cap2 = make_float2(cap_log2, cap_log2), minus2 = make_float2(-2.f * cap_log2, -2.f * cap_log2);
+#pragma unroll
+        for (int i = 0; i < KEYS; i += 2) {
+            const float2 w = make_float2(rcp(1.f + ex2(__uint_as_float(r[i]) * unit)), rcp(1.f + ex2(__uint_as_float(r[i + 1]) * unit)));
+            const float2 t = __ffma2_rn(w, minus2, cap2);
+            r[i] = __float_as_uint(t.x), r[i + 1] = __float_as_uint(t.y);
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < KEYS; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * unit);
+    }
+}
+
 template <int D>
 __global__ void __launch_bounds__(THREADS, 1)
 paged_prefill_tcgen05_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __restrict__ out, long long out_stride,
@@ -268,8 +285,9 @@ paged_prefill_tcgen05_kernel(const bf16* __restrict__ q, long long q_stride, bf1
                              const int* __restrict__ block_table, int bt_stride, const int* __restrict__ cu_q,
                              const int* __restrict__ q_start, int nq, int nkv, int ps, int num_pages, float scale_log2,
                              int window, int mode, int splits, float* __restrict__ part_o, float* __restrict__ part_lse,
-                             int* __restrict__ status, const float* __restrict__ head_bias) {
-    const bool sink = mode & 1, sigmoid = mode & 2;         // bit 1: sigmoid(score + head_bias[head]) instead of a softmax
+                             int* __restrict__ status, const float* __restrict__ per_head, float cap_log2) {
+    const bool sink = mode & 1, sigmoid = mode & 2;         // bit 1: sigmoid(score + per_head[head]) instead of a softmax
+    const bool mapped = mode & 4;       // scores times per_head[head] (null: 1) and, with a cap, cap tanh(score / cap), before the softmax
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     __shared__ __align__(8) unsigned long long kv_full[KV_STAGES], kv_empty[KV_STAGES], s_ready[2][2], p_ready[2][2], pv_done[2], o_final[2];
     __shared__ long long offs[2][KEYS];
@@ -463,7 +481,10 @@ paged_prefill_tcgen05_kernel(const bf16* __restrict__ q, long long q_stride, bf1
         if (sink && split == 0) { m_ref = 0.f; row_sum = 1.f; }
         // sigmoid weights: nothing is normalised; every split's share of a row stands with sum 1 and the merge adds them
         if (sigmoid) { m_ref = 0.f; row_sum = 1.f; }
-        const float bias = (sigmoid && head_bias && valid) ? head_bias[head] * 1.4426950408889634f : 0.f;
+        const float bias = (sigmoid && per_head && valid) ? per_head[head] * 1.4426950408889634f : 0.f;
+        const float unit = (cap_log2 > 0.f ? 2.f * scale_log2 * 1.4426950408889634f / cap_log2 : scale_log2) *
+                           (mapped && per_head && valid ? per_head[head] : 1.f);
+        const float to_log2 = mapped ? 1.f : scale_log2;          // what is left to multiply the (mapped) scores by
         bool ok = true;
         for (int j = 0; j < n_tiles; ++j) {
             ok = __all_sync(FULL, mbar_wait(&s_ready[ti][j & 1], (j >> 1) & 1, &give_up));
@@ -487,8 +508,9 @@ paged_prefill_tcgen05_kernel(const bf16* __restrict__ q, long long q_stride, bf1
                 mbar_arrive(&p_ready[ti][j & 1]);
                 continue;
             }
+            if (mapped) row_map(raw, unit, cap_log2);
             const float mx = unmasked ? row_max<false>(raw, rel_hi, rel_lo) : row_max<true>(raw, rel_hi, rel_lo);
-            const float m_new = fmaxf(m_ref, mx * scale_log2);
+            const float m_new = fmaxf(m_ref, mx * to_log2);
             if (__any_sync(FULL, m_new > m_ref + RESCALE_STEP)) {
                 // move the reference point to the new maximum: O and the sum were taken against the old one
                 const float alpha = m_new == -CUDART_INF_F ? 1.f : ex2(m_ref - m_new);
@@ -509,8 +531,8 @@ paged_prefill_tcgen05_kernel(const bf16* __restrict__ q, long long q_stride, bf1
                 m_ref = m_new;
             }
             const float m_safe = m_ref == -CUDART_INF_F ? 0.f : m_ref;
-            row_sum += unmasked ? row_exp<false>(raw, s_addr, rel_hi, rel_lo, scale_log2, m_safe)
-                                : row_exp<true>(raw, s_addr, rel_hi, rel_lo, scale_log2, m_safe);
+            row_sum += unmasked ? row_exp<false>(raw, s_addr, rel_hi, rel_lo, to_log2, m_safe)
+                                : row_exp<true>(raw, s_addr, rel_hi, rel_lo, to_log2, m_safe);
             tmem_store_wait();
             tc_fence_before();
             mbar_arrive(&p_ready[ti][j & 1]);
@@ -618,7 +640,7 @@ template <int D>
 int launch(const void* q, long long q_stride, void* out, long long out_stride, const void* kc, const void* vc,
            const int* block_table, int bt_stride, const int* cu_q, const int* q_start, int requests, int max_q_len, int nq,
            int nkv, int ps, int num_pages, float scale, int window, int sink, int splits, float* scratch, long long total_tokens,
-           int* status, const float* head_bias, cudaStream_t stream) {
+           int* status, const float* per_head, float softcap, cudaStream_t stream) {
     const size_t smem = (size_t)(D / 64) * (2 * Q_BLOCK + 2 * KV_STAGES * KV_BLOCK) + 1024;
     const cudaError_t err = cudaFuncSetAttribute(paged_prefill_tcgen05_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     FE_REQUIRE(err == cudaSuccess, "paged_prefill_tcgen05: %s", cudaGetErrorString(err));
@@ -630,7 +652,7 @@ int launch(const void* q, long long q_stride, void* out, long long out_stride, c
     float* part_lse = splits > 1 ? scratch + (size_t)total_tokens * nq * splits * D : nullptr;
     fe::launch(paged_prefill_tcgen05_kernel<D>, dim3((unsigned)tiles, nkv, requests), THREADS, smem, stream, (const bf16*)q, q_stride,
                (bf16*)out, out_stride, (const bf16*)kc, (const bf16*)vc, block_table, bt_stride, cu_q, q_start, nq, nkv, ps,
-               num_pages, scale * LOG2E, window, sink, splits, part_o, part_lse, status, head_bias);
+               num_pages, scale * LOG2E, window, sink, splits, part_o, part_lse, status, per_head, softcap * LOG2E);
     if (fe_check_launch("paged_prefill_tcgen05")) return 1;
     if (splits > 1) {
         const long long items = total_tokens * nq;
@@ -656,7 +678,7 @@ extern "C" int fe_paged_prefill_tcgen05(const void* q, long long q_stride, void*
                                         const void* vc, const int* block_table, int bt_stride, const int* cu_q,
                                         const int* q_start, int requests, int max_q_len, int nq, int nkv, int d, int ps,
                                         int num_pages, float scale, int window, int sink, int splits, void* scratch,
-                                        long long total_tokens, int* status, const float* head_bias, cudaStream_t stream) {
+                                        long long total_tokens, int* status, const float* per_head, float softcap, cudaStream_t stream) {
     FE_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "paged_prefill_tcgen05: bad head counts %d/%d", nq, nkv);
     FE_REQUIRE(d == 64 || d == 128, "paged_prefill_tcgen05: head size %d; this kernel takes 64 and 128", d);
     FE_REQUIRE(ps > 0 && num_pages > 0, "paged_prefill_tcgen05: bad page size or page count");
@@ -669,7 +691,7 @@ extern "C" int fe_paged_prefill_tcgen05(const void* q, long long q_stride, void*
     if (requests == 0 || max_q_len == 0) return 0;
     if (d == 64)
         return launch<64>(q, q_stride, out, out_stride, kc, vc, block_table, bt_stride, cu_q, q_start, requests, max_q_len, nq, nkv,
-                          ps, num_pages, scale, window, sink, splits, (float*)scratch, total_tokens, status, head_bias, stream);
+                          ps, num_pages, scale, window, sink, splits, (float*)scratch, total_tokens, status, per_head, softcap, stream);
     return launch<128>(q, q_stride, out, out_stride, kc, vc, block_table, bt_stride, cu_q, q_start, requests, max_q_len, nq, nkv, ps,
-                       num_pages, scale, window, sink, splits, (float*)scratch, total_tokens, status, head_bias, stream);
+                       num_pages, scale, window, sink, splits, (float*)scratch, total_tokens, status, per_head, softcap, stream);
 }

@@ -93,6 +93,9 @@ template <> __device__ __forceinline__ void store8<bf16>(bf16* p, const float* v
     *reinterpret_cast<uint4*>(p) = raw;
 }
 
+// The exact form of GELU: z/2 (1 + erf(z / sqrt(2))).
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
+
 // What a query at position ``pos`` sees of the keys t <= pos, as one int: 0 every key; w > 0 the last w keys (a sliding
 // window); -c < 0 the keys of its own chunk of c positions, counted from position 0.  The first visible key:
 __host__ __device__ __forceinline__ int first_visible(int pos, int window) {

@@ -438,8 +438,8 @@ extern "C" int fe_token_shift(const void* h, const float* mu, float* kept, long 
 //     tap, [taps, C], so that the lanes of a warp read neighbouring numbers;
 //   rotation (q, k): entries i and i + rot/2 of the head's first ``rot`` turn by position * inv_freq[i]; the token's sines
 //     and cosines are worked out once, by the whole block, for all of its heads;
-//   unit norm (q, k; qk_norm): the head divided by sqrt(mean of its squares + eps);
-//   q into ``q_out`` [T, heads * head], k and v into their cache slots [pages, kv_heads, ps, head], zeros beyond dim / vdim.
+//   unit norm (q, k; qk_norm; of v: v_norm): the head divided by sqrt(mean of its squares + eps);
+//   q into ``q_out`` [T, heads * head] (null: the queries need nothing and stay where they are), k and v into their cache slots [pages, kv_heads, ps, head], zeros beyond dim / vdim.
 // The history of a channel is read only by the first taps - 1 tokens of the request's portion.  The block of the portion's
 // first token therefore runs all of them, one after the other, and then brings the history up to date (the blocks of the
 // other early tokens do nothing), so that no block reads what another one writes.
@@ -516,7 +516,7 @@ __global__ void qkv_conv_rope_norm_cache_kernel(const T* __restrict__ proj, long
                                                 T* __restrict__ vc, T* __restrict__ q_out, int T_tokens, int heads, int kv_heads, int dim,
                                                 int vdim, int head, int ps, long long num_slots, int n_seats, int* __restrict__ status,
                                                 const float* __restrict__ q_weight, const float* __restrict__ k_weight, float temp_coef,
-                                                int temp_every) {
+                                                int temp_every, int v_norm) {
     griddep_wait();
     griddep_launch_dependents();
     extern __shared__ float staged[];
@@ -546,7 +546,7 @@ __global__ void qkv_conv_rope_norm_cache_kernel(const T* __restrict__ proj, long
             for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(pos * inv_freq[i], &sines[i], &cosines[i]);
         }
         __syncthreads();
-        for (int hs = warp; hs < per_token; hs += warps) {
+        for (int hs = warp + (q_out ? 0 : heads); hs < per_token; hs += warps) {
             // which head this is: 0 query, 1 key, 2 value; its first channel and its size
             const int what = hs < heads ? 0 : (hs < heads + kv_heads ? 1 : 2);
             const int index = what == 0 ? hs : (what == 1 ? hs - heads : hs - heads - kv_heads);
@@ -601,6 +601,11 @@ __global__ void qkv_conv_rope_norm_cache_kernel(const T* __restrict__ proj, long
                     ss = warp_sum(ss);
                     inv = rsqrtf(ss / (float)hd + eps);
                 }
+            } else if (v_norm) {
+                float ss = 0.f;
+                for (int c = lane; c < hd; c += 32) ss = fmaf(buf[c], buf[c], ss);
+                ss = warp_sum(ss);
+                inv = rsqrtf(ss / (float)hd + eps);
             }
             // after the norm: its weight (one table for the query heads, one for the key heads) and, for a query, the
             // temperature of its position, 1 + coef ln(floor((p + 1) / every) + 1)
@@ -651,8 +656,8 @@ static int launch_qkv_prepare(const void* proj, long long ld, const float* conv,
                               const int* seats, const int* cu_q, const int* token_req, const int* positions, const float* inv_freq, int rot,
                               int qk_norm, float eps, const int* slot_mapping, void* kc, void* vc, void* q_out, int T_tokens, int heads,
                               int kv_heads, int dim, int vdim, int head, int ps, long long num_slots, int n_seats, int* status,
-                              const float* q_weight, const float* k_weight, float temp_coef, int temp_every, cudaStream_t stream) {
-    const int per_token = heads + 2 * kv_heads;
+                              const float* q_weight, const float* k_weight, float temp_coef, int temp_every, int v_norm, cudaStream_t stream) {
+    const int per_token = (q_out ? heads : 0) + 2 * kv_heads;
     // up to 16 warps share out the token's heads evenly: 24 heads are two rounds of 12 warps
     const int rounds = (per_token + 15) / 16;
     int warps = (per_token + rounds - 1) / rounds;
@@ -669,7 +674,7 @@ static int launch_qkv_prepare(const void* proj, long long ld, const float* conv,
     fe::launch(qkv_conv_rope_norm_cache_kernel<T, PER>, T_tokens, warps * 32, smem, stream, (const T*)proj, ld, conv, history,     \
                history_stride, taps, seats, cu_q, token_req, positions, inv_freq, rot, qk_norm, eps, slot_mapping, (T*)kc, (T*)vc,  \
                (T*)q_out, T_tokens, heads, kv_heads, dim, vdim, head, ps, num_slots, n_seats, status, q_weight, k_weight, temp_coef,     \
-               temp_every)
+               temp_every, v_norm)
     if (per == 1) FE_LAUNCH_QKV_PREPARE(1);
     else if (per == 2) FE_LAUNCH_QKV_PREPARE(2);
     else if (per == 4) FE_LAUNCH_QKV_PREPARE(4);
@@ -684,7 +689,7 @@ extern "C" int fe_qkv_conv_rope_norm_cache(const void* proj, long long ld, const
                                            const float* inv_freq, int rot, int qk_norm, float eps, const int* slot_mapping, void* kc,
                                            void* vc, void* q_out, int T, int heads, int kv_heads, int dim, int vdim, int head, int ps,
                                            long long num_slots, int n_seats, int dtype, int* status, const float* q_weight,
-                                           const float* k_weight, float temp_coef, int temp_every, cudaStream_t stream) {
+                                           const float* k_weight, float temp_coef, int temp_every, int v_norm, cudaStream_t stream) {
     FE_REQUIRE((q_weight == nullptr) == (k_weight == nullptr) && (temp_coef == 0.f || temp_every > 0),
                "qkv_conv_rope_norm_cache: norm weights come in pairs, and a temperature needs a positive period");
     FE_REQUIRE(T >= 0 && heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && head >= dim && head >= vdim && head <= 1024,
@@ -698,11 +703,11 @@ extern "C" int fe_qkv_conv_rope_norm_cache(const void* proj, long long ld, const
     if (dtype == FE_F32)
         return launch_qkv_prepare<float>(proj, ld, conv, history, history_stride, taps, seats, cu_q, token_req, positions, inv_freq, rot,
                                          qk_norm, eps, slot_mapping, kc, vc, q_out, T, heads, kv_heads, dim, vdim, head, ps, num_slots,
-                                         n_seats, status, q_weight, k_weight, temp_coef, temp_every, stream);
+                                         n_seats, status, q_weight, k_weight, temp_coef, temp_every, v_norm, stream);
     if (dtype == FE_BF16)
         return launch_qkv_prepare<bf16>(proj, ld, conv, history, history_stride, taps, seats, cu_q, token_req, positions, inv_freq, rot,
                                         qk_norm, eps, slot_mapping, kc, vc, q_out, T, heads, kv_heads, dim, vdim, head, ps, num_slots,
-                                        n_seats, status, q_weight, k_weight, temp_coef, temp_every, stream);
+                                        n_seats, status, q_weight, k_weight, temp_coef, temp_every, v_norm, stream);
     FE_REQUIRE(false, "qkv_conv_rope_norm_cache: unknown dtype %d", dtype);
 }
 
@@ -1131,7 +1136,7 @@ extern "C" int fe_mingru_scan(const float* zxg, const float* bias, float* state,
 }
 
 // ---------------------------------------------------------------------------------------------
-// out = act(gate) * up with gate_up = [gate | up] per row; act 0: silu, 1: the tanh form of GELU,
+// out = act(gate) * up with gate_up = [gate | up] per row; act 0: silu, 2: relu, 1: the tanh form of GELU,
 //   gelu(z) = z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))).
 template <typename T>
 __global__ void gated_activation_kernel(const T* __restrict__ gate_up, T* __restrict__ out, long long total, int I, int act) {
@@ -1141,13 +1146,13 @@ __global__ void gated_activation_kernel(const T* __restrict__ gate_up, T* __rest
         const long long t = e / I;
         const int j = (int)(e - t * I);
         const float g = to_float(gate_up[t * 2 * I + j]), u = to_float(gate_up[t * 2 * I + I + j]);
-        const float a = act == 0 ? silu(g) : 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+        const float a = act == 0 ? silu(g) : act == 2 ? fmaxf(g, 0.f) : 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
         out[e] = from_float<T>(a * u);
     }
 }
 
 extern "C" int fe_gated_activation(const void* gate_up, void* out, int T, int I, int act, int dtype, cudaStream_t stream) {
-    FE_REQUIRE(T >= 0 && I > 0 && (act == 0 || act == 1), "gated_activation: bad sizes or activation %d", act);
+    FE_REQUIRE(T >= 0 && I > 0 && act >= 0 && act <= 2, "gated_activation: bad sizes or activation %d", act);
     const long long total = (long long)T * I;
     if (total == 0) return 0;
     const long long want = (total + 255) / 256;

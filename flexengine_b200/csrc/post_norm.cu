@@ -176,7 +176,7 @@ extern "C" int fe_scale_softcap(float* z, long long n, float scale, float cap, c
 
 // ---------------------------------------------------------------------------------------------
 // out[t, j] = act(gu[t, j] + bias[j]) * (gu[t, I + j] + bias[I + j]); gu float or the compute type, out the compute type.
-// act 0: silu; 1: the tanh form of GELU.
+// act 0: silu; 1: the tanh form of GELU; 2: relu.
 template <typename TI, typename T>
 __global__ void gated_activation_bias_kernel(const TI* __restrict__ gu, const float* __restrict__ bias, T* __restrict__ out, long long total,
                                              int I, int act) {
@@ -190,14 +190,14 @@ __global__ void gated_activation_bias_kernel(const TI* __restrict__ gu, const fl
             g += bias[j];
             u += bias[I + j];
         }
-        const float a = act == 0 ? g / (1.f + expf(-g)) : 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+        const float a = act == 0 ? g / (1.f + expf(-g)) : act == 2 ? fmaxf(g, 0.f) : 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
         out[e] = from_float<T>(a * u);
     }
 }
 
 extern "C" int fe_gated_activation_bias(const void* gu, int in_dtype, const float* bias, void* out, int T, int I, int act, int dtype,
                                         cudaStream_t stream) {
-    FE_REQUIRE(T >= 0 && I > 0 && (act == 0 || act == 1), "gated_activation_bias: bad sizes or activation");
+    FE_REQUIRE(T >= 0 && I > 0 && act >= 0 && act <= 2, "gated_activation_bias: bad sizes or activation");
     const long long total = (long long)T * I;
     if (total == 0) return 0;
     const long long want = (total + 255) / 256;

@@ -1,6 +1,7 @@
 // Retention: linear attention with one fixed decay per head, no softmax and no denominator.
 //   S_t = a_h S_(t-1) + k_t v_t^T ;   o_t = S_t^T q_t          S [d, dv] float per request and head
 // Kernels (all arithmetic float):
+//   activate_rows     float rows: silu of a projection's first columns, runs of columns times a factor each
 //   rotate_heads      float rows of heads from a projection: the first ``rot`` entries of a head turned by
 //                     position * inv_freq (pairs i, i + rot/2), runs of heads times a factor each
 //   retention_scan    the recurrence token by token over the step's portions, the state in registers
@@ -10,13 +11,36 @@
 //                     so three launches do a step: every block's own sum of k v^T (independent of the others), the chain
 //                     S_0 -> S_C -> ... over a portion's blocks (elementwise), and every block's outputs from the state
 //                     before it (independent again).  The products are tiled 64 x 64 over shared memory, 4 x 4 a thread.
-//   retention_decode  a step of one token a request: rotation, recurrence, the head's unit norm and the gate in one kernel
+//   retention_decode  a step of one token a request: rotation or activation, recurrence, the head's unit norm and the gate in one
+//                     kernel (or the heads' float sums as they are, for a norm over all heads)
 #define FE_PDL_CLASS 128
 #include "common.cuh"
 
 using namespace fe;
 
 namespace {
+
+__device__ __forceinline__ float silu(float z) { return z / (1.f + expf(-z)); }
+
+// out[t, c] = silu(proj[t, c]) * factor, the factor f0 for c < c0, f1 for c < c1, 1 beyond.  V columns a thread.
+template <typename T, int V>
+__global__ void activate_rows_kernel(const T* __restrict__ proj, long long ld, float* __restrict__ out, long long total, int columns, int c0,
+                                     float f0, int c1, float f1) {
+    griddep_wait();
+    griddep_launch_dependents();
+    const int per_row = columns / V;
+    for (long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (long long)gridDim.x * blockDim.x) {
+        const long long t = e / per_row;
+        const int c = (int)(e - t * per_row) * V;
+        float v[V];
+        if (V == 8) load8<T>(proj + t * ld + c, v);
+        else v[0] = to_float(proj[t * ld + c]);
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] = silu(v[i]) * (c + i < c0 ? f0 : (c + i < c1 ? f1 : 1.f));
+        if (V == 8) store8<float>(out + t * columns + c, v);
+        else out[t * columns + c] = v[0];
+    }
+}
 
 // ---------------------------------------------------------------------------------------------
 // One thread per (token, head, pair of turned entries or entry that passes).
@@ -56,7 +80,7 @@ constexpr int SCAN_TILE = 8;
 
 template <typename TV, int IPT>
 __global__ void __launch_bounds__(512)
-retention_scan_kernel(const float* __restrict__ qk, const TV* __restrict__ values, long long ldv, const float* __restrict__ decay,
+retention_scan_kernel(const float* __restrict__ qk, long long row, const TV* __restrict__ values, long long ldv, const float* __restrict__ decay,
                       float* state, long long state_stride, const int* __restrict__ seats, const int* __restrict__ cu_q,
                       float* __restrict__ out, int heads, int d, int dv, int n_seats) {
     griddep_wait();
@@ -87,7 +111,6 @@ retention_scan_kernel(const float* __restrict__ qk, const TV* __restrict__ value
     }
     for (int e = threadIdx.x; e < 2 * SCAN_TILE * ROW + SCAN_TILE * columns; e += blockDim.x) smem[e] = 0.f;
     const int begin = cu_q[req], end = cu_q[req + 1];
-    const long long row = 2LL * heads * d;
     __syncthreads();
     for (int t0 = begin; t0 < end; t0 += SCAN_TILE) {
         const int count = min(SCAN_TILE, end - t0);
@@ -148,7 +171,7 @@ retention_scan_kernel(const float* __restrict__ qk, const TV* __restrict__ value
 }
 
 template <typename TV, int IPT>
-int launch_scan(const float* qk, const void* values, long long ldv, const float* decay, float* state, long long state_stride,
+int launch_scan(const float* qk, long long ldqk, const void* values, long long ldv, const float* decay, float* state, long long state_stride,
                 const int* seats, const int* cu_q, float* out, int requests, int heads, int d, int dv, int n_seats, cudaStream_t stream) {
     // a head's value channels are cut into slices until the blocks about fill the device twice; a block keeps two warps at least
     const long long units = (long long)requests * heads;
@@ -160,15 +183,15 @@ int launch_scan(const float* qk, const void* values, long long ldv, const float*
     if (warps > 16) warps = 16;
     slices = (head_warps + warps - 1) / warps;
     const size_t smem = ((size_t)2 * SCAN_TILE * 8 * (IPT + 4) + (size_t)SCAN_TILE * warps * 4 + SCAN_TILE) * sizeof(float);
-    fe::launch(retention_scan_kernel<TV, IPT>, dim3(requests, heads, slices), warps * 32, smem, stream, qk, (const TV*)values, ldv, decay,
+    fe::launch(retention_scan_kernel<TV, IPT>, dim3(requests, heads, slices), warps * 32, smem, stream, qk, ldqk, (const TV*)values, ldv, decay,
                state, state_stride, seats, cu_q, out, heads, d, dv, n_seats);
     return fe_check_launch("retention_scan");
 }
 
 template <typename TV>
-int dispatch_scan(const float* qk, const void* values, long long ldv, const float* decay, float* state, long long state_stride,
+int dispatch_scan(const float* qk, long long ldqk, const void* values, long long ldv, const float* decay, float* state, long long state_stride,
                   const int* seats, const int* cu_q, float* out, int requests, int heads, int d, int dv, int n_seats, cudaStream_t stream) {
-#define FE_SCAN(IPT) return launch_scan<TV, IPT>(qk, values, ldv, decay, state, state_stride, seats, cu_q, out, requests, heads, d, dv, n_seats, stream)
+#define FE_SCAN(IPT) return launch_scan<TV, IPT>(qk, ldqk, values, ldv, decay, state, state_stride, seats, cu_q, out, requests, heads, d, dv, n_seats, stream)
     if (d <= 32) FE_SCAN(4);
     if (d <= 64) FE_SCAN(8);
     if (d <= 128) FE_SCAN(16);
@@ -191,7 +214,7 @@ __device__ __forceinline__ size_t chunk_row(const int* __restrict__ cu_q, int r)
 // head x tile of key channels x tile of value channels), 256 threads as 16 x 16, a thread 4 key x 4 value channels.
 template <typename TV>
 __global__ void __launch_bounds__(256)
-retention_chunk_sums_kernel(const float* __restrict__ qk, const TV* __restrict__ values, long long ldv, const float* __restrict__ decay,
+retention_chunk_sums_kernel(const float* __restrict__ qk, long long row, const TV* __restrict__ values, long long ldv, const float* __restrict__ decay,
                             const int* __restrict__ cu_q, float* __restrict__ sums, int heads, int d, int dv, int nd, int nv) {
     griddep_wait();
     griddep_launch_dependents();
@@ -209,12 +232,11 @@ retention_chunk_sums_kernel(const float* __restrict__ qk, const TV* __restrict__
     const int tid = threadIdx.x;
     if (tid < CHUNK) pw[tid] = tid < len ? (float)pow((double)decay[head], (double)(len - 1 - tid)) : 0.f;
     __syncthreads();
-    const size_t row = 2 * (size_t)heads * d;
     for (int e = tid; e < CHUNK * TILE; e += 256) {
         const int b = e / TILE, i = e - b * TILE;
         const int gi = dt * TILE + i, gj = vt * TILE + i;
         const bool in = b < len;
-        ks[e] = (in && gi < d) ? pw[b] * qk[(size_t)(begin + b) * row + (size_t)heads * d + (size_t)head * d + gi] : 0.f;
+        ks[e] = (in && gi < d) ? pw[b] * qk[(size_t)(begin + b) * (size_t)row + (size_t)heads * d + (size_t)head * d + gi] : 0.f;
         vs[e] = (in && gj < dv) ? to_float(values[(size_t)(begin + b) * ldv + (size_t)head * dv + gj]) : 0.f;
     }
     __syncthreads();
@@ -284,7 +306,7 @@ constexpr size_t CHUNK_OUT_SMEM = ((size_t)2 * TILE * PITCH + (size_t)TILE * TIL
 
 template <typename TV>
 __global__ void __launch_bounds__(256)
-retention_chunk_out_kernel(const float* __restrict__ qk, const TV* __restrict__ values, long long ldv, const float* __restrict__ decay,
+retention_chunk_out_kernel(const float* __restrict__ qk, long long row, const TV* __restrict__ values, long long ldv, const float* __restrict__ decay,
                            const int* __restrict__ cu_q, const float* __restrict__ sums, float* __restrict__ out, int heads, int d, int dv,
                            int nd, int nv) {
     griddep_wait();
@@ -306,7 +328,6 @@ retention_chunk_out_kernel(const float* __restrict__ qk, const TV* __restrict__ 
         const int b = e / TILE, j = e - b * TILE, gj = vt * TILE + j;
         vS[e] = (b < len && gj < dv) ? to_float(values[(size_t)(begin + b) * ldv + (size_t)head * dv + gj]) : 0.f;
     }
-    const size_t row = 2 * (size_t)heads * d;
     const float* before = sums + ((chunk_row(cu_q, r) + c) * heads + head) * (size_t)d * dv;
     float W[4][4] = {}, O[4][4] = {};
     for (int dt = 0; dt < nd; ++dt) {
@@ -376,7 +397,7 @@ retention_chunk_out_kernel(const float* __restrict__ qk, const TV* __restrict__ 
 }
 
 template <typename TV>
-int launch_chunks(const float* qk, const void* values, long long ldv, const float* decay, float* state, long long state_stride,
+int launch_chunks(const float* qk, long long ldqk, const void* values, long long ldv, const float* decay, float* state, long long state_stride,
                   const int* seats, const int* cu_q, float* out, float* sums, int requests, int most_blocks, int heads, int d, int dv,
                   int n_seats, cudaStream_t stream) {
     static bool opted = false;
@@ -388,11 +409,11 @@ int launch_chunks(const float* qk, const void* values, long long ldv, const floa
     }
     const int nd = (d + TILE - 1) / TILE, nv = (dv + TILE - 1) / TILE;
     const size_t per = (size_t)heads * d * dv;
-    fe::launch(retention_chunk_sums_kernel<TV>, dim3(most_blocks, requests, heads * nd * nv), 256, 0, stream, qk, (const TV*)values, ldv,
+    fe::launch(retention_chunk_sums_kernel<TV>, dim3(most_blocks, requests, heads * nd * nv), 256, 0, stream, qk, ldqk, (const TV*)values, ldv,
                decay, cu_q, sums, heads, d, dv, nd, nv);
     fe::launch(retention_chunk_chain_kernel, dim3(requests, (unsigned)((per + 255) / 256)), 256, 0, stream, decay, state, state_stride,
                seats, cu_q, sums, heads, d, dv, n_seats);
-    fe::launch(retention_chunk_out_kernel<TV>, dim3(most_blocks, requests, heads * nv), 256, CHUNK_OUT_SMEM, stream, qk, (const TV*)values,
+    fe::launch(retention_chunk_out_kernel<TV>, dim3(most_blocks, requests, heads * nv), 256, CHUNK_OUT_SMEM, stream, qk, ldqk, (const TV*)values,
                ldv, decay, cu_q, (const float*)sums, out, heads, d, dv, nd, nv);
     return fe_check_launch("retention_chunks");
 }
@@ -407,7 +428,7 @@ __global__ void __launch_bounds__(1024)
 retention_decode_kernel(const T* __restrict__ proj, long long ld, const int* __restrict__ positions, const float* __restrict__ inv_freq,
                         int rot, float key_scale, const float* __restrict__ decay, float* state, long long state_stride,
                         const int* __restrict__ seats, T* __restrict__ out, long long ldo, float eps, float scale, int heads, int d,
-                        int dv, int n_seats, int groups) {
+                        int dv, int n_seats, int groups, int activated, float* __restrict__ raw) {
     griddep_wait();
     griddep_launch_dependents();
     extern __shared__ __align__(16) float smem[];
@@ -424,6 +445,10 @@ retention_decode_kernel(const T* __restrict__ proj, long long ld, const int* __r
     const int half = rot >> 1;
     for (int i = tid; i < d; i += blockDim.x) {
         float q = to_float(qrow[i]), k = to_float(krow[i]);
+        if (activated) {
+            q = silu(q);
+            k = silu(k);
+        }
         if (i < rot) {
             const bool low = i < half;
             const int other = low ? i + half : i - half;
@@ -450,7 +475,8 @@ retention_decode_kernel(const T* __restrict__ proj, long long ld, const int* __r
     for (int j0 = 0; j0 < dv; j0 += columns) {
         const int j = j0 + jj;
         const bool own = g < groups && j < dv;
-        const float vj = own ? to_float(vrow[j]) : 0.f;
+        float vj = own ? to_float(vrow[j]) : 0.f;
+        if (activated) vj = silu(vj);
         float acc = 0.f;
         if (own && mine) {
             float* col = mine + j;
@@ -476,6 +502,10 @@ retention_decode_kernel(const T* __restrict__ proj, long long ld, const int* __r
             ss = fmaf(o, o, ss);
         }
         __syncthreads();
+    }
+    if (raw) {                                      // the norm reads all heads of the row: it comes afterwards
+        for (int j = tid; j < dv; j += blockDim.x) raw[((size_t)r * heads + head) * dv + j] = os[j];
+        return;
     }
     ss = block_sum(ss, red);
     const float inv = rsqrtf(ss / (float)dv + eps) * scale;
@@ -509,19 +539,40 @@ extern "C" int fe_rotate_heads(const void* proj, long long ld, const int* positi
     return fe_check_launch("rotate_heads");
 }
 
-// qk float [T, 2 heads d] (queries, then keys); values [T, >= heads dv] in ``dtype`` with rows ldv entries long; decay float
+// out float [T, columns]: silu of the first ``columns`` columns of proj (rows ld entries long); columns below c0 times f0, from there
+// below c1 times f1.
+extern "C" int fe_activate_rows(const void* proj, long long ld, float* out, int T, int columns, int c0, float f0, int c1, float f1, int dtype,
+                                cudaStream_t stream) {
+    FE_REQUIRE(T >= 0 && columns > 0 && ld >= columns && c0 >= 0 && c1 >= c0, "activate_rows: bad sizes");
+    FE_REQUIRE(dtype == FE_F32 || dtype == FE_BF16, "activate_rows: unknown dtype %d", dtype);
+    const bool vec = columns % 8 == 0 && ld % 8 == 0 && (((size_t)proj | (size_t)out) & 31) == 0;
+    const long long total = (long long)T * (vec ? columns / 8 : columns);
+    if (total == 0) return 0;
+    const long long want = (total + 255) / 256;
+    const unsigned blocks = (unsigned)(want < 65535LL * 8 ? want : 65535LL * 8);
+    if (dtype == FE_F32) {
+        if (vec) fe::launch(activate_rows_kernel<float, 8>, blocks, 256, 0, stream, (const float*)proj, ld, out, total, columns, c0, f0, c1, f1);
+        else fe::launch(activate_rows_kernel<float, 1>, blocks, 256, 0, stream, (const float*)proj, ld, out, total, columns, c0, f0, c1, f1);
+    } else {
+        if (vec) fe::launch(activate_rows_kernel<bf16, 8>, blocks, 256, 0, stream, (const bf16*)proj, ld, out, total, columns, c0, f0, c1, f1);
+        else fe::launch(activate_rows_kernel<bf16, 1>, blocks, 256, 0, stream, (const bf16*)proj, ld, out, total, columns, c0, f0, c1, f1);
+    }
+    return fe_check_launch("activate_rows");
+}
+
+// qk float [T, >= 2 heads d] (queries, then keys; rows ldqk entries long); values [T, >= heads dv] in ``dtype`` with rows ldv entries long; decay float
 // [heads]; state float [n_seats, >= heads d dv]; out float [T, heads dv].
-extern "C" int fe_retention_scan(const float* qk, const void* values, long long ldv, const float* decay, float* state,
+extern "C" int fe_retention_scan(const float* qk, long long ldqk, const void* values, long long ldv, const float* decay, float* state,
                                  long long state_stride, const int* seats, const int* cu_q, float* out, int requests, int heads, int d,
                                  int dv, int n_seats, int dtype, cudaStream_t stream) {
     FE_REQUIRE(requests >= 0 && heads > 0 && heads <= 65535 && d > 0 && d <= 256 && dv > 0 && n_seats >= 0 &&
-                   (long long)heads * d * dv <= state_stride && ldv >= (long long)heads * dv,
+                   (long long)heads * d * dv <= state_stride && ldv >= (long long)heads * dv && ldqk >= 2LL * heads * d,
                "retention_scan: bad sizes (heads %d, key size %d up to 256, value size %d)", heads, d, dv);
     FE_REQUIRE(dtype == FE_F32 || dtype == FE_BF16, "retention_scan: unknown dtype %d", dtype);
     if (requests == 0) return 0;
     if (dtype == FE_F32)
-        return dispatch_scan<float>(qk, values, ldv, decay, state, state_stride, seats, cu_q, out, requests, heads, d, dv, n_seats, stream);
-    return dispatch_scan<bf16>(qk, values, ldv, decay, state, state_stride, seats, cu_q, out, requests, heads, d, dv, n_seats, stream);
+        return dispatch_scan<float>(qk, ldqk, values, ldv, decay, state, state_stride, seats, cu_q, out, requests, heads, d, dv, n_seats, stream);
+    return dispatch_scan<bf16>(qk, ldqk, values, ldv, decay, state, state_stride, seats, cu_q, out, requests, heads, d, dv, n_seats, stream);
 }
 
 // The same as fe_retention_scan for steps with long portions, in blocks of 64 tokens (three launches).  ``sums`` is scratch:
@@ -529,34 +580,36 @@ extern "C" int fe_retention_scan(const float* qk, const void* values, long long 
 // portion of the step or more.
 extern "C" int fe_retention_chunk_tokens() { return CHUNK; }
 
-extern "C" int fe_retention_chunks(const float* qk, const void* values, long long ldv, const float* decay, float* state,
+extern "C" int fe_retention_chunks(const float* qk, long long ldqk, const void* values, long long ldv, const float* decay, float* state,
                                    long long state_stride, const int* seats, const int* cu_q, float* out, float* sums, int requests,
                                    int most_tokens, int heads, int d, int dv, int n_seats, int dtype, cudaStream_t stream) {
     FE_REQUIRE(requests >= 0 && requests <= 65535 && heads > 0 && d > 0 && dv > 0 && n_seats >= 0 && most_tokens >= 0 &&
-                   (long long)heads * d * dv <= state_stride && ldv >= (long long)heads * dv &&
+                   (long long)heads * d * dv <= state_stride && ldv >= (long long)heads * dv && ldqk >= 2LL * heads * d &&
                    (long long)heads * ((d + TILE - 1) / TILE) * ((dv + TILE - 1) / TILE) <= 65535,
                "retention_chunks: bad sizes (heads %d, key size %d, value size %d, %d requests)", heads, d, dv, requests);
     FE_REQUIRE(dtype == FE_F32 || dtype == FE_BF16, "retention_chunks: unknown dtype %d", dtype);
     if (requests == 0 || most_tokens == 0) return 0;
     const int most_blocks = (most_tokens + CHUNK - 1) / CHUNK;
     if (dtype == FE_F32)
-        return launch_chunks<float>(qk, values, ldv, decay, state, state_stride, seats, cu_q, out, sums, requests, most_blocks, heads, d, dv,
+        return launch_chunks<float>(qk, ldqk, values, ldv, decay, state, state_stride, seats, cu_q, out, sums, requests, most_blocks, heads, d, dv,
                                     n_seats, stream);
-    return launch_chunks<bf16>(qk, values, ldv, decay, state, state_stride, seats, cu_q, out, sums, requests, most_blocks, heads, d, dv,
+    return launch_chunks<bf16>(qk, ldqk, values, ldv, decay, state, state_stride, seats, cu_q, out, sums, requests, most_blocks, heads, d, dv,
                                n_seats, stream);
 }
 
 // A step of one token a request in one kernel.  proj [R, >= 2 heads d + 2 heads dv] = q | k | v | g in ``dtype`` with rows ld
 // entries long; the keys are multiplied by key_scale after the rotation; out [R, >= heads dv] in ``dtype`` with rows ldo long gets
-// every head divided by its root mean square, times silu(g), times scale.
+// every head divided by its root mean square, times silu(g), times scale.  activated: q, k and v go through silu first (then nothing
+// turns).  raw (may be null): float [R, heads dv] gets the heads' sums as they are instead; out and g are not touched.
 extern "C" int fe_retention_decode(const void* proj, long long ld, const int* positions, const float* inv_freq, int rot, float key_scale,
                                    const float* decay, float* state, long long state_stride, const int* seats, void* out, long long ldo,
-                                   float eps, float scale, int requests, int heads, int d, int dv, int n_seats, int dtype,
-                                   cudaStream_t stream) {
+                                   float eps, float scale, int requests, int heads, int d, int dv, int n_seats, int activated, float* raw,
+                                   int dtype, cudaStream_t stream) {
     FE_REQUIRE(requests >= 0 && heads > 0 && heads <= 65535 && d > 0 && dv > 0 && n_seats >= 0 && rot >= 0 && rot % 2 == 0 && rot <= d &&
                    (long long)heads * d * dv <= state_stride && ld >= 2LL * heads * d + 2LL * heads * dv && ldo >= (long long)heads * dv,
                "retention_decode: bad sizes (heads %d, key size %d, value size %d, %d turned)", heads, d, dv, rot);
     FE_REQUIRE(rot == 0 || inv_freq != nullptr, "retention_decode: a rotation needs its frequencies");
+    FE_REQUIRE(!activated || rot == 0, "retention_decode: activated queries and keys do not turn");
     FE_REQUIRE(dtype == FE_F32 || dtype == FE_BF16, "retention_decode: unknown dtype %d", dtype);
     if (requests == 0) return 0;
     int columns = ((dv < 256 ? dv : 256) + 31) / 32 * 32;
@@ -566,9 +619,11 @@ extern "C" int fe_retention_decode(const void* proj, long long ld, const int* po
     FE_REQUIRE(smem <= 48 * 1024, "retention_decode: key size %d and value size %d need more shared memory than a block has", d, dv);
     if (dtype == FE_F32)
         fe::launch(retention_decode_kernel<float>, dim3(requests, heads), groups * columns, smem, stream, (const float*)proj, ld, positions,
-                   inv_freq, rot, key_scale, decay, state, state_stride, seats, (float*)out, ldo, eps, scale, heads, d, dv, n_seats, groups);
+                   inv_freq, rot, key_scale, decay, state, state_stride, seats, (float*)out, ldo, eps, scale, heads, d, dv, n_seats, groups,
+                   activated, raw);
     else
         fe::launch(retention_decode_kernel<bf16>, dim3(requests, heads), groups * columns, smem, stream, (const bf16*)proj, ld, positions,
-                   inv_freq, rot, key_scale, decay, state, state_stride, seats, (bf16*)out, ldo, eps, scale, heads, d, dv, n_seats, groups);
+                   inv_freq, rot, key_scale, decay, state, state_stride, seats, (bf16*)out, ldo, eps, scale, heads, d, dv, n_seats, groups,
+                   activated, raw);
     return fe_check_launch("retention_decode");
 }

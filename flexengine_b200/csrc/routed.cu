@@ -29,8 +29,13 @@ __device__ __forceinline__ float expert_activation(float g, float u, float limit
     return g / (1.f + expf(-g)) * u;
 }
 
-// What an expert without a gate does with its one product.
-__device__ __forceinline__ float squared_relu(float z) { return z > 0.f ? z * z : 0.f; }
+// What an expert without a gate does with its one product: the square of relu, or the exact GELU.  (The products' kernels take
+// the choice in the place of the gated experts' limit.)
+constexpr float SINGLE_RELU2 = 0.f, SINGLE_GELU = 1.f;
+__device__ __forceinline__ float single_activation(float z, float which) {
+    if (which == SINGLE_GELU) return gelu_erf(z);
+    return z > 0.f ? z * z : 0.f;
+}
 
 // One warp per token.  ties go to the lower expert index.  ``over_chosen`` 0: the weights are the chosen experts' shares of
 // the softmax over all logits; 1: the ``top`` largest logits are chosen and the weights are the softmax over those alone.
@@ -188,7 +193,7 @@ __global__ void route_plan_kernel(const int* __restrict__ chosen, int pairs, int
 
 // The two grouped products.  Tile 64 rows x 64 columns, 16 of K a stage, 256 threads with 4 x 4 outputs each; float
 // accumulation in ascending k.  MODE 1 (GATED): columns n and n + F of the expert's matrix are taken together and
-// silu(gate) * up is written (compute type); MODE 2: an expert without a gate, relu(product)^2 is written (compute type);
+// silu(gate) * up is written (compute type); MODE 2: an expert without a gate, single_activation is written (compute type);
 // MODE 0: the plain product is written in float.
 namespace {
 constexpr int BM = 64, BN = 64, BK = 16, TM = 4, TN = 4;
@@ -268,7 +273,7 @@ routed_product_kernel(const T* __restrict__ A, const int* __restrict__ pair_of_r
                 const float g = acc[i][j];
                 reinterpret_cast<T*>(out)[at] = from_float<T>(expert_activation(g, acu[i][j], limit));
             } else if (MODE == 2) {
-                reinterpret_cast<T*>(out)[at] = from_float<T>(squared_relu(acc[i][j]));
+                reinterpret_cast<T*>(out)[at] = from_float<T>(single_activation(acc[i][j], limit));
             } else {
                 reinterpret_cast<float*>(out)[at] = acc[i][j];
             }
@@ -370,7 +375,7 @@ routed_product_few_kernel(const T* __restrict__ A, const int* __restrict__ pair_
                 if (lane == 0 && nbase + c < N) {
                     const size_t at = (size_t)(row0 + r) * N + nbase + c;
                     if (GATED) reinterpret_cast<T*>(out)[at] = from_float<T>(expert_activation(g, u, limit));
-                    else if (MODE == 2) reinterpret_cast<T*>(out)[at] = from_float<T>(squared_relu(g));
+                    else if (MODE == 2) reinterpret_cast<T*>(out)[at] = from_float<T>(single_activation(g, limit));
                     else reinterpret_cast<float*>(out)[at] = g;
                 }
             }
@@ -404,7 +409,7 @@ routed_product_few_kernel(const T* __restrict__ A, const int* __restrict__ pair_
             if (lane == 0 && r < rows) {
                 const size_t at = (size_t)(row0 + r) * N + n;
                 if (GATED) reinterpret_cast<T*>(out)[at] = from_float<T>(expert_activation(g, u, limit));
-                else if (MODE == 2) reinterpret_cast<T*>(out)[at] = from_float<T>(squared_relu(g));
+                else if (MODE == 2) reinterpret_cast<T*>(out)[at] = from_float<T>(single_activation(g, limit));
                 else reinterpret_cast<float*>(out)[at] = g;
             }
         }
@@ -511,7 +516,7 @@ routed_product_mma_kernel(const bf16* __restrict__ A, const int* __restrict__ pa
                     const size_t at = (size_t)(row0 + r) * N + gn;
                     const float g = stage[warp][0][rr][cc];
                     if (GATED) reinterpret_cast<bf16*>(out)[at] = __float2bfloat16_rn(expert_activation(g, stage[warp][GATED ? 1 : 0][rr][cc], limit));
-                    else if (MODE == 2) reinterpret_cast<bf16*>(out)[at] = __float2bfloat16_rn(squared_relu(g));
+                    else if (MODE == 2) reinterpret_cast<bf16*>(out)[at] = __float2bfloat16_rn(single_activation(g, limit));
                     else reinterpret_cast<float*>(out)[at] = g;
                 }
             }
@@ -634,7 +639,7 @@ routed_product_pipe_kernel(const bf16* __restrict__ A, const int* __restrict__ p
                     const size_t at = (size_t)(row0 + r) * N + gn;
                     const float g = mine[rr * 20 + cc];
                     if (GATED) reinterpret_cast<bf16*>(out)[at] = __float2bfloat16_rn(expert_activation(g, mine[16 * 20 + rr * 20 + cc], limit));
-                    else if (MODE == 2) reinterpret_cast<bf16*>(out)[at] = __float2bfloat16_rn(squared_relu(g));
+                    else if (MODE == 2) reinterpret_cast<bf16*>(out)[at] = __float2bfloat16_rn(single_activation(g, limit));
                     else reinterpret_cast<float*>(out)[at] = g;
                 }
             }
@@ -673,8 +678,8 @@ extern "C" long long fe_routed_experts_workspace(int T, int top, int experts, in
 }
 
 // h [T, D]; chosen, weights [T, top]; gate_up [experts, 2F, D]; down [experts, D, F]; shared [T, D] or null; out [T, D].
-// limit: 0 for silu(gate) * up, else the clamped activation (see expert_activation).  single 1: the experts have no gate,
-// gate_up is [experts, F, D] and an expert is down(relu(up h)^2).  identity: choices in [experts, experts + identity) stand
+// limit: 0 for silu(gate) * up, else the clamped activation (see expert_activation).  single 1 or 2: the experts have no
+// gate, gate_up is [experts, F, D] and an expert is down(relu(up h)^2) (1) or down(gelu(up h)) (2, the exact form).  identity: choices in [experts, experts + identity) stand
 // for experts that return their input.
 extern "C" int fe_routed_experts(const void* h, const int* chosen, const float* weights, const void* gate_up, const void* down,
                                  const void* shared, void* out, void* workspace, long long workspace_bytes, int T, int top,
@@ -706,7 +711,8 @@ extern "C" int fe_routed_experts(const void* h, const int* chosen, const float* 
     const bool few = pairs <= 64 && few_smem1 <= 160 * 1024 && few_smem2 <= 160 * 1024;
     // tensor cores with 128-row tiles and pipelined copies when rows start on 16-byte boundaries in both products
     const bool piped = !few && dtype == FE_BF16 && D % 8 == 0 && F % 8 == 0;
-    FE_REQUIRE(identity >= 0 && (single == 0 || single == 1), "routed_experts: bad options");
+    FE_REQUIRE(identity >= 0 && single >= 0 && single <= 2 && (single == 0 || limit == 0.f), "routed_experts: bad options");
+    const float act_of = single == 0 ? limit : (single == 2 ? SINGLE_GELU : SINGLE_RELU2);
     fe::launch(route_plan_kernel, 1, 256, 0, stream, chosen, (int)pairs, experts, identity, few ? few_rows : (piped ? PBM : BM), offsets,
                row_of_pair, pair_of_row, tiles, tile_expert, tile_row0, status);
     const int* c_pairs = pair_of_row;
@@ -714,7 +720,7 @@ extern "C" int fe_routed_experts(const void* h, const int* chosen, const float* 
     const int *c_offsets = offsets, *c_tiles = tiles, *c_expert = tile_expert, *c_row0 = tile_row0;
 #define FE_ROUTED_PRODUCTS(KERNEL1, KERNEL2, TYPE, GRID1, GRID2, THREADS, SMEM1, SMEM2)                                                   \
     fe::launch(KERNEL1, GRID1, THREADS, SMEM1, stream, (const TYPE*)h, c_pairs, top, (const TYPE*)gate_up, (void*)act, c_offsets, c_tiles, \
-               c_expert, c_row0, F, D, limit);                                                                                            \
+               c_expert, c_row0, F, D, act_of);                                                                                            \
     fe::launch(KERNEL2, GRID2, THREADS, SMEM2, stream, (const TYPE*)act, c_none, top, (const TYPE*)down, (void*)y, c_offsets, c_tiles,    \
                c_expert, c_row0, D, F, 0.f)
     if (few) {

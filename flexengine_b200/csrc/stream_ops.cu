@@ -186,7 +186,7 @@ extern "C" int fe_depth_average(float* history, float* x, const void* a, const v
 // ---------------------------------------------------------------------------------------------
 // Elementwise activations.  kind 0: tanh.  kind 1: xIELU with the two numbers params = (p, q) on the device:
 //   z > 0: softplus(p) z^2 + z/2;    z <= 0: (1/2 + softplus(q)) (exp(z) - 1 - z) + z/2.
-// kind 2: the square of relu(z).
+// kind 2: the square of relu(z).  kind 3: the exact GELU, z/2 (1 + erf(z / sqrt(2))).
 __device__ __forceinline__ float softplusf(float v) { return log1pf(expf(v)); }
 
 template <typename T>
@@ -208,6 +208,7 @@ __global__ void activation_kernel(const T* __restrict__ x, T* __restrict__ out, 
             for (int e = 0; e < 8; ++e) {
                 if (kind == 0) z[e] = tanhf(z[e]);
                 else if (kind == 2) z[e] = z[e] > 0.f ? z[e] * z[e] : 0.f;
+                else if (kind == 3) z[e] = gelu_erf(z[e]);
                 else z[e] = z[e] > 0.f ? fmaf(up * z[e], z[e], 0.5f * z[e]) : fmaf(down, expm1f(z[e]) - z[e], 0.5f * z[e]);
             }
             store8<T>(out + i, z);
@@ -219,6 +220,7 @@ __global__ void activation_kernel(const T* __restrict__ x, T* __restrict__ out, 
         float y;
         if (kind == 0) y = tanhf(z);
         else if (kind == 2) y = z > 0.f ? z * z : 0.f;
+        else if (kind == 3) y = gelu_erf(z);
         else y = z > 0.f ? fmaf(up * z, z, 0.5f * z) : fmaf(down, expm1f(z) - z, 0.5f * z);
         out[i] = from_float<T>(y);
     }
@@ -226,7 +228,7 @@ __global__ void activation_kernel(const T* __restrict__ x, T* __restrict__ out, 
 
 extern "C" int fe_activation(const void* x, void* out, long long n, int kind, const float* params, int dtype,
                              cudaStream_t stream) {
-    FE_REQUIRE(n >= 0 && (kind == 0 || kind == 2 || (kind == 1 && params != nullptr)), "activation: bad arguments (kind %d)", kind);
+    FE_REQUIRE(n >= 0 && (kind == 0 || kind == 2 || kind == 3 || (kind == 1 && params != nullptr)), "activation: bad arguments (kind %d)", kind);
     if (n == 0) return 0;
     const int threads = 256;
     const long long want = (n / 8 + threads) / threads;

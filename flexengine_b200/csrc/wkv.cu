@@ -303,44 +303,54 @@ extern "C" int fe_wkv_recurrence(const void* r, const void* k, const void* v, co
 }
 
 // ---------------------------------------------------------------------------------------------
-// y[t, head] = o[t, head] / sqrt(mean(o[t, head]^2) + eps) * weight * silu(g) * scale: one warp per (token, head).
-// ``weight`` may be null (a unit norm).  A row of g is ldg entries long and a row of out ldo (views of wider buffers).
-template <typename T>
-__global__ void head_rmsnorm_gate_kernel(const float* __restrict__ o, const float* __restrict__ weight, const T* __restrict__ g,
+// y[t, head] = o[t, head] / sqrt(mean(o[t, head]^2) + eps) * weight * act(g) * scale, act silu or sigmoid: one warp per (token,
+// head), or with WIDE one block (a head of many entries, as one norm over all heads of a row is).  ``weight`` may be null (a unit
+// norm).  A row of g (its own type: the compute type or float) is ldg entries long and a row of out ldo (views of wider buffers).
+template <typename T, typename TG, bool WIDE>
+__global__ void head_rmsnorm_gate_kernel(const float* __restrict__ o, const float* __restrict__ weight, const TG* __restrict__ g,
                                          long long ldg, T* __restrict__ out, long long ldo, float eps, float scale, long long pairs,
-                                         int heads, int d) {
+                                         int heads, int d, int sigmoid_gate) {
     griddep_wait();
     griddep_launch_dependents();
-    const long long warp = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (warp >= pairs) return;
-    const int lane = threadIdx.x & 31;
-    const int head = (int)(warp % heads);
-    const long long t = warp / heads;
-    const float* x = o + warp * d;
+    __shared__ float scratch[33];
+    const long long item = WIDE ? blockIdx.x : (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (item >= pairs) return;
+    const int first = WIDE ? threadIdx.x : threadIdx.x & 31, step = WIDE ? blockDim.x : 32;
+    const int head = (int)(item % heads);
+    const long long t = item / heads;
+    const float* x = o + item * d;
     float ss = 0.f;
-    for (int i = lane; i < d; i += 32) ss += x[i] * x[i];
-    ss = warp_sum(ss);
+    for (int i = first; i < d; i += step) ss += x[i] * x[i];
+    ss = WIDE ? block_sum(ss, scratch) : warp_sum(ss);
     const float inv = rsqrtf(ss / (float)d + eps) * scale;
-    for (int i = lane; i < d; i += 32) {
+    for (int i = first; i < d; i += step) {
         const float gate = to_float(g[t * ldg + head * d + i]);
         const float w = weight ? weight[head * d + i] : 1.f;
-        out[t * ldo + head * d + i] = from_float<T>(x[i] * inv * w * (gate / (1.f + expf(-gate))));
+        out[t * ldo + head * d + i] = from_float<T>(x[i] * inv * w * ((sigmoid_gate ? 1.f : gate) / (1.f + expf(-gate))));
     }
 }
 
-extern "C" int fe_head_rmsnorm_gate(const float* o, const float* weight, const void* g, long long ldg, void* out, long long ldo, float eps,
-                                    float scale, int T, int heads, int d, int dtype, cudaStream_t stream) {
-    FE_REQUIRE(T >= 0 && heads > 0 && d > 0 && ldg >= (long long)heads * d && ldo >= (long long)heads * d, "head_rmsnorm_gate: bad sizes");
-    if (T == 0) return 0;
-    const long long pairs = (long long)T * heads;
-    const unsigned blocks = (unsigned)((pairs + 3) / 4);
-    if (dtype == FE_F32)
-        fe::launch(head_rmsnorm_gate_kernel<float>, blocks, 128, 0, stream, o, weight, (const float*)g, ldg, (float*)out, ldo, eps, scale,
-                   pairs, heads, d);
-    else if (dtype == FE_BF16)
-        fe::launch(head_rmsnorm_gate_kernel<bf16>, blocks, 128, 0, stream, o, weight, (const bf16*)g, ldg, (bf16*)out, ldo, eps, scale,
-                   pairs, heads, d);
+template <typename T, typename TG>
+static int launch_head_rmsnorm_gate(const float* o, const float* weight, const void* g, long long ldg, void* out, long long ldo, float eps,
+                                    float scale, int T_tokens, int heads, int d, int sigmoid_gate, cudaStream_t stream) {
+    const long long pairs = (long long)T_tokens * heads;
+    if (d > 512)
+        fe::launch(head_rmsnorm_gate_kernel<T, TG, true>, (unsigned)pairs, 256, 0, stream, o, weight, (const TG*)g, ldg, (T*)out, ldo, eps, scale,
+                   pairs, heads, d, sigmoid_gate);
     else
-        FE_REQUIRE(false, "head_rmsnorm_gate: unknown dtype %d", dtype);
+        fe::launch(head_rmsnorm_gate_kernel<T, TG, false>, (unsigned)((pairs + 3) / 4), 128, 0, stream, o, weight, (const TG*)g, ldg, (T*)out,
+                   ldo, eps, scale, pairs, heads, d, sigmoid_gate);
     return fe_check_launch("head_rmsnorm_gate");
+}
+
+extern "C" int fe_head_rmsnorm_gate(const float* o, const float* weight, const void* g, int g_dtype, long long ldg, void* out, long long ldo,
+                                    float eps, float scale, int T, int heads, int d, int sigmoid_gate, int dtype, cudaStream_t stream) {
+    FE_REQUIRE(T >= 0 && heads > 0 && d > 0 && ldg >= (long long)heads * d && ldo >= (long long)heads * d, "head_rmsnorm_gate: bad sizes");
+    FE_REQUIRE((dtype == FE_F32 || dtype == FE_BF16) && (g_dtype == FE_F32 || g_dtype == dtype), "head_rmsnorm_gate: unknown dtypes %d, %d", dtype, g_dtype);
+    if (T == 0) return 0;
+    if (dtype == FE_F32)
+        return launch_head_rmsnorm_gate<float, float>(o, weight, g, ldg, out, ldo, eps, scale, T, heads, d, sigmoid_gate, stream);
+    if (g_dtype == FE_F32)
+        return launch_head_rmsnorm_gate<bf16, float>(o, weight, g, ldg, out, ldo, eps, scale, T, heads, d, sigmoid_gate, stream);
+    return launch_head_rmsnorm_gate<bf16, bf16>(o, weight, g, ldg, out, ldo, eps, scale, T, heads, d, sigmoid_gate, stream);
 }

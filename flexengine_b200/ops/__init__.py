@@ -207,6 +207,31 @@ def add_rmsnorm(residual, delta, weight, eps, out_dtype, rows=None, upcoming=Non
     return out
 
 
+def add_layernorm(residual, delta, weight, bias, eps, out_dtype, rows=None, post=None, plus=None):
+    """Fused residual add + layer norm, w (x - mean) / sqrt(variance + eps) + b; ``rows`` as in ``add_rmsnorm``.  ``post`` =
+    (weight, bias, eps, scale, bias still to add or None): the branch output goes through a layer norm of its own on its way
+    into the stream, times ``scale``; delta may be float32 whatever the compute dtype.  ``plus`` (float32, shaped like the
+    residual): rows that are added to the stream as well."""
+    post_w, post_b, post_eps, post_scale, y_bias = post if post is not None else (None, None, 0.0, 1.0, None)
+    _need_cuda(residual, delta, weight, bias, rows, post_w, post_b, y_bias, plus)
+    T, H = residual.shape
+    if residual.dtype != torch.float32 or not residual.is_contiguous():
+        raise TypeError("the residual stream is contiguous float32")
+    for vector in (weight, bias, post_w, post_b, y_bias):
+        if vector is not None and (vector.dtype != torch.float32 or vector.numel() != H):
+            raise TypeError("norm weights and biases are float32 vectors of the stream's width")
+    if delta is not None and (delta.dtype not in (torch.float32, out_dtype) or tuple(delta.shape) != (T, H) or not delta.is_contiguous()):
+        raise ValueError("a branch output is contiguous, shaped like the residual, float32 or in the compute dtype")
+    if plus is not None and (plus.dtype != torch.float32 or plus.shape != residual.shape or not plus.is_contiguous()):
+        raise ValueError("what is added to the stream is contiguous float32, shaped like it")
+    n_out = T if rows is None else rows.numel()
+    out = torch.empty((n_out, H), dtype=out_dtype, device=residual.device)
+    _run(_core(), "fe_layer_norm", _ptr(residual), _ptr(delta), _c_int(_code(delta.dtype) if delta is not None else 0), _ptr(y_bias),
+         _ptr(post_w), _ptr(post_b), _c_float(post_eps), _c_float(post_scale), _ptr(plus), _ptr(weight), _ptr(bias), _c_float(eps),
+         _ptr(out), _ptr(rows), _c_int(n_out), _c_int(H), _c_int(T), _c_int(_code(out_dtype)), _stream())
+    return out
+
+
 FUSES_RESIDUAL_NORM = True      # linear(..., follow=) may end a branch: see Prenormed
 
 
@@ -303,8 +328,9 @@ def linear(x, w, bias=None, out_float32=False, follow=None, upcoming=None):
 SKINNY_MAX_ROWS = 8          # beyond this the library product is as fast or faster
 SKINNY_QKV_MAX_ROWS = 8      # the fused projection + bias + rotation + cache write takes one 8-row tile of tokens
 EPI_BF16, EPI_F32, EPI_SWIGLU, EPI_GEGLU = 0, 1, 2, 5      # 5: the gated epilogue with the tanh form of GELU
-EPI_RELU2 = 6                                               # relu(product)^2, no gate
-GATED_EPILOGUES = {"silu": EPI_SWIGLU, "gelu_tanh": EPI_GEGLU}
+EPI_RELU2, EPI_REGLU, EPI_GELU = 6, 7, 8                    # relu(product)^2, no gate; the gated epilogue with relu; the exact GELU, no gate
+GATED_EPILOGUES = {"silu": EPI_SWIGLU, "gelu_tanh": EPI_GEGLU, "relu": EPI_REGLU}
+SINGLE_EPILOGUES = {"relu2": EPI_RELU2, "gelu": EPI_GELU}
 
 
 def skinny_ok(x, w) -> bool:
@@ -320,7 +346,7 @@ def skinny_gemm(x, w, epilogue: int = EPI_BF16, upcoming=None):
     x, sumsq, tiles, eps = _rows_and_scale(x)
     M, K = x.shape
     N = w.shape[0]
-    if epilogue in (EPI_SWIGLU, EPI_GEGLU):
+    if epilogue in (EPI_SWIGLU, EPI_GEGLU, EPI_REGLU):
         out = torch.empty((M, N // 2), dtype=torch.bfloat16, device=x.device)
     else:
         out = torch.empty((M, N), dtype=torch.float32 if epilogue == EPI_F32 else torch.bfloat16, device=x.device)
@@ -347,13 +373,13 @@ def tcgen05_ok(x, w) -> bool:
 
 def gemm_tcgen05(x, w, epilogue: int = EPI_BF16):
     """x [M, K] times w [N, K]^T on tcgen05 tensor cores (TMA operands, TMEM accumulator);
-    epilogue EPI_BF16, EPI_SWIGLU, EPI_GEGLU or EPI_RELU2.  See csrc/gemm_tcgen05.cu."""
+    epilogue EPI_BF16, EPI_SWIGLU, EPI_GEGLU, EPI_REGLU, EPI_RELU2 or EPI_GELU.  See csrc/gemm_tcgen05.cu."""
     _need_cuda(x, w)
     M, K = x.shape
     N = w.shape[0]
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or not x.is_contiguous() or not w.is_contiguous():
         raise TypeError("gemm_tcgen05 takes contiguous bfloat16 operands")
-    out = torch.empty((M, N // 2 if epilogue in (EPI_SWIGLU, EPI_GEGLU) else N), dtype=torch.bfloat16, device=x.device)
+    out = torch.empty((M, N // 2 if epilogue in (EPI_SWIGLU, EPI_GEGLU, EPI_REGLU) else N), dtype=torch.bfloat16, device=x.device)
     _run(_bf16(), "fe_gemm_tcgen05", _ptr(x), _ptr(w), _ptr(out), _c_int(M), _c_int(N), _c_int(K), _c_int(epilogue),
          _ptr(status_word(x.device)), _stream())
     return out
@@ -383,11 +409,11 @@ def linear_swiglu(x, w, intermediate, upcoming=None):
     return swiglu(linear(x, w), intermediate)
 
 
-GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
+GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu": 2}
 
 
 def gated_activation(gate_up, intermediate, activation, bias=None, out_dtype=None):
-    """act(gate) * up of rows [gate | up]; act "silu" or "gelu_tanh" (the tanh form of GELU), float arithmetic.  ``bias``
+    """act(gate) * up of rows [gate | up]; act "silu", "relu" or "gelu_tanh" (the tanh form of GELU), float arithmetic.  ``bias``
     (float32 [2 * intermediate]) is added to both first; the rows may then be a float32 product and ``out_dtype`` the
     compute dtype."""
     _need_cuda(gate_up, bias)
@@ -411,7 +437,7 @@ def gated_activation(gate_up, intermediate, activation, bias=None, out_dtype=Non
 
 
 def linear_gated(x, w, intermediate, activation):
-    """act(x Wg^T) * (x Wu^T) with w = [Wg; Wu] ([2I, K]), act "silu" or "gelu_tanh": the weight-streaming kernel for a
+    """act(x Wg^T) * (x Wu^T) with w = [Wg; Wu] ([2I, K]), act "silu", "gelu_tanh" or "relu": the weight-streaming kernel for a
     handful of rows and the tcgen05 kernel for a prompt's worth apply the gate's function in their epilogues; otherwise
     the product and the activation kernel."""
     if activation == "silu":
@@ -493,22 +519,32 @@ def qkv_projection(h, w, bias, positions, inv_freq, rot, slot_mapping, k_cache, 
     return qkv
 
 
-ATTENTION_SINK, ATTENTION_SIGMOID = 1, 2       # bits of the attention kernels' mode
+ATTENTION_SINK, ATTENTION_SIGMOID, ATTENTION_MAPPED = 1, 2, 4       # bits of the attention kernels' mode
 
 
-def _attention_mode(sink: bool, sigmoid: bool) -> int:
-    return (ATTENTION_SINK if sink else 0) | (ATTENTION_SIGMOID if sigmoid else 0)
+def _attention_mode(sink: bool, sigmoid: bool, mapped: bool = False) -> int:
+    return (ATTENTION_SINK if sink else 0) | (ATTENTION_SIGMOID if sigmoid else 0) | (ATTENTION_MAPPED if mapped else 0)
+
+
+def _score_map(sigmoid, head_bias, softcap, head_scales):
+    """(mapped, the numbers per head, softcap) as the kernels take them: biases under sigmoid weights, else factors of the scores."""
+    mapped = softcap > 0.0 or head_scales is not None
+    if mapped and (sigmoid or softcap < 0.0):
+        raise ValueError("softcap and head scales belong to a softmax; softcap is not negative")
+    return mapped, (head_scales if mapped else head_bias), (float(softcap) if mapped else 0.0)
 
 
 def paged_attention_simt(q, q_stride, k_cache, v_cache, block_table, cu_q, q_start, token_request, T, nq, nkv, d,
-                         page_size, scale, window, sink=False, sigmoid=False, head_bias=None):
+                         page_size, scale, window, sink=False, sigmoid=False, head_bias=None, softcap=0.0,
+                         head_scales=None):
     out = torch.empty((T, nq * d), dtype=k_cache.dtype, device=k_cache.device)
-    mode = _attention_mode(sink, sigmoid)
+    mapped, per_head, softcap = _score_map(sigmoid, head_bias, softcap, head_scales)
+    mode = _attention_mode(sink, sigmoid, mapped)
     _run(_core(), "fe_paged_attention_simt", _ptr(q), _c_ll(q_stride), _ptr(out), _c_ll(nq * d), _ptr(k_cache),
          _ptr(v_cache), _ptr(block_table), _c_int(block_table.shape[1]), _ptr(cu_q), _ptr(q_start),
          _ptr(token_request), _c_int(T), _c_int(nq), _c_int(nkv), _c_int(d), _c_int(page_size),
          _c_int(k_cache.shape[0]), _c_float(scale), _c_int(window), _c_int(mode), _c_int(_code(k_cache.dtype)),
-         _ptr(status_word(k_cache.device)), _ptr(head_bias), _stream())
+         _ptr(status_word(k_cache.device)), _ptr(per_head), _c_float(softcap), _stream())
     return out
 
 
@@ -568,21 +604,23 @@ def decode_splits(requests: int, nkv: int, max_ctx_len: int, sms: int | None = N
 
 
 def paged_decode_mma(q, q_stride, k_cache, v_cache, block_table, cu_q, q_start, requests, nq, nkv, d, page_size,
-                     scale, window, splits, out=None, upcoming=None, sink=False, sigmoid=False, head_bias=None):
+                     scale, window, splits, out=None, upcoming=None, sink=False, sigmoid=False, head_bias=None, softcap=0.0,
+                     head_scales=None):
     """Tensor-core decode attention (one token per request), keys split ``splits`` ways.  ``upcoming``: the
     matrix that the next kernel streams (the output projection); extra blocks of the merge kernel ask for its
     start to be brought into L2."""
     if out is None:
         out = torch.empty((requests, nq * d), dtype=torch.bfloat16, device=k_cache.device)
+    mapped, per_head, softcap = _score_map(sigmoid, head_bias, softcap, head_scales)
     lib = _bf16()
     need = lib.fe_paged_decode_scratch_bytes(_c_int(requests), _c_int(nq), _c_int(d), _c_int(splits))
     work = scratch(k_cache.device, need) if need else None
     _run(lib, "fe_paged_decode_mma_upcoming", _ptr(q), _c_ll(q_stride), _ptr(out), _c_ll(out.stride(0)), _ptr(work),
          _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _c_int(block_table.shape[1]), _ptr(cu_q), _ptr(q_start),
          _c_int(requests), _c_int(nq), _c_int(nkv), _c_int(d), _c_int(page_size), _c_int(k_cache.shape[0]),
-         _c_float(scale), _c_int(window), _c_int(_attention_mode(sink, sigmoid)), _c_int(splits),
+         _c_float(scale), _c_int(window), _c_int(_attention_mode(sink, sigmoid, mapped)), _c_int(splits),
          *_upcoming(upcoming, requests, UPCOMING_BYTES_MERGE),
-         _ptr(status_word(k_cache.device)), _ptr(head_bias), _stream())
+         _ptr(status_word(k_cache.device)), _ptr(per_head), _c_float(softcap), _stream())
     return out
 
 
@@ -627,27 +665,31 @@ def decode_cluster_splits(splits: int, max_ctx_len: int, clusters: int = 0, resi
 
 
 def paged_decode_cluster(q, q_stride, k_cache, v_cache, block_table, cu_q, q_start, requests, nq, nkv, d, page_size,
-                         scale, window, splits, out=None, sink=False, sigmoid=False, head_bias=None):
+                         scale, window, splits, out=None, sink=False, sigmoid=False, head_bias=None, softcap=0.0,
+                         head_scales=None):
     """Decode attention with the splits of each (request, key/value head) as one thread-block cluster that merges
     its partial results through distributed shared memory: one launch, no scratch memory; splits <= 16."""
     if out is None:
         out = torch.empty((requests, nq * d), dtype=torch.bfloat16, device=k_cache.device)
+    mapped, per_head, softcap = _score_map(sigmoid, head_bias, softcap, head_scales)
     _run(_bf16(), "fe_paged_decode_cluster", _ptr(q), _c_ll(q_stride), _ptr(out), _c_ll(out.stride(0)), _ptr(k_cache),
          _ptr(v_cache), _ptr(block_table), _c_int(block_table.shape[1]), _ptr(cu_q), _ptr(q_start), _c_int(requests),
          _c_int(nq), _c_int(nkv), _c_int(d), _c_int(page_size), _c_int(k_cache.shape[0]), _c_float(scale), _c_int(window),
-         _c_int(_attention_mode(sink, sigmoid)), _c_int(splits), _ptr(status_word(k_cache.device)), _ptr(head_bias), _stream())
+         _c_int(_attention_mode(sink, sigmoid, mapped)), _c_int(splits), _ptr(status_word(k_cache.device)), _ptr(per_head), _c_float(softcap), _stream())
     return out
 
 
 def paged_prefill_mma(q, q_stride, k_cache, v_cache, block_table, cu_q, q_start, T, requests, max_q_len, nq, nkv, d,
-                      page_size, scale, window, sink=False, sigmoid=False, head_bias=None):
+                      page_size, scale, window, sink=False, sigmoid=False, head_bias=None, softcap=0.0,
+                      head_scales=None):
     """Tensor-core attention for portions of any length (decoded tokens are portions of one)."""
     out = torch.empty((T, nq * d), dtype=torch.bfloat16, device=k_cache.device)
+    mapped, per_head, softcap = _score_map(sigmoid, head_bias, softcap, head_scales)
     _run(_bf16(), "fe_paged_prefill_mma", _ptr(q), _c_ll(q_stride), _ptr(out), _c_ll(nq * d), _ptr(k_cache),
          _ptr(v_cache), _ptr(block_table), _c_int(block_table.shape[1]), _ptr(cu_q), _ptr(q_start), _c_int(requests),
          _c_int(max_q_len), _c_int(nq), _c_int(nkv), _c_int(d), _c_int(page_size), _c_int(k_cache.shape[0]),
-         _c_float(scale), _c_int(window), _c_int(_attention_mode(sink, sigmoid)), _ptr(status_word(k_cache.device)), _ptr(head_bias),
-         _stream())
+         _c_float(scale), _c_int(window), _c_int(_attention_mode(sink, sigmoid, mapped)), _ptr(status_word(k_cache.device)), _ptr(per_head),
+         _c_float(softcap), _stream())
     return out
 
 
@@ -691,27 +733,30 @@ def prefill_splits(lengths, starts, nq, nkv, window=0, sms: int | None = None) -
 
 
 def paged_prefill_tcgen05(q, q_stride, k_cache, v_cache, block_table, cu_q, q_start, T, requests, max_q_len, nq, nkv, d,
-                          page_size, scale, window, splits=1, sink=False, sigmoid=False, head_bias=None):
+                          page_size, scale, window, splits=1, sink=False, sigmoid=False, head_bias=None, softcap=0.0,
+                          head_scales=None):
     """Prefill attention on tcgen05 tensor cores: 128 (query, head) rows a block, head sizes 64 and 128.
     ``splits`` > 1 shares the keys of each pair of row tiles out over that many blocks and merges their results."""
     out = torch.empty((T, nq * d), dtype=torch.bfloat16, device=k_cache.device)
     part = scratch(k_cache.device, 4 * T * nq * splits * (d + 1)) if splits > 1 else None
+    mapped, per_head, softcap = _score_map(sigmoid, head_bias, softcap, head_scales)
     _run(_bf16(), "fe_paged_prefill_tcgen05", _ptr(q), _c_ll(q_stride), _ptr(out), _c_ll(nq * d), _ptr(k_cache),
          _ptr(v_cache), _ptr(block_table), _c_int(block_table.shape[1]), _ptr(cu_q), _ptr(q_start), _c_int(requests),
          _c_int(max_q_len), _c_int(nq), _c_int(nkv), _c_int(d), _c_int(page_size), _c_int(k_cache.shape[0]),
-         _c_float(scale), _c_int(window), _c_int(_attention_mode(sink, sigmoid)), _c_int(splits), _ptr(part),
-         _c_ll(T), _ptr(status_word(k_cache.device)), _ptr(head_bias), _stream())
+         _c_float(scale), _c_int(window), _c_int(_attention_mode(sink, sigmoid, mapped)), _c_int(splits), _ptr(part),
+         _c_ll(T), _ptr(status_word(k_cache.device)), _ptr(per_head), _c_float(softcap), _stream())
     return out
 
 
 def paged_attention(qkv, k_cache, v_cache, block_table, ctx, nq, nkv, d, page_size, scale, window, upcoming=None, sink=False,
-                    weights="softmax", head_bias=None):
+                    weights="softmax", head_bias=None, softcap=0.0, head_scales=None):
     """Causal grouped-query attention of the step's tokens over their requests' pages.
     qkv [T, >= nq d] holds the (rotated) queries in its first nq d columns; returns [T, nq d].
     ``window``: what a query sees of the earlier keys: 0 all of them, w > 0 the last w, -c < 0 those of its own chunk of
     c positions (counted from position 0).  ``sink``: 1 is added to the softmax's denominator.
     ``weights`` "sigmoid": no softmax; a visible key weighs sigmoid(score + head_bias[head]) (``head_bias`` float32 [nq] or
-    None), not normalised over the keys.
+    None), not normalised over the keys.  ``head_scales`` (float32 [nq]): scores are multiplied by the head's number as well as
+    by ``scale``; ``softcap`` > 0: they then become softcap * tanh(score / softcap), before the softmax.
     float32 runs on CUDA cores (true 32-bit); bfloat16 on tensor cores: the split-KV decode
     kernel when every request brings one token, else a prefill kernel (tcgen05 for portions of
     head size 64 or 128, mma.sync otherwise)."""
@@ -726,9 +771,14 @@ def paged_attention(qkv, k_cache, v_cache, block_table, ctx, nq, nkv, d, page_si
         _need_cuda(head_bias)
         if not sigmoid or head_bias.dtype != torch.float32 or head_bias.numel() != nq:
             raise ValueError("paged_attention: a head bias goes with sigmoid weights and is float32 [heads]")
+    if head_scales is not None:
+        _need_cuda(head_scales)
+        if head_scales.dtype != torch.float32 or head_scales.numel() != nq:
+            raise ValueError("paged_attention: head scales are float32 [heads]")
+    score = {"softcap": softcap, "head_scales": head_scales}
     if qkv.dtype == torch.float32 or d > 256:          # the tensor-core kernels take head sizes up to 256
         return paged_attention_simt(qkv, qkv.stride(0), k_cache, v_cache, block_table, ctx.cu_q, ctx.q_start,
-                                    ctx.token_request, T, nq, nkv, d, page_size, scale, window, sink, sigmoid, head_bias)
+                                    ctx.token_request, T, nq, nkv, d, page_size, scale, window, sink, sigmoid, head_bias, **score)
     requests = ctx.cu_q.numel() - 1
     if ctx.max_q_len == 1 and nq // nkv <= 16:
         # a window or a chunk bounds the keys a token walks (plus the tile of 32 that its first key lies in)
@@ -738,18 +788,18 @@ def paged_attention(qkv, k_cache, v_cache, block_table, ctx, nq, nkv, d, page_si
                                           lambda s: clusters_resident(requests, nq, nkv, d, s))
         if clustered:
             return paged_decode_cluster(qkv, qkv.stride(0), k_cache, v_cache, block_table, ctx.cu_q, ctx.q_start, requests,
-                                        nq, nkv, d, page_size, scale, window, clustered, sink=sink, sigmoid=sigmoid, head_bias=head_bias)
+                                        nq, nkv, d, page_size, scale, window, clustered, sink=sink, sigmoid=sigmoid, head_bias=head_bias, **score)
         return paged_decode_mma(qkv, qkv.stride(0), k_cache, v_cache, block_table, ctx.cu_q, ctx.q_start, requests,
                                 nq, nkv, d, page_size, scale, window, splits, upcoming=upcoming, sink=sink, sigmoid=sigmoid,
-                                head_bias=head_bias)
+                                head_bias=head_bias, **score)
     lengths = getattr(ctx, "host_lengths", None)
     if tcgen05_attention_ok(ctx.max_q_len, nq, nkv, d, lengths, getattr(ctx, "host_starts", None)):
         splits = prefill_splits(lengths, ctx.host_starts, nq, nkv, window) if lengths else 1
         return paged_prefill_tcgen05(qkv, qkv.stride(0), k_cache, v_cache, block_table, ctx.cu_q, ctx.q_start, T, requests,
                                      ctx.max_q_len, nq, nkv, d, page_size, scale, window, splits, sink=sink, sigmoid=sigmoid,
-                                     head_bias=head_bias)
+                                     head_bias=head_bias, **score)
     return paged_prefill_mma(qkv, qkv.stride(0), k_cache, v_cache, block_table, ctx.cu_q, ctx.q_start, T, requests,
-                             ctx.max_q_len, nq, nkv, d, page_size, scale, window, sink=sink, sigmoid=sigmoid, head_bias=head_bias)
+                             ctx.max_q_len, nq, nkv, d, page_size, scale, window, sink=sink, sigmoid=sigmoid, head_bias=head_bias, **score)
 
 
 # ---- several residual streams, token shift, gated attention, minGRU ---------------------------------------------
@@ -812,7 +862,7 @@ def token_shift(h, mu, kept, state_slots, cu_q, token_request):
 
 def qkv_conv_rope_norm_cache(projected, conv, history, taps, state_slots, cu_q, token_request, positions, inv_freq, rot_dims,
                              qk_norm, eps, slot_mapping, k_cache, v_cache, heads, kv_heads, dim, vdim, head, page_size,
-                             q_weight=None, k_weight=None, temp=None):
+                             q_weight=None, k_weight=None, temp=None, value_norm=False):
     """What attention does between its projection and its scores, in one kernel (csrc/hyper_ops.cu).  ``projected``
     [T, >= channels] holds q | k | v (``heads`` and ``kv_heads`` heads of ``dim``, ``kv_heads`` of ``vdim``).  A causal
     convolution of ``taps`` taps over time per channel (``conv`` [taps, channels] float32, tap by tap, None for none; ``history``
@@ -822,7 +872,9 @@ def qkv_conv_rope_norm_cache(projected, conv, history, taps, state_slots, cu_q, 
     [pages, kv_heads, page_size, head] (slot_mapping None: no write) and the queries returned [T, heads head], all padded
     with zeros from dim or vdim to ``head``.  ``q_weight``, ``k_weight`` (float32 [dim]): weights of the query and the key
     norm, shared by the heads.  ``temp`` = (coef, every): the query at position p is then multiplied by
-    1 + coef * ln(floor((p + 1) / every) + 1)."""
+    1 + coef * ln(floor((p + 1) / every) + 1).  ``value_norm``: every value head is divided by its root mean square.
+    Queries that need nothing at all (no convolution, rotation, norm, temperature or padding) stay where they are: the
+    projection itself comes back, its first heads * head columns are the queries."""
     _need_cuda(projected, conv, history, state_slots, cu_q, token_request, positions, inv_freq, slot_mapping, k_cache, v_cache,
                q_weight, k_weight)
     if (q_weight is None) != (k_weight is None) or any(w is not None and (w.dtype != torch.float32 or w.numel() != dim)
@@ -845,7 +897,9 @@ def qkv_conv_rope_norm_cache(projected, conv, history, taps, state_slots, cu_q, 
         raise ValueError("qkv_conv_rope_norm_cache: history is float32 [seats, (taps - 1) channels]")
     if inv_freq is not None and (inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_dims // 2):
         raise ValueError("inv_freq must be float32 [rot_dims / 2]")
-    queries = torch.empty((T, heads * head), dtype=projected.dtype, device=projected.device)
+    in_place = (conv is None and inv_freq is None and not qk_norm and temp is None and head == dim and projected.stride(0) % 8 == 0
+                and projected.data_ptr() % 16 == 0)
+    queries = None if in_place else torch.empty((T, heads * head), dtype=projected.dtype, device=projected.device)
     seats = history.shape[0] if history is not None else 0
     _run(_core(), "fe_qkv_conv_rope_norm_cache", _ptr(projected), _c_ll(projected.stride(0)), _ptr(conv), _ptr(history if taps > 1 else None),
          _c_ll(history.stride(0) if history is not None else 0), _c_int(taps), _ptr(state_slots), _ptr(cu_q), _ptr(token_request),
@@ -853,8 +907,8 @@ def qkv_conv_rope_norm_cache(projected, conv, history, taps, state_slots, cu_q, 
          _ptr(slot_mapping), _ptr(k_cache), _ptr(v_cache), _ptr(queries), _c_int(T), _c_int(heads), _c_int(kv_heads), _c_int(dim),
          _c_int(vdim), _c_int(head), _c_int(page_size), _c_ll(k_cache.shape[0] * page_size), _c_int(seats),
          _c_int(_code(projected.dtype)), _ptr(status_word(projected.device)), _ptr(q_weight), _ptr(k_weight), _c_float(temp_coef),
-         _c_int(temp_every), _stream())
-    return queries
+         _c_int(temp_every), _c_int(1 if value_norm else 0), _stream())
+    return projected if in_place else queries
 
 
 ROTATION_PAIRS = {"halves": 0, "interleaved": 1}
@@ -1012,11 +1066,11 @@ def depth_average(history, x, mixed, fed, alpha, depth):
          _c_ll(x.numel()), _c_int(_code(mixed.dtype)), _stream())
 
 
-ACTIVATIONS = {"tanh": 0, "xielu": 1, "relu2": 2}
+ACTIVATIONS = {"tanh": 0, "xielu": 1, "relu2": 2, "gelu": 3}
 
 
 def activation(x, kind, params=None):
-    """Elementwise, float arithmetic, the input's dtype out: "tanh", "relu2" (the square of relu), or "xielu" with
+    """Elementwise, float arithmetic, the input's dtype out: "tanh", "relu2" (the square of relu), "gelu" (the exact form), or "xielu" with
     params = (p, q) on the device: z > 0: softplus(p) z^2 + z/2; z <= 0: (1/2 + softplus(q)) (exp(z) - 1 - z) + z/2."""
     _need_cuda(x, params)
     if kind not in ACTIVATIONS:
@@ -1030,14 +1084,14 @@ def activation(x, kind, params=None):
 
 
 def linear_activated(x, w, kind):
-    """act(x w^T) for an activation without parameters ("relu2", "tanh").  The square of relu is an epilogue of the
+    """act(x w^T) for an activation without parameters ("relu2", "gelu", "tanh").  The first two are epilogues of the
     weight-streaming kernel (a handful of rows) and of the tcgen05 kernel (a prompt's worth); otherwise the product, then the
     activation kernel."""
-    if kind == "relu2" and not isinstance(x, Prenormed):
+    if kind in SINGLE_EPILOGUES and not isinstance(x, Prenormed):
         if _fits(x, w) == "skinny":
-            return skinny_gemm(x, w, EPI_RELU2)
+            return skinny_gemm(x, w, SINGLE_EPILOGUES[kind])
         if tcgen05_ok(x, w):
-            return gemm_tcgen05(x, w, EPI_RELU2)
+            return gemm_tcgen05(x, w, SINGLE_EPILOGUES[kind])
     return activation(linear(x, w), kind)
 
 
@@ -1075,19 +1129,26 @@ def wkv_recurrence(r, k, v, decay_logits, w0, u, state, state_slots, cu_q, heads
     return out
 
 
-def head_rmsnorm_gate(out, weight, g, eps, heads, out_dtype, scale=1.0, into=None):
+HEAD_GATES = ("silu", "sigmoid")
+
+
+def head_rmsnorm_gate(out, weight, g, eps, heads, out_dtype, scale=1.0, into=None, gate="silu"):
     """Every head of ``out`` (float32 [T, heads dim]) divided by its root mean square, times ``weight`` (None: a unit norm),
-    times silu(g), times ``scale``.  ``g`` and ``into`` (where the rows go) may be views with any row stride."""
+    times silu(g) (``gate`` "sigmoid": sigmoid(g)), times ``scale``.  ``g`` (in the compute dtype or float32) and ``into`` (where
+    the rows go) may be views with any row stride.  With ``heads`` 1 the whole row has one root mean square."""
     _need_cuda(out, weight, g, into)
+    if gate not in HEAD_GATES:
+        raise ValueError(f"unknown gate {gate!r}; known: {HEAD_GATES}")
     T, inner = out.shape
-    if out.dtype != torch.float32 or (weight is not None and weight.dtype != torch.float32) or g.dtype != out_dtype \
+    if out.dtype != torch.float32 or (weight is not None and weight.dtype != torch.float32) or g.dtype not in (out_dtype, torch.float32) \
             or tuple(g.shape) != (T, inner) or not out.is_contiguous() or g.stride(1) != 1 or inner % heads:
         raise ValueError("head_rmsnorm_gate: float32 rows and weight, a gate of the same shape in the compute dtype")
     y = into if into is not None else torch.empty((T, inner), dtype=out_dtype, device=out.device)
     if tuple(y.shape) != (T, inner) or y.dtype != out_dtype or y.stride(1) != 1:
         raise ValueError("head_rmsnorm_gate: the rows go to [T, heads dim] in the compute dtype with unit column stride")
-    _run(_core(), "fe_head_rmsnorm_gate", _ptr(out), _ptr(weight), _ptr(g), _c_ll(g.stride(0)), _ptr(y), _c_ll(y.stride(0)),
-         _c_float(eps), _c_float(scale), _c_int(T), _c_int(heads), _c_int(inner // heads), _c_int(_code(out_dtype)), _stream())
+    _run(_core(), "fe_head_rmsnorm_gate", _ptr(out), _ptr(weight), _ptr(g), _c_int(_code(g.dtype)), _c_ll(g.stride(0)), _ptr(y),
+         _c_ll(y.stride(0)), _c_float(eps), _c_float(scale), _c_int(T), _c_int(heads), _c_int(inner // heads),
+         _c_int(HEAD_GATES.index(gate)), _c_int(_code(out_dtype)), _stream())
     return y
 
 
@@ -1112,6 +1173,20 @@ def rotate_heads(projected, heads, dim, positions, inv_freq, rot_dims, scales):
     return out
 
 
+def activate_rows(projected, columns, activation, scales):
+    """float32 [T, columns]: silu of the first ``columns`` columns of ``projected`` (any row stride); ``scales`` ((count, factor),
+    (count, factor)) multiplies the first run of columns by one factor and the second by another."""
+    _need_cuda(projected)
+    T = projected.shape[0]
+    (n0, f0), (n1, f1) = scales
+    if activation != "silu" or projected.dim() != 2 or projected.shape[1] < columns or projected.stride(1) != 1 or n0 + n1 > columns:
+        raise ValueError("activate_rows: silu of columns that the projection has, with unit column stride")
+    out = torch.empty((T, columns), dtype=torch.float32, device=projected.device)
+    _run(_core(), "fe_activate_rows", _ptr(projected), _c_ll(projected.stride(0)), _ptr(out), _c_int(T), _c_int(columns), _c_int(n0),
+         _c_float(f0), _c_int(n0 + n1), _c_float(f1), _c_int(_code(projected.dtype)), _stream())
+    return out
+
+
 # a step whose longest portion has this many tokens or more runs the recurrence in blocks of tokens
 RETENTION_CHUNKS_FROM = 32
 
@@ -1119,35 +1194,38 @@ RETENTION_CHUNKS_FROM = 32
 def retention_scan(qk, values, decay, state, state_slots, cu_q, heads, dim, vdim, max_q_len=0):
     """S <- decay_h S + k_t v_t^T, o_t = S^T q_t per request and head over the step's tokens (csrc/retention.cu); S [dim, vdim]
     float32 lives in ``state[seat, : heads dim vdim]`` (zeros and nothing kept for a seat below 0).  qk float32
-    [T, 2 heads dim] (queries, then keys); values [T, heads vdim] with any row stride; returns float32 [T, heads vdim]."""
+    [T, 2 heads dim] (queries, then keys) with any row stride; values [T, heads vdim] with any row stride; returns float32 [T, heads vdim]."""
     _need_cuda(qk, values, decay, state, state_slots, cu_q)
     T = qk.shape[0]
-    if qk.dtype != torch.float32 or tuple(qk.shape) != (T, 2 * heads * dim) or not qk.is_contiguous() or decay.dtype != torch.float32 \
+    if qk.dtype != torch.float32 or tuple(qk.shape) != (T, 2 * heads * dim) or qk.stride(1) != 1 or decay.dtype != torch.float32 \
             or decay.numel() != heads or state.dtype != torch.float32 or state.stride(-1) != 1 or state.shape[-1] < heads * dim * vdim \
             or tuple(values.shape) != (T, heads * vdim) or values.stride(1) != 1:
-        raise ValueError("retention_scan: qk is contiguous float32 [T, 2 heads dim], values [T, heads vdim], decay float32 [heads], "
+        raise ValueError("retention_scan: qk is float32 [T, 2 heads dim], values [T, heads vdim], decay float32 [heads], "
                          "the state float32 [seats, >= heads dim vdim]")
     out = torch.empty((T, heads * vdim), dtype=torch.float32, device=qk.device)
     if max_q_len >= RETENTION_CHUNKS_FROM:
         # long portions: blocks of tokens summed side by side and chained (three launches) instead of a walk token by token
         block = _core().fe_retention_chunk_tokens()
         sums = torch.empty((T // block + cu_q.numel() - 1, heads * dim * vdim), dtype=torch.float32, device=qk.device)
-        _run(_core(), "fe_retention_chunks", _ptr(qk), _ptr(values), _c_ll(values.stride(0)), _ptr(decay), _ptr(state),
+        _run(_core(), "fe_retention_chunks", _ptr(qk), _c_ll(qk.stride(0)), _ptr(values), _c_ll(values.stride(0)), _ptr(decay), _ptr(state),
              _c_ll(state.stride(0)), _ptr(state_slots), _ptr(cu_q), _ptr(out), _ptr(sums), _c_int(cu_q.numel() - 1), _c_int(max_q_len),
              _c_int(heads), _c_int(dim), _c_int(vdim), _c_int(state.shape[0]), _c_int(_code(values.dtype)), _stream())
         return out
-    _run(_core(), "fe_retention_scan", _ptr(qk), _ptr(values), _c_ll(values.stride(0)), _ptr(decay), _ptr(state), _c_ll(state.stride(0)),
+    _run(_core(), "fe_retention_scan", _ptr(qk), _c_ll(qk.stride(0)), _ptr(values), _c_ll(values.stride(0)), _ptr(decay), _ptr(state), _c_ll(state.stride(0)),
          _ptr(state_slots), _ptr(cu_q), _ptr(out), _c_int(cu_q.numel() - 1), _c_int(heads), _c_int(dim), _c_int(vdim),
          _c_int(state.shape[0]), _c_int(_code(values.dtype)), _stream())
     return out
 
 
 def retention_decode(projected, heads, dim, vdim, positions, inv_freq, rot_dims, key_scale, decay, state, state_slots, eps, out_dtype,
-                     scale=1.0, into=None):
+                     scale=1.0, into=None, activation=None, raw=False):
     """A step of ONE token a request in one kernel (csrc/retention.cu): ``projected`` [R, >= 2 heads dim + 2 heads vdim] =
     q | k | v | g (any row stride); rotation of q and k, the keys times ``key_scale``, S <- decay_h S + k v^T in
     ``state[seat]`` (zeros and nothing kept for a seat below 0), o = S^T q, every head of o divided by its root mean square,
-    times silu(g), times ``scale``.  Returns [R, heads vdim] in ``out_dtype`` (``into`` where given, a view with any row stride)."""
+    times silu(g), times ``scale``.  Returns [R, heads vdim] in ``out_dtype`` (``into`` where given, a view with any row stride).  ``activation`` "silu": q, k and v go through it first (and
+    nothing turns).  ``raw``: o itself comes back, float32 [R, heads vdim], for a norm over all heads."""
+    if activation not in (None, "silu"):
+        raise ValueError(f"unknown activation {activation!r}")
     _need_cuda(projected, positions, inv_freq, decay, state, state_slots, into)
     R = projected.shape[0]
     inner = heads * vdim
@@ -1158,14 +1236,83 @@ def retention_decode(projected, heads, dim, vdim, positions, inv_freq, rot_dims,
                          "[seats, >= heads dim vdim], a seat and a position per row")
     if inv_freq is not None and (inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_dims // 2):
         raise ValueError("inv_freq must be float32 [rot_dims / 2]")
-    y = into if into is not None else torch.empty((R, inner), dtype=out_dtype, device=projected.device)
-    if tuple(y.shape) != (R, inner) or y.dtype != out_dtype or y.stride(1) != 1:
+    sums = torch.empty((R, inner), dtype=torch.float32, device=projected.device) if raw else None
+    y = into if into is not None else sums.view(R, inner) if raw else torch.empty((R, inner), dtype=out_dtype, device=projected.device)
+    if tuple(y.shape) != (R, inner) or (y.dtype != out_dtype and not raw) or y.stride(1) != 1:
         raise ValueError("retention_decode: the rows go to [R, heads vdim] in the compute dtype with unit column stride")
     _run(_core(), "fe_retention_decode", _ptr(projected), _c_ll(projected.stride(0)), _ptr(positions), _ptr(inv_freq),
          _c_int(rot_dims if inv_freq is not None else 0), _c_float(key_scale), _ptr(decay), _ptr(state), _c_ll(state.stride(0)),
          _ptr(state_slots), _ptr(y), _c_ll(y.stride(0)), _c_float(eps), _c_float(scale), _c_int(R), _c_int(heads), _c_int(dim),
-         _c_int(vdim), _c_int(state.shape[0]), _c_int(_code(out_dtype)), _stream())
-    return y
+         _c_int(vdim), _c_int(state.shape[0]), _c_int(1 if activation else 0), _ptr(sums), _c_int(_code(out_dtype)), _stream())
+    return sums if raw else y
+
+
+# ---- the gated delta rule ------------------------------------------------------------------------------------------
+def _check_delta(what, projected, conv, state, history_at, a_log, dt_bias, heads, kv_heads, dim, vdim):
+    taps, C = conv.shape
+    if C != 2 * kv_heads * dim + heads * vdim or projected.dtype != torch.float32 or projected.dim() != 2 or projected.stride(1) != 1 \
+            or projected.shape[1] < C + heads * vdim + 2 * heads or conv.dtype != torch.float32 or not conv.is_contiguous() \
+            or state.dtype != torch.float32 or state.stride(-1) != 1 or state.shape[-1] < history_at + (taps - 1) * C \
+            or history_at < heads * dim * vdim or a_log.dtype != torch.float32 or a_log.numel() != heads or dt_bias.dtype != torch.float32 \
+            or dt_bias.numel() != heads:
+        raise ValueError(f"{what}: projected float32 [T, q | k | v | g | b | a], conv float32 [taps, channels], a float32 state row of the "
+                         "heads' states and the convolutions' history, A_log and dt_bias float32 [heads]")
+
+
+def delta_prepare(projected, conv, state, history_at, state_slots, cu_q, token_request, a_log, dt_bias, unit_eps, query_scale,
+                  heads, kv_heads, dim, vdim, max_q_len=0):
+    """What the gated delta rule does between its projection and its recurrence (csrc/delta.cu).  ``projected`` float32
+    [T, q | k | v | g | b | a].  Convolution over time (``conv`` [taps, channels], tap by tap; the last taps - 1 projected rows of
+    a request lie in state[seat, history_at:] and are brought up to date) and silu of q | k | v, q and k made unit vectors per
+    head, q times ``query_scale``.  Returns (float32 [T, channels], the decays and step sizes in the form ``delta_scan``
+    takes them).  ``max_q_len``: the longest portion of the step (0: as many tokens as the step has)."""
+    _need_cuda(projected, conv, state, state_slots, cu_q, a_log, dt_bias)
+    _check_delta("delta_prepare", projected, conv, state, history_at, a_log, dt_bias, heads, kv_heads, dim, vdim)
+    T, (taps, C), requests = projected.shape[0], conv.shape, cu_q.numel() - 1
+    lib = _core()
+    out = torch.empty((T, C), dtype=torch.float32, device=projected.device)
+    numbers = torch.empty((T // lib.fe_delta_block_tokens() + requests, heads, lib.fe_delta_block_numbers()), dtype=torch.float32,
+                          device=projected.device)
+    _run(lib, "fe_delta_prepare", _ptr(projected), _c_ll(projected.stride(0)), _ptr(conv), _c_int(taps), _ptr(state), _c_ll(state.stride(0)),
+         _c_ll(history_at), _ptr(state_slots), _ptr(cu_q), _ptr(a_log), _ptr(dt_bias), _c_float(unit_eps), _c_float(query_scale), _ptr(out),
+         _ptr(numbers), _c_int(requests), _c_int(max_q_len or T), _c_int(heads), _c_int(kv_heads), _c_int(dim), _c_int(vdim),
+         _c_int(state.shape[0]), _stream())
+    return out, numbers
+
+
+def delta_scan(qkv, gates, state, state_slots, cu_q, heads, kv_heads, dim, vdim, max_q_len=0):
+    """S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q per request and head over the step's tokens; S [dim, vdim]
+    float32 lives in ``state[seat, : heads dim vdim]`` (zeros and nothing kept for a seat below 0).  ``qkv`` and ``gates`` as
+    ``delta_prepare`` returns them; returns float32 [T, heads vdim]."""
+    _need_cuda(qkv, gates, state, state_slots, cu_q)
+    T, requests, lib = qkv.shape[0], cu_q.numel() - 1, _core()
+    if qkv.dtype != torch.float32 or tuple(qkv.shape) != (T, 2 * kv_heads * dim + heads * vdim) or not qkv.is_contiguous() \
+            or gates.dtype != torch.float32 or not gates.is_contiguous() \
+            or gates.numel() < (T // lib.fe_delta_block_tokens() + requests) * heads * lib.fe_delta_block_numbers() \
+            or state.dtype != torch.float32 or state.stride(-1) != 1 or state.shape[-1] < heads * dim * vdim:
+        raise ValueError("delta_scan: qkv and gates as delta_prepare returns them, the state float32 [seats, >= heads dim vdim]")
+    out = torch.empty((T, heads * vdim), dtype=torch.float32, device=qkv.device)
+    _run(lib, "fe_delta_scan", _ptr(qkv), _ptr(gates), _ptr(state), _c_ll(state.stride(0)), _ptr(state_slots), _ptr(cu_q), _ptr(out),
+         _c_int(requests), _c_int(heads), _c_int(kv_heads), _c_int(dim), _c_int(vdim), _c_int(state.shape[0]), _stream())
+    return out
+
+
+def delta_decode(projected, conv, state, history_at, state_slots, a_log, dt_bias, norm_weight, eps, unit_eps, query_scale,
+                 heads, kv_heads, dim, vdim, out_dtype):
+    """A step of ONE token a request, everything between the projection and the output product in one kernel (csrc/delta.cu):
+    ``delta_prepare`` and ``delta_scan``, then every head divided by its root mean square, times ``norm_weight`` (float32
+    [vdim]), times silu of its gate row.  Returns [R, heads vdim] in ``out_dtype``."""
+    _need_cuda(projected, conv, state, state_slots, a_log, dt_bias, norm_weight)
+    _check_delta("delta_decode", projected, conv, state, history_at, a_log, dt_bias, heads, kv_heads, dim, vdim)
+    R, taps = projected.shape[0], conv.shape[0]
+    if norm_weight.dtype != torch.float32 or norm_weight.numel() != vdim or state_slots.numel() < R:
+        raise ValueError("delta_decode: the norm weight is float32 [vdim], a seat per row")
+    out = torch.empty((R, heads * vdim), dtype=out_dtype, device=projected.device)
+    _run(_core(), "fe_delta_decode", _ptr(projected), _c_ll(projected.stride(0)), _ptr(conv), _c_int(taps), _ptr(state),
+         _c_ll(state.stride(0)), _c_ll(history_at), _ptr(state_slots), _ptr(a_log), _ptr(dt_bias), _ptr(norm_weight), _c_float(eps),
+         _c_float(unit_eps), _c_float(query_scale), _ptr(out), _c_int(R), _c_int(heads), _c_int(kv_heads), _c_int(dim), _c_int(vdim),
+         _c_int(state.shape[0]), _c_int(_code(out_dtype)), _stream())
+    return out
 
 
 # ---- attention over a cached latent ------------------------------------------------------------------------------
@@ -1246,7 +1393,7 @@ ROUTED_TCGEN05_MIN_PAIRS = 1024     # fewer sorted rows than this: the mma.sync 
 ROUTED_TCGEN05_MIN_K = 1024          # narrower experts: level or behind (512 x 384: 0.090 against 0.052 ms at 2,048 rows)
 
 
-ROUTED_SINGLE = ("relu2",)            # activations of experts without a gate: one matrix up, one down
+ROUTED_SINGLE = ("relu2", "gelu")     # activations of experts without a gate: one matrix up, one down (the kernels' codes 1, 2)
 
 
 def routed_tcgen05_ok(h, pairs, H, F) -> bool:
@@ -1256,7 +1403,7 @@ def routed_tcgen05_ok(h, pairs, H, F) -> bool:
             and min(H, F) >= ROUTED_TCGEN05_MIN_K and h.data_ptr() % 16 == 0)
 
 
-def _routed_experts_tcgen05(h, chosen, weights, gate_up, down, shared, limit=0.0, single=False, identity=0):
+def _routed_experts_tcgen05(h, chosen, weights, gate_up, down, shared, limit=0.0, single=None, identity=0):
     """The routed feed-forward with its products on tcgen05 tensor cores: plan (counting sort, row tiles of 128 per
     expert), the rows of h gathered into sorted order, gate/up with the activation in the epilogue, down into float32,
     combination.  Everything stays on the device."""
@@ -1279,7 +1426,7 @@ def _routed_experts_tcgen05(h, chosen, weights, gate_up, down, shared, limit=0.0
          _ptr(offsets[experts:]), _stream())
     act = torch.empty((pairs, F), dtype=torch.bfloat16, device=dev)
     _run(tensor, "fe_gemm_tcgen05_grouped", _ptr(rows), _ptr(gate_up), _ptr(act), _c_int(pairs), _c_int(experts), _c_int(F if single else 2 * F),
-         _c_int(H), _c_int(EPI_RELU2 if single else EPI_SWIGLU), _ptr(tiles), _ptr(tile_expert), _ptr(tile_row0), _ptr(offsets), _c_float(limit), _ptr(status), _stream())
+         _c_int(H), _c_int(SINGLE_EPILOGUES[single] if single else EPI_SWIGLU), _ptr(tiles), _ptr(tile_expert), _ptr(tile_row0), _ptr(offsets), _c_float(limit), _ptr(status), _stream())
     y = torch.empty((pairs, H), dtype=torch.float32, device=dev)
     _run(tensor, "fe_gemm_tcgen05_grouped", _ptr(act), _ptr(down), _ptr(y), _c_int(pairs), _c_int(experts), _c_int(H), _c_int(F),
          _c_int(EPI_F32), _ptr(tiles), _ptr(tile_expert), _ptr(tile_row0), _ptr(offsets), _c_float(0.0), _ptr(status), _stream())
@@ -1294,21 +1441,21 @@ def routed_experts(h, chosen, weights, gate_up, down, shared=None, activation="s
     given; gate_up [experts, 2F, H] ([gate; up] per expert), down [experts, H, F].  ``activation`` "clamped": with
     g = min(gate_e h_t, limit) and u = clamp(up_e h_t, -limit, limit) an expert is down_e( g sigmoid(1.702 g) (u + 1) ).
     The (token, choice) pairs are sorted by expert on the device and every expert multiplies its own rows (csrc/routed.cu):
-    nothing comes back to the host.  ``activation`` "relu2": experts without a gate; ``gate_up`` is then [experts, F, H] and
-    an expert is down_e( relu(up_e h_t)^2 ).  ``identity``: choices in [experts, experts + identity) stand for experts that
+    nothing comes back to the host.  ``activation`` "relu2", "gelu": experts without a gate; ``gate_up`` is then [experts, F, H]
+    and an expert is down_e( act(up_e h_t) ), act the square of relu or the exact GELU.  ``identity``: choices in [experts, experts + identity) stand for experts that
     return their input: out[t] += weight * h_t."""
     _need_cuda(h, chosen, weights, gate_up, down, shared)
     T, H = h.shape
     experts, F2, _ = gate_up.shape
-    single = activation in ROUTED_SINGLE
+    single = activation if activation in ROUTED_SINGLE else None
     F, top = (F2 if single else F2 // 2), chosen.shape[1]
     if tuple(gate_up.shape) != (experts, F if single else 2 * F, H) or tuple(down.shape) != (experts, H, F) or gate_up.dtype != h.dtype \
             or down.dtype != h.dtype or not (gate_up.is_contiguous() and down.is_contiguous() and h.is_contiguous()) \
             or chosen.dtype != torch.int32 or weights.dtype != torch.float32 \
             or (shared is not None and (shared.dtype != h.dtype or shared.shape != h.shape or not shared.is_contiguous())):
         raise ValueError("routed_experts: shapes or dtypes do not fit")
-    if activation not in ("silu", "clamped", "relu2") or (activation == "clamped" and not limit > 0.0):
-        raise ValueError("routed_experts: the activation is 'silu', 'relu2' or 'clamped' with a positive limit")
+    if activation not in ("silu", "clamped") + ROUTED_SINGLE or (activation == "clamped" and not limit > 0.0):
+        raise ValueError("routed_experts: the activation is 'silu', 'relu2', 'gelu' or 'clamped' with a positive limit")
     limit = float(limit) if activation == "clamped" else 0.0
     if routed_tcgen05_ok(h, T * top, H, F):
         return _routed_experts_tcgen05(h, chosen, weights, gate_up, down, shared, limit, single, identity)
@@ -1318,7 +1465,7 @@ def routed_experts(h, chosen, weights, gate_up, down, shared=None, activation="s
     out = torch.empty((T, H), dtype=h.dtype, device=h.device)
     _run(lib, "fe_routed_experts", _ptr(h), _ptr(chosen), _ptr(weights), _ptr(gate_up), _ptr(down), _ptr(shared), _ptr(out),
          _ptr(work), _c_ll(need), _c_int(T), _c_int(top), _c_int(experts), _c_int(H), _c_int(F), _c_int(_code(h.dtype)),
-         _c_float(limit), _ptr(status_word(h.device)), _c_int(1 if single else 0), _c_int(identity), _stream())
+         _c_float(limit), _ptr(status_word(h.device)), _c_int(1 + ROUTED_SINGLE.index(single) if single else 0), _c_int(identity), _stream())
     return out
 
 

@@ -81,7 +81,8 @@ class GatedDeltaMixer(Mixer):
                                    self.norm_weight, self.eps, self.unit_eps, self.query_scale, *sizes, ctx.dtype)
             return ops.linear(out, self.o_weight)
         qkv, gates = ops.delta_prepare(projected, self._conv_by_tap, state, self.matrix_elements, ctx.state_slots, ctx.cu_q,
-                                       ctx.token_request, self.A_log, self.dt_bias, self.unit_eps, self.query_scale, *sizes)
+                                       ctx.token_request, self.A_log, self.dt_bias, self.unit_eps, self.query_scale, *sizes,
+                                       max_q_len=ctx.max_q_len)
         o = ops.delta_scan(qkv, gates, state, ctx.state_slots, ctx.cu_q, *sizes, max_q_len=ctx.max_q_len)
         g = projected[:, self.channels:self.channels + self.inner_width]
         out = ops.head_rmsnorm_gate(o, self._head_weight, g, self.eps, self.heads, ctx.dtype)

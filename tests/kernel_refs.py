@@ -468,7 +468,7 @@ def retention_decode(projected, heads, dim, vdim, positions, inv_freq, rot_dims,
 
 # ---- the gated delta rule ------------------------------------------------------------------------------
 def delta_prepare(projected, conv, state, history_at, state_slots, cu_q, token_request, a_log, dt_bias, unit_eps, query_scale,
-                  heads, kv_heads, dim, vdim):
+                  heads, kv_heads, dim, vdim, max_q_len=0):
     """projected float32 [T, q | k | v | g | b | a].  Convolution (``conv`` [taps, channels]; the last taps - 1 rows of a request
     in state[seat, history_at:], brought up to date) and silu of q | k | v, q and k unit vectors per head, q times
     ``query_scale``: float32 [T, channels]; and float32 [T, 2 heads]: the decays, then the step sizes."""
