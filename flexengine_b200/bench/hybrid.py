@@ -1,7 +1,9 @@
-"""``--workload fuvozen|fuvuvik|fedutar|rikolix``: prefill and decode throughput of one of these designs at a few sizes that resemble a
+"""``--workload fuvozen|fuvuvik|fedutar|rikolix|bebulorn``: prefill and decode throughput of one of these designs at a few sizes that resemble a
 real model's layers (random weights), beside the closest existing model at equal width, depth and vocabulary (a Qwen2
 decoder; for Fedutar the Fuvozen design, which also has a recurrence with a matrix state and routed experts; for Rikolix the
-Fuvozen design too, which also has attention over a cached latent, routed experts and a dense feed-forward without a gate), and, at one size, an
+Fuvozen design too, which also has attention over a cached latent, routed experts and a dense feed-forward without a gate; for
+Bebulorn the Fedutar design, which also has norms on both sides of a sublayer, linear attention with a state matrix, routed experts
+and a repeated span), and, at one size, an
 operation-by-operation table of both: time, the bytes and flops of the work, and how far each operation is from the
 roofline of the measured peaks (time / max(bytes / copy rate, flops / bf16 rate)).
 
@@ -103,8 +105,34 @@ def rikolix_config(width, layers, vocab, heads):
     return {"architecture": "Rikolix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "layers": stack}
 
 
+def bebulorn_config(width, layers, vocab, heads):
+    """``layers`` runs of a layer: the first two layers run twice in a row, the others once.  Layers in turns of three: softmax
+    attention under a window of 1,024 (heads of 128 in groups of four, squashed scores), the gated delta rule (width / 128 value
+    heads of 128 over half as many query/key heads of 128, four taps), lightning attention (width / 128 heads of 64 key x 128
+    value channels, as the retention of the Fedutar model beside it); feed-forwards in turns: dense of 2.5 x width, then 8
+    experts without a gate of 1.25 x width of which a token uses 2, beside a shared one of the same size."""
+    distinct = max(3, layers - 2)
+    r_heads = max(1, width // 128)
+    stack = []
+    for i in range(distinct):
+        turn = i % 3
+        if turn == 0:
+            mixer = {"type": "attention", "mixer": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "mask": {"size": 1024},
+                                                    "scale": 128 ** -0.5, "softcap": 30.0}}
+        elif turn == 1:
+            mixer = {"type": "delta", "mixer": {"heads": r_heads, "kv_heads": max(1, r_heads // 2), "dim": 128, "vdim": 128, "conv": 4}}
+        else:
+            mixer = {"type": "lightning", "mixer": {"heads": r_heads, "dim": 64, "vdim": 128,
+                                                    "decay": [1.0 - 2.0 ** -(5 + h % 6) for h in range(r_heads)]}}
+        mlp = {"kind": "dense", "ff": width * 5 // 2} if i % 2 == 0 else \
+            {"kind": "moe", "expert": {"ff": width * 5 // 4}, "router": {"experts": 8, "top": 2}, "shared": {"ff": width * 5 // 4}}
+        stack.append(dict(mixer, mlp=mlp))
+    return {"architecture": "Bebulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "loop": {"start": 0, "stop": 2, "times": 2 if layers > distinct else 1}, "layers": stack}
+
+
 DESIGNS = {"fuvozen": ("Fuvozen", fuvozen_config), "fuvuvik": ("Fuvuvik", fuvuvik_config), "fedutar": ("Fedutar", fedutar_config),
-           "rikolix": ("Rikolix", rikolix_config)}
+           "rikolix": ("Rikolix", rikolix_config), "bebulorn": ("Bebulorn", bebulorn_config)}
 
 
 def qwen2_config(width, layers, vocab, heads):
@@ -117,7 +145,8 @@ def qwen2_config(width, layers, vocab, heads):
 
 
 # the model a design is measured beside (default: the Qwen2 decoder)
-BESIDE = {"fedutar": ("fuvozen", "Fuvozen", fuvozen_config), "rikolix": ("fuvozen", "Fuvozen", fuvozen_config)}
+BESIDE = {"fedutar": ("fuvozen", "Fuvozen", fuvozen_config), "rikolix": ("fuvozen", "Fuvozen", fuvozen_config),
+          "bebulorn": ("fedutar", "Fedutar", fedutar_config)}
 
 SIZES = {"1k": (1024, 8, 32000, 8), "2k": (2048, 8, 32000, 16), "4k": (4096, 4, 32000, 32)}
 
@@ -146,6 +175,8 @@ class TimedOps:
             end.record()
             torch.cuda.synchronize()
             tensors = [a for a in list(args) + list(kwargs.values()) if torch.is_tensor(a)]
+            post = kwargs.get("post")
+            tensors += [a for a in (post or ()) if torch.is_tensor(a)]
             tensors += [o for o in (out if isinstance(out, (tuple, list)) else [out]) if torch.is_tensor(o)]
             seen, nbytes = set(), 0
             for t in tensors:
@@ -159,7 +190,7 @@ class TimedOps:
                 flops = 2.0 * args[0].shape[0] * args[0].shape[1] * args[0].shape[2] * args[1].shape[1]
             elif name == "routed_experts":
                 pairs = args[1].numel()
-                if kwargs.get("activation") == "relu2":           # experts without a gate: one matrix up, one down
+                if kwargs.get("activation") in ("relu2", "gelu"):           # experts without a gate: one matrix up, one down
                     flops = 2.0 * pairs * 2 * args[3].shape[1] * args[3].shape[2]
                 else:
                     flops = 2.0 * pairs * 3 * (args[3].shape[1] // 2) * args[3].shape[2]
@@ -189,6 +220,30 @@ class TimedOps:
                 tokens, requests = args[0].shape[0], args[5].numel() - 1
                 flops = 4.0 * tokens * heads * d * dv
                 nbytes = tokens * (2 * heads * d * 4 + heads * dv * (args[1].element_size() + 4)) + 2 * 4 * requests * heads * d * dv
+            elif name == "retention_decode":
+                # one token a request: its row of the projection, the state read and written, the heads' rows
+                heads, d, dv = args[1], args[2], args[3]
+                rows = args[0].shape[0]
+                flops = 4.0 * rows * heads * d * dv
+                nbytes = rows * (args[0].shape[1] * args[0].element_size() + heads * dv * out.element_size() + 2 * 4 * heads * d * dv)
+            elif name in ("delta_scan", "delta_prepare", "delta_decode"):
+                # the recurrence: two products with the state and its update a token; a request's state read and written once
+                heads, kv, d, dv = args[5:9] if name == "delta_scan" else args[11:15]
+                tokens = args[0].shape[0]
+                C = 2 * kv * d + heads * dv
+                states = 2 * 4 * heads * d * dv * (tokens if name == "delta_decode" else args[4].numel() - 1)
+                if name == "delta_scan":
+                    flops, nbytes = 6.0 * tokens * heads * d * dv, tokens * 4 * (C + 2 * heads + heads * dv) + states
+                elif name == "delta_prepare":
+                    nbytes = tokens * 4 * (2 * C + 4 * heads)
+                else:
+                    flops, nbytes = 6.0 * tokens * heads * d * dv, tokens * (args[0].shape[1] * 4 + heads * dv * out.element_size()) + states
+            elif name == "qkv_conv_rope_norm_cache":
+                # the projection's rows read, keys and values into the cache, queries out (not where they stay in place)
+                heads, kv, d, dv, head = args[15:20]
+                tokens, width = args[0].shape[0], args[0].element_size()
+                same = out.data_ptr() == args[0].data_ptr()
+                nbytes = tokens * width * (((0 if same else heads) + kv) * d + kv * dv + ((0 if same else heads) + 2 * kv) * head)
             elif name == "stream_rmsnorm":
                 # the streams are read, and written back when a sublayer's output goes in; its output and gate are read
                 update = kwargs.get("update")
@@ -303,8 +358,8 @@ def run(args) -> int:
     if args.kernels:
         width, layers, vocab, heads = SIZES[sizes[-1] if getattr(args, "size", None) else "2k"]
         # as many layers as show every kind of layer the design has
-        tables[key] = measure(design_config(width, 2 if key == "fuvozen" else 4, vocab, heads), vocab, TimedOps(ops, torch))
-        tables[other] = measure(other_config(width, 2, vocab, heads), vocab, TimedOps(ops, torch))
+        tables[key] = measure(design_config(width, {"fuvozen": 2, "bebulorn": 8}.get(key, 4), vocab, heads), vocab, TimedOps(ops, torch))
+        tables[other] = measure(other_config(width, 4 if other == "fedutar" else 2, vocab, heads), vocab, TimedOps(ops, torch))
     sampler.stop()
     first = results[sizes[0]][key]
     line = {"metric": f"decode tokens/s ({design} design, size {sizes[0]}, batch {BATCH}, {PROMPT}-token prompts)",
