@@ -651,12 +651,68 @@ __global__ void qkv_conv_rope_norm_cache_kernel(const T* __restrict__ proj, long
     }
 }
 
+// Keys as they are and values, divided by their root mean square with v_norm, into their cache slots: what is left of the preparation
+// where nothing else is asked for.  A warp per (token, head of keys or values), eight entries a lane and round; rows start on
+// 16-byte boundaries.
+constexpr int KV_ROUNDS = 4;
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+kv_cache_kernel(const T* __restrict__ proj, long long ld, int first, const int* __restrict__ slot_mapping, T* __restrict__ kc, T* __restrict__ vc,
+                int T_tokens, int kv_heads, int dim, int vdim, int head, int ps, long long num_slots, float eps, int v_norm,
+                int* __restrict__ status) {
+    griddep_wait();
+    griddep_launch_dependents();
+    const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (item >= (long long)T_tokens * 2 * kv_heads) return;
+    const int lane = threadIdx.x & 31;
+    const int t = (int)(item / (2 * kv_heads)), hs = (int)(item % (2 * kv_heads));
+    const bool value = hs >= kv_heads;
+    const int index = value ? hs - kv_heads : hs, hd = value ? vdim : dim;
+    const int slot = slot_mapping[t];
+    const T* src = proj + (size_t)t * ld + first + (value ? kv_heads * dim + index * vdim : index * dim);
+    float v[KV_ROUNDS][8], ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < KV_ROUNDS; ++k) {
+        const int c = (k * 32 + lane) * 8;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[k][e] = 0.f;
+        if (c < hd) load8<T>(src + c, v[k]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss = fmaf(v[k][e], v[k][e], ss);
+    }
+    if (slot < 0) return;
+    if (slot >= num_slots) {
+        if (lane == 0 && status) atomicOr(status, FE_STATUS_BAD_SLOT);
+        return;
+    }
+    const float inv = value && v_norm ? rsqrtf(warp_sum(ss) / (float)hd + eps) : 1.f;
+    const long long page = slot / ps, off = slot % ps;
+    T* dst = (value ? vc : kc) + ((page * kv_heads + index) * ps + off) * head;
+#pragma unroll
+    for (int k = 0; k < KV_ROUNDS; ++k) {
+        const int c = (k * 32 + lane) * 8;
+        if (c >= head) continue;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[k][e] *= inv;               // beyond the head's own size they are zeros
+        store8<T>(dst + c, v[k]);
+    }
+}
+
 template <typename T>
 static int launch_qkv_prepare(const void* proj, long long ld, const float* conv, float* history, long long history_stride, int taps,
                               const int* seats, const int* cu_q, const int* token_req, const int* positions, const float* inv_freq, int rot,
                               int qk_norm, float eps, const int* slot_mapping, void* kc, void* vc, void* q_out, int T_tokens, int heads,
                               int kv_heads, int dim, int vdim, int head, int ps, long long num_slots, int n_seats, int* status,
                               const float* q_weight, const float* k_weight, float temp_coef, int temp_every, int v_norm, cudaStream_t stream) {
+    if (!q_out && !conv && !(inv_freq && rot > 0) && !qk_norm && !k_weight && dim % 8 == 0 && vdim % 8 == 0 && head % 8 == 0 && ld % 8 == 0 &&
+        head <= KV_ROUNDS * 256 && (((size_t)proj | (size_t)kc | (size_t)vc) & 15) == 0) {
+        if (!slot_mapping) return 0;
+        const long long items = (long long)T_tokens * 2 * kv_heads;
+        fe::launch(kv_cache_kernel<T>, (unsigned)((items + 7) / 8), 256, 0, stream, (const T*)proj, ld, heads * dim, slot_mapping, (T*)kc, (T*)vc,
+                   T_tokens, kv_heads, dim, vdim, head, ps, num_slots, eps, v_norm, status);
+        return fe_check_launch("kv_cache");
+    }
     const int per_token = (q_out ? heads : 0) + 2 * kv_heads;
     // up to 16 warps share out the token's heads evenly: 24 heads are two rounds of 12 warps
     const int rounds = (per_token + 15) / 16;
