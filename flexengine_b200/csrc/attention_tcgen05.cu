@@ -274,16 +274,18 @@ __device__ __forceinline__ void row_map(unsigned* r, float unit, float cap_log2)
             m0 = max3(m0, fabsf(__uint_as_float(r[i])), fabsf(__uint_as_float(r[i + 1])));
             m1 = max3(m1, fabsf(__uint_as_float(r[i + 2])), fabsf(__uint_as_float(r[i + 3])));
         }
-        if (__all_sync(0xffffffffu, fmaxf(m0, m1) * fabsf(to_z) <= 0.6f)) {
-            const float2 z2 = make_float2(to_z, to_z), cap2 = make_float2(cap_log2, cap_log2);
-            const float2 c4 = make_float2(0.015486690f, 0.015486690f), c3 = make_float2(-0.052109625f, -0.052109625f),
-                         c2 = make_float2(0.13310358f, 0.13310358f), c1 = make_float2(-0.33332323f, -0.33332323f), c0 = make_float2(0.99999993f, 0.99999993f);
+        // the powers of to_z and the cap are folded into the coefficients (a factor so small that they would vanish takes the other way)
+        if (__all_sync(0xffffffffu, fmaxf(m0, m1) * fabsf(to_z) <= 0.6f && fabsf(to_z) > 1e-4f)) {
+            const float zz = to_z * to_z, k0 = to_z * cap_log2, k1 = k0 * zz, k2 = k1 * zz, k3 = k2 * zz, k4 = k3 * zz;
+            const float2 c4 = make_float2(0.015486690f * k4, 0.015486690f * k4), c3 = make_float2(-0.052109625f * k3, -0.052109625f * k3),
+                         c2 = make_float2(0.13310358f * k2, 0.13310358f * k2), c1 = make_float2(-0.33332323f * k1, -0.33332323f * k1),
+                         c0 = make_float2(0.99999993f * k0, 0.99999993f * k0);
 #pragma unroll
             for (int i = 0; i < KEYS; i += 2) {
-                const float2 z = __fmul2_rn(make_float2(__uint_as_float(r[i]), __uint_as_float(r[i + 1])), z2);
-                const float2 w = __fmul2_rn(z, z);
+                const float2 s = make_float2(__uint_as_float(r[i]), __uint_as_float(r[i + 1]));
+                const float2 w = __fmul2_rn(s, s);
                 const float2 p = __ffma2_rn(__ffma2_rn(__ffma2_rn(__ffma2_rn(c4, w, c3), w, c2), w, c1), w, c0);
-                const float2 t = __fmul2_rn(__fmul2_rn(z, cap2), p);
+                const float2 t = __fmul2_rn(s, p);
                 r[i] = __float_as_uint(t.x), r[i + 1] = __float_as_uint(t.y);
             }
             return;
