@@ -243,7 +243,7 @@ __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) { return __
 __device__ __forceinline__ float2 both(float x) { return make_float2(x, x); }
 
 template <int NX, bool VEC>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(128)
 delta_scan_kernel(const float* __restrict__ qkv, const float* __restrict__ coefs, float* state, long long state_stride,
                   const int* __restrict__ seats, const int* __restrict__ cu_q, float* __restrict__ out, int heads, int kv_heads, int d,
                   int dv, int n_seats) {
@@ -468,16 +468,9 @@ delta_scan_kernel(const float* __restrict__ qkv, const float* __restrict__ coefs
 template <int NX, bool VEC>
 int launch_scan(const float* qkv, const float* coefs, float* state, long long state_stride, const int* seats, const int* cu_q, float* out,
                 int requests, int heads, int kv_heads, int d, int dv, int n_seats, cudaStream_t stream) {
-    // a head's value channels are cut into slices until the blocks about fill the device; a block keeps four warps, since every
-    // block copies the queries and keys of all key channels for itself
-    const long long units = (long long)requests * heads;
-    const int head_warps = (dv + 3) / 4;
-    const int most = (head_warps + 3) / 4;
-    int slices = (int)((fe_sm_count() + units - 1) / units);
-    slices = slices < 1 ? 1 : (slices > most ? most : slices);
-    int warps = (head_warps + slices - 1) / slices;
-    if (warps > 8) warps = 8;
-    slices = (head_warps + warps - 1) / warps;
+    // Blocks of four warps, sixteen value channels: two of them fit a multiprocessor, so that up to two warps a scheduler hide one
+    // another's waits; fewer warps a block would copy the queries and keys of all key channels more often than that is worth.
+    const int head_warps = (dv + 3) / 4, warps = head_warps < 4 ? head_warps : 4, slices = (head_warps + warps - 1) / warps;
     const size_t smem = 2 * ((size_t)SCAN_TILE * (2 * 64 * NX + warps * 4) + SCAN_BLOCKS * COEFS) * sizeof(float);
     if (smem > 48 * 1024) {
         const cudaError_t err = cudaFuncSetAttribute(delta_scan_kernel<NX, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
