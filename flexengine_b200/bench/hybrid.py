@@ -106,9 +106,9 @@ def rikolix_config(width, layers, vocab, heads):
 
 
 def bebulorn_config(width, layers, vocab, heads):
-    """``layers`` runs of a layer: the first two layers run twice in a row, the others once.  Layers in turns of three: softmax
-    attention under a window of 1,024 (heads of 128 in groups of four, squashed scores), the gated delta rule (width / 128 value
-    heads of 128 over half as many query/key heads of 128, four taps), lightning attention (width / 128 heads of 64 key x 128
+    """``layers`` runs of a layer: the first layers run twice in a row (two of six, one of three), the others once.  Layers in
+    turns of three: softmax attention under a window of 1,024 (heads of 128 in groups of four, squashed scores), the gated
+    delta rule (width / 128 value heads of 128 over half as many query/key heads of 128, four taps), lightning attention (width / 128 heads of 64 key x 128
     value channels, as the retention of the Fedutar model beside it); feed-forwards in turns: dense of 2.5 x width, then 8
     experts without a gate of 1.25 x width of which a token uses 2, beside a shared one of the same size."""
     distinct = max(3, layers - 2)
@@ -128,7 +128,7 @@ def bebulorn_config(width, layers, vocab, heads):
             {"kind": "moe", "expert": {"ff": width * 5 // 4}, "router": {"experts": 8, "top": 2}, "shared": {"ff": width * 5 // 4}}
         stack.append(dict(mixer, mlp=mlp))
     return {"architecture": "Bebulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
-            "loop": {"start": 0, "stop": 2, "times": 2 if layers > distinct else 1}, "layers": stack}
+            "loop": {"start": 0, "stop": max(1, layers - distinct), "times": 2 if layers > distinct else 1}, "layers": stack}
 
 
 DESIGNS = {"fuvozen": ("Fuvozen", fuvozen_config), "fuvuvik": ("Fuvuvik", fuvuvik_config), "fedutar": ("Fedutar", fedutar_config),
