@@ -204,7 +204,8 @@ class CacheManager:
                 # the next query sits at position >= rc.tokens and sees keys t > position - w
                 first_needed = rc.tokens - w + 1
             table = rc.tables[gi]
-            for j in range(min(len(table), max(0, first_needed) // g.page_size)):
+            kept = -(-getattr(g.spec, "keep", 0) // g.page_size)          # pages of the first keys, which stay visible
+            for j in range(kept, min(len(table), max(0, first_needed) // g.page_size)):
                 if table[j] != RELEASED:
                     g.pool.release(table[j])
                     table[j] = RELEASED

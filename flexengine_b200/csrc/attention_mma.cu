@@ -3,7 +3,7 @@
 //
 // Math as the reference's block-wise path (inference/attention/paged.py:50-70): running maximum,
 // running sum and value accumulator in float; key t is visible to the query at position p iff
-// t <= p (and t > p - window when window > 0; t in the chunk of -window positions that holds p when window < 0); query
+// t <= p (and t > p - window, or t < keep, when window > 0; t in the chunk of -window positions that holds p when window < 0); query
 // head h reads key/value head h / (nq / nkv).  ``sink``: the softmax starts as if a key of score 0 and value 0 had been
 // seen (running maximum 0, running sum 1), which adds 1 to its denominator; of the blocks and warps that share a row's
 // keys, the first one does.  ``mode`` carries the sink in bit 0; bit 1 asks for sigmoid weights instead of a softmax: a
@@ -87,10 +87,10 @@ struct KvSource {
     int nkv, kvh, d, ps, ps_shift, num_pages;     // ps_shift: log2(ps) when ps is a power of two, else -1
 };
 
-// Element offset of key ``key``'s row in the cache, or -1 for a key outside [lo, hi] (or whose
+// Element offset of key ``key``'s row in the cache, or -1 for a key outside [lo, hi] and [0, keep) (or whose
 // page id is out of range, which also sets the status word).
-__device__ __forceinline__ long long row_offset(const KvSource& src, int key, int lo, int hi, int* status) {
-    if (key < lo || key > hi) return -1;
+__device__ __forceinline__ long long row_offset(const KvSource& src, int key, int lo, int hi, int keep, int* status) {
+    if ((key < lo && key >= keep) || key > hi) return -1;
     const int page = src.table[src.ps_shift >= 0 ? key >> src.ps_shift : key / src.ps];
     if (page < 0 || page >= src.num_pages) {
         if (status) atomicOr(status, FE_STATUS_BAD_PAGE);
@@ -136,7 +136,7 @@ __device__ __forceinline__ float score_map_unit(float scale_log2, float cap_log2
 template <int DMAX, bool UPPER, int KEYS = TK>
 __device__ __forceinline__ void compute_tile(const bf16* ks, const bf16* vs, const unsigned (*qfrag)[4],
                                              float (*o)[4], float* m, float* l, int first_key, int d,
-                                             float scale_log2, int pos0, int pos1, int lo0, int lo1, bool masked,
+                                             float scale_log2, int pos0, int pos1, int lo0, int lo1, int keep, bool masked,
                                              bool sigmoid = false, float bias0 = 0.f, float bias1 = 0.f,
                                              bool mapped = false, float cap_log2 = 0.f) {
     const int lane = threadIdx.x & 31, t = lane & 3;
@@ -177,7 +177,7 @@ __device__ __forceinline__ void compute_tile(const bf16* ks, const bf16* vs, con
 #pragma unroll
             for (int e = 0; e < (UPPER ? 4 : 2); ++e) {
                 const int key = first_key + j * 8 + 2 * t + (e & 1);
-                const bool vis = e < 2 ? (key <= pos0 && key >= lo0) : (key <= pos1 && key >= lo1);
+                const bool vis = e < 2 ? (key <= pos0 && (key >= lo0 || key < keep)) : (key <= pos1 && (key >= lo1 || key < keep));
                 if (!vis) s[j][e] = -CUDART_INF_F;
             }
         }
@@ -305,7 +305,7 @@ paged_decode_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __rest
                     float* __restrict__ part_o, float* __restrict__ part_lse, const bf16* __restrict__ kc,
                     const bf16* __restrict__ vc, const int* __restrict__ block_table, int bt_stride,
                     const int* __restrict__ cu_q, const int* __restrict__ q_start, int nq, int nkv, int d, int ps,
-                    int num_pages, float scale_log2, int window, int mode, int* __restrict__ status,
+                    int num_pages, float scale_log2, int window, int keep, int mode, int* __restrict__ status,
                     const float* __restrict__ per_head, float cap_log2) {
     griddep_wait();
     griddep_launch_dependents();
@@ -322,9 +322,10 @@ paged_decode_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __rest
     const int tok = cu_q[b];
     const int pos = q_start[b];
     const int lo = first_visible(pos, window);
-    const int tile_lo = lo / TK, tile_hi = pos / TK;
-    const int per = (tile_hi - tile_lo + 1 + splits - 1) / splits;
-    const int t_begin = tile_lo + split * per, t_end = min(tile_hi + 1, t_begin + per);
+    // tiles are counted along the list of those walked: tiles of kept keys first, then the window's
+    const int kept = kept_tiles<TK>(lo, keep), all_tiles = kept + pos / TK - lo / TK + 1;
+    const int per = (all_tiles + splits - 1) / splits;
+    const int t_begin = split * per, t_end = min(all_tiles, t_begin + per);
     const int n_tiles = max(0, t_end - t_begin);
 
     KvSource src{kc, vc, block_table + (size_t)b * bt_stride, nkv, kvh, d, ps, (ps & (ps - 1)) == 0 ? __ffs(ps) - 1 : -1,
@@ -337,7 +338,7 @@ paged_decode_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __rest
     // all the first tiles' keys are looked up at once (one trip to the block table, not one per tile)
     if (threadIdx.x < AHEAD * TK) {
         const int a = threadIdx.x / TK, k = threadIdx.x - a * TK;
-        first_offs[a][k] = a < n_tiles ? row_offset(src, (t_begin + a) * TK + k, lo, pos, status) : -1;
+        first_offs[a][k] = a < n_tiles ? row_offset(src, listed_tile<TK>(t_begin + a, kept, lo) * TK + k, lo, pos, keep, status) : -1;
     }
     __syncthreads();
 #pragma unroll
@@ -380,7 +381,7 @@ paged_decode_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __rest
         // the stage of tile it - 1 is free (both warps finished it): tile it + AHEAD goes there
         long long next = -1;
         const bool more = it + AHEAD < n_tiles;
-        if (more && threadIdx.x < TK) next = row_offset(src, (t_begin + it + AHEAD) * TK + threadIdx.x, lo, pos, status);
+        if (more && threadIdx.x < TK) next = row_offset(src, listed_tile<TK>(t_begin + it + AHEAD, kept, lo) * TK + threadIdx.x, lo, pos, keep, status);
         cp_async_wait<AHEAD - 1>();                  // this thread's part of tile ``it`` has landed
         __syncthreads();                             // ... and everyone else's; the offsets of the last copy have been read
         if (more) {
@@ -391,9 +392,9 @@ paged_decode_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __rest
         }
         cp_async_commit();
         const bf16* sp = smem + (it % STAGES) * 2 * TILE + warp * DECODE_KEYS * pitch<DMAX>();
-        const int first = (t_begin + it) * TK + warp * DECODE_KEYS;
-        compute_tile<DMAX, UPPER, DECODE_KEYS>(sp, sp + TILE, qfrag, o, m, l, first, d, scale_log2, pos, pos, lo, lo,
-                                               first + DECODE_KEYS - 1 > pos || first < lo, sigmoid, bias0, bias1, mapped, cap_log2);
+        const int first = listed_tile<TK>(t_begin + it, kept, lo) * TK + warp * DECODE_KEYS;
+        compute_tile<DMAX, UPPER, DECODE_KEYS>(sp, sp + TILE, qfrag, o, m, l, first, d, scale_log2, pos, pos, lo, lo, keep,
+                                               first + DECODE_KEYS - 1 > pos || (first < lo && first + DECODE_KEYS > keep), sigmoid, bias0, bias1, mapped, cap_log2);
     }
     cp_async_wait<0>();
 #pragma unroll
@@ -591,7 +592,7 @@ __global__ void __launch_bounds__(PREFILL_WARPS * 32)
 paged_prefill_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __restrict__ out, long long out_stride,
                      const bf16* __restrict__ kc, const bf16* __restrict__ vc, const int* __restrict__ block_table,
                      int bt_stride, const int* __restrict__ cu_q, const int* __restrict__ q_start, int nq, int nkv,
-                     int d, int ps, int num_pages, float scale_log2, int window, int mode, int* __restrict__ status,
+                     int d, int ps, int num_pages, float scale_log2, int window, int keep, int mode, int* __restrict__ status,
                      const float* __restrict__ per_head, float cap_log2) {
     griddep_wait();
     griddep_launch_dependents();
@@ -620,13 +621,13 @@ paged_prefill_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __res
     const int qi_first = m_block / G, qi_last = min(n_q - 1, (m_block + PREFILL_ROWS - 1) / G);
     const int hi = start + qi_last;
     const int lo = first_visible(start + qi_first, window);
-    const int s_begin = lo / PREFILL_KEYS, n_stages = hi / PREFILL_KEYS - s_begin + 1;
+    const int kept = kept_tiles<PREFILL_KEYS>(lo, keep), n_stages = kept + hi / PREFILL_KEYS - lo / PREFILL_KEYS + 1;
     KvSource src{kc, vc, block_table + (size_t)r * bt_stride, nkv, kvh, d, ps, (ps & (ps - 1)) == 0 ? __ffs(ps) - 1 : -1,
                  num_pages};
     // threads 0 .. 63 look up one key each of the stage after next; all threads copy
     if (threadIdx.x < PREFILL_KEYS) {
-        offs[0][threadIdx.x] = row_offset(src, s_begin * PREFILL_KEYS + threadIdx.x, lo, hi, status);
-        offs[1][threadIdx.x] = n_stages > 1 ? row_offset(src, (s_begin + 1) * PREFILL_KEYS + threadIdx.x, lo, hi, status) : -1;
+        offs[0][threadIdx.x] = row_offset(src, listed_tile<PREFILL_KEYS>(0, kept, lo) * PREFILL_KEYS + threadIdx.x, lo, hi, keep, status);
+        offs[1][threadIdx.x] = n_stages > 1 ? row_offset(src, listed_tile<PREFILL_KEYS>(1, kept, lo) * PREFILL_KEYS + threadIdx.x, lo, hi, keep, status) : -1;
     }
     __syncthreads();
     copy_rows<DMAX, THREADS, PREFILL_KEYS>(smem, smem + STAGE, src, offs[0]);
@@ -669,18 +670,18 @@ paged_prefill_kernel(const bf16* __restrict__ q, long long q_stride, bf16* __res
         const bf16* st = smem + (it & 1) * 2 * STAGE;
 #pragma unroll
         for (int sub = 0; sub < PREFILL_KEYS / TK; ++sub) {
-            const int first = (s_begin + it) * PREFILL_KEYS + sub * TK;
-            if (w_any && first <= w_pos_max && first + TK - 1 >= w_lo_min) {
+            const int first = listed_tile<PREFILL_KEYS>(it, kept, lo) * PREFILL_KEYS + sub * TK;
+            if (w_any && first <= w_pos_max && (first + TK - 1 >= w_lo_min || first < keep)) {
                 // rows differ in what they see only near the diagonal and the window edge
-                const bool masked = first + TK - 1 > w_pos_min || first < w_lo_max || !(v0 && v1);
+                const bool masked = first + TK - 1 > w_pos_min || (first < w_lo_max && first + TK > keep) || !(v0 && v1);
                 compute_tile<DMAX, true>(st + sub * TK * pitch<DMAX>(), st + STAGE + sub * TK * pitch<DMAX>(), qfrag, o, m,
-                                         l, first, d, scale_log2, pos0, pos1, lo0, lo1, masked, sigmoid, bias0, bias1, mapped, cap_log2);
+                                         l, first, d, scale_log2, pos0, pos1, lo0, lo1, keep, masked, sigmoid, bias0, bias1, mapped, cap_log2);
             }
         }
         // offsets of stage it + 2 go where those of stage ``it`` were: all copies of stage ``it``'s
         // offsets were issued before the barrier above, and the next barrier publishes the new ones
         if (it + 2 < n_stages && threadIdx.x < PREFILL_KEYS)
-            offs[it & 1][threadIdx.x] = row_offset(src, (s_begin + it + 2) * PREFILL_KEYS + threadIdx.x, lo, hi, status);
+            offs[it & 1][threadIdx.x] = row_offset(src, listed_tile<PREFILL_KEYS>(it + 2, kept, lo) * PREFILL_KEYS + threadIdx.x, lo, hi, keep, status);
     }
     cp_async_wait<0>();
 #pragma unroll
@@ -719,8 +720,9 @@ template <typename K> int allow_smem(K kernel, size_t bytes, const char* what) {
     return 0;
 }
 
-int check_common(const char* what, int nq, int nkv, int d, int ps, int num_pages, int window, long long q_stride,
+int check_common(const char* what, int nq, int nkv, int d, int ps, int num_pages, int window, int keep, long long q_stride,
                  long long out_stride) {
+    FE_REQUIRE(keep >= 0 && (keep == 0 || window > 0), "%s: kept first keys go with a window", what);
     FE_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "%s: bad head counts %d/%d", what, nq, nkv);
     FE_REQUIRE(d >= 16 && d <= 256 && d % 16 == 0, "%s: head size %d is not a multiple of 16 in [16, 256]", what, d);
     FE_REQUIRE(ps > 0 && num_pages > 0, "%s: bad page size or page count", what);
@@ -745,9 +747,9 @@ extern "C" long long fe_paged_decode_scratch_bytes(int requests, int nq, int d, 
 extern "C" int fe_paged_decode_mma_upcoming(const void* q, long long q_stride, void* out, long long out_stride, void* scratch,
                                             const void* kc, const void* vc, const int* block_table, int bt_stride,
                                             const int* cu_q, const int* q_start, int requests, int nq, int nkv, int d, int ps,
-                                            int num_pages, float scale, int window, int sink, int splits, const void* upcoming,
+                                            int num_pages, float scale, int window, int keep, int sink, int splits, const void* upcoming,
                                             long long upcoming_bytes, int* status, const float* per_head, float softcap, cudaStream_t stream) {
-    if (check_common("paged_decode", nq, nkv, d, ps, num_pages, window, q_stride, out_stride)) return 1;
+    if (check_common("paged_decode", nq, nkv, d, ps, num_pages, window, keep, q_stride, out_stride)) return 1;
     FE_REQUIRE(nq / nkv <= 16, "paged_decode: %d query heads per key/value head; this kernel takes up to 16", nq / nkv);
     FE_REQUIRE(splits >= 1 && splits <= MAX_SPLITS_SHARED && requests >= 0,
                "paged_decode: %d splits; this kernel takes 1 to %d", splits, MAX_SPLITS_SHARED);
@@ -762,7 +764,7 @@ extern "C" int fe_paged_decode_mma_upcoming(const void* q, long long q_stride, v
         if (allow_smem(paged_decode_kernel<DMAX, UPPER>, decode_smem<DMAX>(), "paged_decode")) return 1;          \
         fe::launch(paged_decode_kernel<DMAX, UPPER>, grid, DECODE_WARPS * 32, decode_smem<DMAX>(), stream,                               \
             (const bf16*)q, q_stride, (bf16*)out, out_stride, part_o, part_lse, (const bf16*)kc, (const bf16*)vc, \
-            block_table, bt_stride, cu_q, q_start, nq, nkv, d, ps, num_pages, scale_log2, window, sink, status, per_head, softcap * LOG2E);  \
+            block_table, bt_stride, cu_q, q_start, nq, nkv, d, ps, num_pages, scale_log2, window, keep, sink, status, per_head, softcap * LOG2E);  \
     } while (0)
     const bool upper = nq / nkv > 8;
     if (d <= 64) { if (upper) FE_DECODE(64, true); else FE_DECODE(64, false); }
@@ -836,9 +838,9 @@ extern "C" int fe_paged_decode_cluster_resident(int requests, int nq, int nkv, i
 extern "C" int fe_paged_decode_cluster(const void* q, long long q_stride, void* out, long long out_stride,
                                        const void* kc, const void* vc, const int* block_table, int bt_stride,
                                        const int* cu_q, const int* q_start, int requests, int nq, int nkv, int d, int ps,
-                                       int num_pages, float scale, int window, int sink, int splits, int* status,
+                                       int num_pages, float scale, int window, int keep, int sink, int splits, int* status,
                                        const float* per_head, float softcap, cudaStream_t stream) {
-    if (check_common("paged_decode", nq, nkv, d, ps, num_pages, window, q_stride, out_stride)) return 1;
+    if (check_common("paged_decode", nq, nkv, d, ps, num_pages, window, keep, q_stride, out_stride)) return 1;
     FE_REQUIRE(nq / nkv <= 16, "paged_decode: %d query heads per key/value head; this kernel takes up to 16", nq / nkv);
     FE_REQUIRE(splits >= 1 && splits <= CLUSTER_MAX_SPLITS && requests >= 0,
                "paged_decode (cluster): %d splits; a cluster takes 1 to %d", splits, CLUSTER_MAX_SPLITS);
@@ -876,7 +878,7 @@ extern "C" int fe_paged_decode_cluster(const void* q, long long q_stride, void* 
         cfg.dynamicSmemBytes = decode_smem<DMAX>(STAGES);                                                              \
         const cudaError_t err = cudaLaunchKernelEx(&cfg, kernel, (const bf16*)q, q_stride, (bf16*)out, out_stride,     \
             (float*)nullptr, (float*)nullptr, (const bf16*)kc, (const bf16*)vc, block_table, bt_stride, cu_q, q_start, \
-            nq, nkv, d, ps, num_pages, scale_log2, window, sink, status, per_head, softcap * LOG2E);                                   \
+            nq, nkv, d, ps, num_pages, scale_log2, window, keep, sink, status, per_head, softcap * LOG2E);                             \
         FE_REQUIRE(err == cudaSuccess, "paged_decode (cluster of %d): %s", splits, cudaGetErrorString(err));           \
     } while (0)
     const bool upper = nq / nkv > 8;
@@ -894,15 +896,15 @@ extern "C" int fe_paged_decode_mma(const void* q, long long q_stride, void* out,
                                    int num_pages, float scale, int window, int splits, int* status,
                                    cudaStream_t stream) {
     return fe_paged_decode_mma_upcoming(q, q_stride, out, out_stride, scratch, kc, vc, block_table, bt_stride, cu_q, q_start,
-                                        requests, nq, nkv, d, ps, num_pages, scale, window, 0, splits, nullptr, 0, status, nullptr, 0.f, stream);
+                                        requests, nq, nkv, d, ps, num_pages, scale, window, 0, 0, splits, nullptr, 0, status, nullptr, 0.f, stream);
 }
 
 extern "C" int fe_paged_prefill_mma(const void* q, long long q_stride, void* out, long long out_stride,
                                     const void* kc, const void* vc, const int* block_table, int bt_stride,
                                     const int* cu_q, const int* q_start, int requests, int max_q_len, int nq, int nkv,
-                                    int d, int ps, int num_pages, float scale, int window, int sink, int* status,
+                                    int d, int ps, int num_pages, float scale, int window, int keep, int sink, int* status,
                                     const float* per_head, float softcap, cudaStream_t stream) {
-    if (check_common("paged_prefill", nq, nkv, d, ps, num_pages, window, q_stride, out_stride)) return 1;
+    if (check_common("paged_prefill", nq, nkv, d, ps, num_pages, window, keep, q_stride, out_stride)) return 1;
     FE_REQUIRE(requests >= 0 && max_q_len >= 0, "paged_prefill: bad request count or length");
     if (requests == 0 || max_q_len == 0) return 0;
     const long long rows = (long long)max_q_len * (nq / nkv);
@@ -915,7 +917,7 @@ extern "C" int fe_paged_prefill_mma(const void* q, long long q_stride, void* out
         if (allow_smem(paged_prefill_kernel<DMAX>, prefill_smem<DMAX>(), "paged_prefill")) return 1;           \
         fe::launch(paged_prefill_kernel<DMAX>, grid, PREFILL_WARPS * 32, prefill_smem<DMAX>(), stream,                 \
             (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kc, (const bf16*)vc, block_table,  \
-            bt_stride, cu_q, q_start, nq, nkv, d, ps, num_pages, scale_log2, window, sink, status, per_head, softcap * LOG2E); \
+            bt_stride, cu_q, q_start, nq, nkv, d, ps, num_pages, scale_log2, window, keep, sink, status, per_head, softcap * LOG2E); \
     } while (0)
     if (d <= 64) FE_PREFILL(64);
     else if (d <= 128) FE_PREFILL(128);

@@ -4,7 +4,7 @@
 // position 0, one key per lane; scores, running maximum, running sum and the value accumulator
 // are float (online softmax, as the reference's block-wise path:
 // inference/attention/paged.py:50-70).  Key t is visible to the query at position p iff t <= p
-// (and t > p - window when window > 0; t in the chunk of -window positions that holds p when window < 0)
+// (and t > p - window, or t < keep, when window > 0; t in the chunk of -window positions that holds p when window < 0)
 // (paged.py:31-32).  ``sink``: the softmax starts as if a key of score 0 and value 0 had been seen, which adds
 // 1 to its denominator.  ``mode`` bit 1 (bit 0 is the sink): no softmax; the weight of a visible key is
 // sigmoid(score + per_head[h]), not normalised over the keys.  Bit 2: scores are multiplied by per_head[h] (null: by 1) and, with
@@ -27,7 +27,7 @@ __global__ void paged_attention_simt_kernel(const T* __restrict__ q, long long q
                                             int bt_stride, const int* __restrict__ cu_q,
                                             const int* __restrict__ q_start, const int* __restrict__ token_req,
                                             int T_tokens, int nq, int nkv, int d, int ps, int num_pages, float scale,
-                                            int window, int mode, const float* __restrict__ per_head, float softcap, int* __restrict__ status) {
+                                            int window, int keep, int mode, const float* __restrict__ per_head, float softcap, int* __restrict__ status) {
     griddep_wait();
     griddep_launch_dependents();
     extern __shared__ float q_smem[];
@@ -55,9 +55,11 @@ __global__ void paged_attention_simt_kernel(const T* __restrict__ q, long long q
 
     const int lo = first_visible(pos, window);
     const int* table = block_table + (size_t)r * bt_stride;
-    for (int kb = (lo / 32) * 32; kb <= pos; kb += 32) {
+    const int kept = kept_tiles<32>(lo, keep), blocks = kept + pos / 32 - lo / 32 + 1;
+    for (int at = 0; at < blocks; ++at) {
+        const int kb = listed_tile<32>(at, kept, lo) * 32;
         const int t = kb + lane;
-        bool valid = t >= lo && t <= pos;
+        bool valid = (t >= lo || t < keep) && t <= pos;
         float s = -CUDART_INF_F;
         long long base = 0;
         if (valid) {
@@ -121,7 +123,7 @@ template <typename T>
 static int launch_simt(const void* q, long long q_stride, void* out, long long out_stride, const void* kc,
                        const void* vc, const int* block_table, int bt_stride, const int* cu_q, const int* q_start,
                        const int* token_req, int T_tokens, int nq, int nkv, int d, int ps, int num_pages,
-                       float scale, int window, int sink, const float* per_head, float softcap, int* status, cudaStream_t stream) {
+                       float scale, int window, int keep, int sink, const float* per_head, float softcap, int* status, cudaStream_t stream) {
     const int warps = 4;
     const long long total = (long long)T_tokens * nq;
     const int blocks = (int)((total + warps - 1) / warps);
@@ -129,7 +131,7 @@ static int launch_simt(const void* q, long long q_stride, void* out, long long o
 #define FE_LAUNCH_SIMT(DPL)                                                                                      \
     fe::launch(paged_attention_simt_kernel<T, DPL>, blocks, warps * 32, smem, stream,                                    \
         (const T*)q, q_stride, (T*)out, out_stride, (const T*)kc, (const T*)vc, block_table, bt_stride, cu_q,   \
-        q_start, token_req, T_tokens, nq, nkv, d, ps, num_pages, scale, window, sink, per_head, softcap, status)
+        q_start, token_req, T_tokens, nq, nkv, d, ps, num_pages, scale, window, keep, sink, per_head, softcap, status)
     if (d <= 32) FE_LAUNCH_SIMT(1);
     else if (d <= 64) FE_LAUNCH_SIMT(2);
     else if (d <= 128) FE_LAUNCH_SIMT(4);
@@ -143,7 +145,7 @@ static int launch_simt(const void* q, long long q_stride, void* out, long long o
 extern "C" int fe_paged_attention_simt(const void* q, long long q_stride, void* out, long long out_stride,
                                        const void* kc, const void* vc, const int* block_table, int bt_stride,
                                        const int* cu_q, const int* q_start, const int* token_req, int T_tokens,
-                                       int nq, int nkv, int d, int ps, int num_pages, float scale, int window,
+                                       int nq, int nkv, int d, int ps, int num_pages, float scale, int window, int keep,
                                        int sink, int dtype, int* status, const float* per_head, float softcap, cudaStream_t stream) {
     FE_REQUIRE(T_tokens >= 0 && nq > 0 && nkv > 0 && nq % nkv == 0, "paged_attention: bad head counts %d/%d", nq, nkv);
     FE_REQUIRE(d >= 16 && d <= 1024 && d % 16 == 0, "paged_attention: head size %d is not a multiple of 16 in [16, 1024]", d);
@@ -152,9 +154,9 @@ extern "C" int fe_paged_attention_simt(const void* q, long long q_stride, void* 
     if (T_tokens == 0) return 0;
     if (dtype == FE_F32)
         return launch_simt<float>(q, q_stride, out, out_stride, kc, vc, block_table, bt_stride, cu_q, q_start,
-                                  token_req, T_tokens, nq, nkv, d, ps, num_pages, scale, window, sink, per_head, softcap, status, stream);
+                                  token_req, T_tokens, nq, nkv, d, ps, num_pages, scale, window, keep, sink, per_head, softcap, status, stream);
     if (dtype == FE_BF16)
         return launch_simt<bf16>(q, q_stride, out, out_stride, kc, vc, block_table, bt_stride, cu_q, q_start,
-                                 token_req, T_tokens, nq, nkv, d, ps, num_pages, scale, window, sink, per_head, softcap, status, stream);
+                                 token_req, T_tokens, nq, nkv, d, ps, num_pages, scale, window, keep, sink, per_head, softcap, status, stream);
     FE_REQUIRE(false, "paged_attention: unknown dtype %d", dtype);
 }

@@ -1,7 +1,7 @@
 // Paged causal grouped-query attention for prefill portions on the fifth-generation tensor cores.
 //
 // Math as the reference's block-wise path (inference/attention/paged.py:50-70): scores
-// q.k / sqrt(d), key t visible to the query at position p iff t <= p (and t > p - window when
+// q.k / sqrt(d), key t visible to the query at position p iff t <= p (and t > p - window, or t < keep, when
 // window > 0; t in the chunk of -window positions that holds p when window < 0; with ``sink`` the softmax of a row
 // starts as if a key of score 0 and value 0 had been seen, in the first split of its keys), running maximum / sum / output in float (online softmax), query head h reads
 // key/value head h / (nq / nkv).
@@ -189,14 +189,15 @@ __device__ __forceinline__ int swizzled(int r, int c, int block_bytes) {
 
 // The softmax of one row over a key tile, the 64 scores in registers.  MASKED: the tile crosses
 // the causal edge or the window's edge for some row of the warp; ``hi`` and ``lo`` are then this
-// row's last and first visible key relative to the tile.
+// row's last and first visible key relative to the tile, and keys below ``keep`` are visible however far back they are.
+__device__ __forceinline__ bool hidden(int key, int hi, int lo, int keep) { return key > hi || (key < lo && key >= keep); }
 __device__ __forceinline__ float max3(float a, float b, float c) {
     float m;
     asm("max.f32 %0, %1, %2, %3;\n" : "=f"(m) : "f"(a), "f"(b), "f"(c));
     return m;
 }
 template <bool MASKED>
-__device__ __forceinline__ float row_max(const unsigned* r, int hi, int lo) {
+__device__ __forceinline__ float row_max(const unsigned* r, int hi, int lo, int keep) {
     float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, m2 = -CUDART_INF_F, m3 = -CUDART_INF_F;
 #pragma unroll
     for (int i = 0; i < KEYS; i += 8) {
@@ -204,7 +205,7 @@ __device__ __forceinline__ float row_max(const unsigned* r, int hi, int lo) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
             v[e] = __uint_as_float(r[i + e]);
-            if (MASKED && (i + e > hi || i + e < lo)) v[e] = -CUDART_INF_F;
+            if (MASKED && hidden(i + e, hi, lo, keep)) v[e] = -CUDART_INF_F;
         }
         m0 = max3(m0, v[0], v[1]), m1 = max3(m1, v[2], v[3]), m2 = max3(m2, v[4], v[5]), m3 = max3(m3, v[6], v[7]);
     }
@@ -213,7 +214,7 @@ __device__ __forceinline__ float row_max(const unsigned* r, int hi, int lo) {
 // P = 2^(s scale - ref) as bfloat16 pairs over the scores' own columns (32 of the 64); returns the row's sum.
 // The multiply-adds and the sums run two floats per instruction.
 template <bool MASKED>
-__device__ __forceinline__ float row_exp(const unsigned* r, unsigned p_addr, int hi, int lo, float scale_log2, float ref) {
+__device__ __forceinline__ float row_exp(const unsigned* r, unsigned p_addr, int hi, int lo, int keep, float scale_log2, float ref) {
     float2 sum = make_float2(0.f, 0.f);
     const float2 scale2 = make_float2(scale_log2, scale_log2), ref2 = make_float2(-ref, -ref);
 #pragma unroll
@@ -225,8 +226,8 @@ __device__ __forceinline__ float row_exp(const unsigned* r, unsigned p_addr, int
             const float2 t = __ffma2_rn(make_float2(__uint_as_float(r[k]), __uint_as_float(r[k + 1])), scale2, ref2);
             float2 e = make_float2(ex2(t.x), ex2(t.y));
             if (MASKED) {
-                if (k > hi || k < lo) e.x = 0.f;
-                if (k + 1 > hi || k + 1 < lo) e.y = 0.f;
+                if (hidden(k, hi, lo, keep)) e.x = 0.f;
+                if (hidden(k + 1, hi, lo, keep)) e.y = 0.f;
             }
             sum = __fadd2_rn(sum, e);
             const __nv_bfloat162 pair = __floats2bfloat162_rn(e.x, e.y);
@@ -240,7 +241,7 @@ __device__ __forceinline__ float row_exp(const unsigned* r, unsigned p_addr, int
 // Sigmoid weights instead of a softmax: P = 1 / (1 + 2^-(s scale + bias)) as bfloat16 pairs over the scores' own columns;
 // nothing is summed, a masked key weighs 0.
 template <bool MASKED>
-__device__ __forceinline__ void row_sigmoid(const unsigned* r, unsigned p_addr, int hi, int lo, float scale_log2, float bias) {
+__device__ __forceinline__ void row_sigmoid(const unsigned* r, unsigned p_addr, int hi, int lo, int keep, float scale_log2, float bias) {
     const float2 scale2 = make_float2(-scale_log2, -scale_log2), bias2 = make_float2(-bias, -bias);
 #pragma unroll
     for (int c = 0; c < KEYS; c += 32) {
@@ -251,8 +252,8 @@ __device__ __forceinline__ void row_sigmoid(const unsigned* r, unsigned p_addr, 
             const float2 t = __ffma2_rn(make_float2(__uint_as_float(r[k]), __uint_as_float(r[k + 1])), scale2, bias2);
             float2 e = make_float2(rcp(1.f + ex2(t.x)), rcp(1.f + ex2(t.y)));
             if (MASKED) {
-                if (k > hi || k < lo) e.x = 0.f;
-                if (k + 1 > hi || k + 1 < lo) e.y = 0.f;
+                if (hidden(k, hi, lo, keep)) e.x = 0.f;
+                if (hidden(k + 1, hi, lo, keep)) e.y = 0.f;
             }
             const __nv_bfloat162 pair = __floats2bfloat162_rn(e.x, e.y);
             packed[i] = *reinterpret_cast<const unsigned*>(&pair);
@@ -309,7 +310,7 @@ paged_prefill_tcgen05_kernel(const bf16* __restrict__ q, long long q_stride, bf1
                              const bf16* __restrict__ kc, const bf16* __restrict__ vc,
                              const int* __restrict__ block_table, int bt_stride, const int* __restrict__ cu_q,
                              const int* __restrict__ q_start, int nq, int nkv, int ps, int num_pages, float scale_log2,
-                             int window, int mode, int splits, float* __restrict__ part_o, float* __restrict__ part_lse,
+                             int window, int keep, int mode, int splits, float* __restrict__ part_o, float* __restrict__ part_lse,
                              int* __restrict__ status, const float* __restrict__ per_head, float cap_log2) {
     const bool sink = mode & 1, sigmoid = mode & 2;         // bit 1: sigmoid(score + per_head[head]) instead of a softmax
     const bool mapped = mode & 4;       // scores times per_head[head] (null: 1) and, with a cap, cap tanh(score / cap), before the softmax
@@ -344,8 +345,9 @@ paged_prefill_tcgen05_kernel(const bf16* __restrict__ q, long long q_stride, bf1
     const int hi = start + qi_last;
     const int lo = first_visible(start + qi_first, window);
     // this block's share of the key tiles; with one split, all of them
-    const int all_tiles = hi / KEYS - lo / KEYS + 1, per_split = (all_tiles + splits - 1) / splits;
-    const int t_begin = lo / KEYS + split * per_split, n_tiles = min(per_split, all_tiles - split * per_split);
+    const int kept = kept_tiles<KEYS>(lo, keep);       // tiles are counted along the list of those walked
+    const int all_tiles = kept + hi / KEYS - lo / KEYS + 1, per_split = (all_tiles + splits - 1) / splits;
+    const int t_begin = split * per_split, n_tiles = min(per_split, all_tiles - split * per_split);
     if (n_tiles <= 0) {
         // nothing left for this split: its rows say so, and the merge reads nothing more of them
         const int m = m_pair + tid;
@@ -421,9 +423,9 @@ paged_prefill_tcgen05_kernel(const bf16* __restrict__ q, long long q_stride, bf1
                 mbar_wait(&kv_empty[s], ((j / KV_STAGES) & 1) ^ 1, &give_up);     // free from the start
                 long long* tile_offs = offs[j & 1];
                 if (lt < KEYS) {
-                    const int key = (t_begin + j) * KEYS + lt;
+                    const int key = listed_tile<KEYS>(t_begin + j, kept, lo) * KEYS + lt;
                     long long off = -1;
-                    if (key >= lo && key <= hi) {
+                    if ((key >= lo || key < keep) && key <= hi) {
                         const int page = block_table[(size_t)r * bt_stride + (ps_shift >= 0 ? key >> ps_shift : key / ps)];
                         if (page < 0 || page >= num_pages) {
                             if (status) atomicOr(status, FE_STATUS_BAD_PAGE);
@@ -522,19 +524,19 @@ paged_prefill_tcgen05_kernel(const bf16* __restrict__ q, long long q_stride, bf1
             tmem_load_wait();
             tie32(raw);
             tie32(raw + 32);
-            const int key0 = (t_begin + j) * KEYS;
-            const bool unmasked = key0 + KEYS - 1 <= pos_min && key0 >= lo_max;      // for the whole warp
-            const int rel_hi = pos - key0, rel_lo = row_lo - key0;
+            const int key0 = listed_tile<KEYS>(t_begin + j, kept, lo) * KEYS;
+            const bool unmasked = key0 + KEYS - 1 <= pos_min && (key0 >= lo_max || key0 + KEYS <= keep);      // for the whole warp
+            const int rel_hi = pos - key0, rel_lo = row_lo - key0, rel_keep = keep - key0;
             if (sigmoid) {
-                if (unmasked) row_sigmoid<false>(raw, s_addr, rel_hi, rel_lo, scale_log2, bias);
-                else row_sigmoid<true>(raw, s_addr, rel_hi, rel_lo, scale_log2, bias);
+                if (unmasked) row_sigmoid<false>(raw, s_addr, rel_hi, rel_lo, rel_keep, scale_log2, bias);
+                else row_sigmoid<true>(raw, s_addr, rel_hi, rel_lo, rel_keep, scale_log2, bias);
                 tmem_store_wait();
                 tc_fence_before();
                 mbar_arrive(&p_ready[ti][j & 1]);
                 continue;
             }
             if (mapped) row_map(raw, unit, cap_log2);
-            const float mx = unmasked ? row_max<false>(raw, rel_hi, rel_lo) : row_max<true>(raw, rel_hi, rel_lo);
+            const float mx = unmasked ? row_max<false>(raw, rel_hi, rel_lo, rel_keep) : row_max<true>(raw, rel_hi, rel_lo, rel_keep);
             const float m_new = fmaxf(m_ref, mx * to_log2);
             if (__any_sync(FULL, m_new > m_ref + RESCALE_STEP)) {
                 // move the reference point to the new maximum: O and the sum were taken against the old one
@@ -556,8 +558,8 @@ paged_prefill_tcgen05_kernel(const bf16* __restrict__ q, long long q_stride, bf1
                 m_ref = m_new;
             }
             const float m_safe = m_ref == -CUDART_INF_F ? 0.f : m_ref;
-            row_sum += unmasked ? row_exp<false>(raw, s_addr, rel_hi, rel_lo, to_log2, m_safe)
-                                : row_exp<true>(raw, s_addr, rel_hi, rel_lo, to_log2, m_safe);
+            row_sum += unmasked ? row_exp<false>(raw, s_addr, rel_hi, rel_lo, rel_keep, to_log2, m_safe)
+                                : row_exp<true>(raw, s_addr, rel_hi, rel_lo, rel_keep, to_log2, m_safe);
             tmem_store_wait();
             tc_fence_before();
             mbar_arrive(&p_ready[ti][j & 1]);
@@ -664,7 +666,7 @@ prefill_merge_kernel(const float* __restrict__ part_o, const float* __restrict__
 template <int D>
 int launch(const void* q, long long q_stride, void* out, long long out_stride, const void* kc, const void* vc,
            const int* block_table, int bt_stride, const int* cu_q, const int* q_start, int requests, int max_q_len, int nq,
-           int nkv, int ps, int num_pages, float scale, int window, int sink, int splits, float* scratch, long long total_tokens,
+           int nkv, int ps, int num_pages, float scale, int window, int keep, int sink, int splits, float* scratch, long long total_tokens,
            int* status, const float* per_head, float softcap, cudaStream_t stream) {
     const size_t smem = (size_t)(D / 64) * (2 * Q_BLOCK + 2 * KV_STAGES * KV_BLOCK) + 1024;
     const cudaError_t err = cudaFuncSetAttribute(paged_prefill_tcgen05_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -677,7 +679,7 @@ int launch(const void* q, long long q_stride, void* out, long long out_stride, c
     float* part_lse = splits > 1 ? scratch + (size_t)total_tokens * nq * splits * D : nullptr;
     fe::launch(paged_prefill_tcgen05_kernel<D>, dim3((unsigned)tiles, nkv, requests), THREADS, smem, stream, (const bf16*)q, q_stride,
                (bf16*)out, out_stride, (const bf16*)kc, (const bf16*)vc, block_table, bt_stride, cu_q, q_start, nq, nkv, ps,
-               num_pages, scale * LOG2E, window, sink, splits, part_o, part_lse, status, per_head, softcap * LOG2E);
+               num_pages, scale * LOG2E, window, keep, sink, splits, part_o, part_lse, status, per_head, softcap * LOG2E);
     if (fe_check_launch("paged_prefill_tcgen05")) return 1;
     if (splits > 1) {
         const long long items = total_tokens * nq;
@@ -702,21 +704,21 @@ extern "C" long long fe_paged_prefill_tcgen05_scratch_floats(long long total_tok
 extern "C" int fe_paged_prefill_tcgen05(const void* q, long long q_stride, void* out, long long out_stride, const void* kc,
                                         const void* vc, const int* block_table, int bt_stride, const int* cu_q,
                                         const int* q_start, int requests, int max_q_len, int nq, int nkv, int d, int ps,
-                                        int num_pages, float scale, int window, int sink, int splits, void* scratch,
+                                        int num_pages, float scale, int window, int keep, int sink, int splits, void* scratch,
                                         long long total_tokens, int* status, const float* per_head, float softcap, cudaStream_t stream) {
     FE_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "paged_prefill_tcgen05: bad head counts %d/%d", nq, nkv);
     FE_REQUIRE(d == 64 || d == 128, "paged_prefill_tcgen05: head size %d; this kernel takes 64 and 128", d);
     FE_REQUIRE(ps > 0 && num_pages > 0, "paged_prefill_tcgen05: bad page size or page count");
     FE_REQUIRE(q_stride % 8 == 0 && out_stride % 8 == 0 && (((size_t)q | (size_t)out | (size_t)kc | (size_t)vc) & 15) == 0,
                "paged_prefill_tcgen05: rows must start on 16-byte boundaries");
-    FE_REQUIRE(requests >= 0 && max_q_len >= 0, "paged_prefill_tcgen05: bad request count or length");
+    FE_REQUIRE(requests >= 0 && max_q_len >= 0 && keep >= 0 && (keep == 0 || window > 0), "paged_prefill_tcgen05: bad request count or length, or kept keys without a window");
     FE_REQUIRE(splits >= 1 && splits <= MAX_SPLITS, "paged_prefill_tcgen05: %d splits; 1 to %d", splits, MAX_SPLITS);
     FE_REQUIRE(splits == 1 || (scratch != nullptr && ((size_t)scratch & 15) == 0 && total_tokens > 0),
                "paged_prefill_tcgen05: splits need scratch memory on a 16-byte boundary and the number of tokens");
     if (requests == 0 || max_q_len == 0) return 0;
     if (d == 64)
         return launch<64>(q, q_stride, out, out_stride, kc, vc, block_table, bt_stride, cu_q, q_start, requests, max_q_len, nq, nkv,
-                          ps, num_pages, scale, window, sink, splits, (float*)scratch, total_tokens, status, per_head, softcap, stream);
+                          ps, num_pages, scale, window, keep, sink, splits, (float*)scratch, total_tokens, status, per_head, softcap, stream);
     return launch<128>(q, q_stride, out, out_stride, kc, vc, block_table, bt_stride, cu_q, q_start, requests, max_q_len, nq, nkv, ps,
-                       num_pages, scale, window, sink, splits, (float*)scratch, total_tokens, status, per_head, softcap, stream);
+                       num_pages, scale, window, keep, sink, splits, (float*)scratch, total_tokens, status, per_head, softcap, stream);
 }

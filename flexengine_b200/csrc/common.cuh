@@ -96,6 +96,27 @@ template <> __device__ __forceinline__ void store8<bf16>(bf16* p, const float* v
 // The exact form of GELU: z/2 (1 + erf(z / sqrt(2))).
 __device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
 
+// e^x for x <= 0 to about half an ulp: x = k ln 2 + r with k whole and |r| <= ln 2 / 2 (ln 2 in two parts, Cody and Waite's
+// reduction), the Taylor polynomial of e^r - 1 to the seventh power (the next term is below 6e-9), and k added to the exponent.  A
+// recurrence multiplies the same decay into its state token after token: errors of a rounding or two that always fall to the same
+// side, as the hardware's 2^x has them next to 1, add up over a long sequence; half an ulp either way does not.
+__device__ __forceinline__ float exp_decay(float x) {
+    x = fmaxf(x, -87.f);
+    const float magic = 12582912.f;                       // 1.5 2^23: adding it rounds to a whole number
+    const float t = fmaf(x, 1.44269504f, magic);
+    const float k = t - magic;
+    float r = fmaf(k, -0.693359375f, x);                  // the upper part of ln 2 has nine bits: k times it is exact
+    r = fmaf(k, 2.12194440e-4f, r);
+    float p = 1.f / 5040.f;
+    p = fmaf(p, r, 1.f / 720.f);
+    p = fmaf(p, r, 1.f / 120.f);
+    p = fmaf(p, r, 1.f / 24.f);
+    p = fmaf(p, r, 1.f / 6.f);
+    p = fmaf(p, r, 0.5f);
+    p = fmaf(p * r, r, r);                                // r + r^2 (1/2 + ...)
+    return __int_as_float(__float_as_int(1.f + p) + (__float_as_int(t) << 23));
+}
+
 // What a query at position ``pos`` sees of the keys t <= pos, as one int: 0 every key; w > 0 the last w keys (a sliding
 // window); -c < 0 the keys of its own chunk of c positions, counted from position 0.  The first visible key:
 __host__ __device__ __forceinline__ int first_visible(int pos, int window) {
@@ -103,6 +124,16 @@ __host__ __device__ __forceinline__ int first_visible(int pos, int window) {
     if (window < 0 && pos > 0) return pos - pos % (-window);
     return 0;
 }
+
+// Under a window (w > 0) the first ``keep`` keys of a sequence may stay visible however far back they are.  Keys are walked in
+// tiles of TILE keys aligned to position 0; what is walked is a list of tiles: the tiles that hold kept keys before the
+// tile of the first key inside the window (``kept_tiles`` of them), then the tiles from that one on.
+template <int TILE> __host__ __device__ __forceinline__ int kept_tiles(int lo, int keep) {
+    const int n = (keep + TILE - 1) / TILE;
+    return n < lo / TILE ? n : lo / TILE;
+}
+// The i-th tile of that list.
+template <int TILE> __host__ __device__ __forceinline__ int listed_tile(int i, int kept, int lo) { return i < kept ? i : lo / TILE + (i - kept); }
 
 // Programmatic dependent launch: a kernel launched through fe::launch may begin while the kernel
 // before it in the stream is still running.  Everything it reads that an earlier kernel wrote,

@@ -72,9 +72,10 @@ extern "C" int fe_carry_tokens(int* token_ids, const int* rows, const int* sourc
 // ---------------------------------------------------------------------------------------------
 // One block per output row.  rows == nullptr: row i; the residual is updated in place (residual
 // += delta).  rows != nullptr: output row i reads residual row rows[i] (+ delta row rows[i]) and
-// the residual is left as it is.  The row is staged in shared memory (H floats).
-template <typename T>
-__global__ void add_rmsnorm_kernel(float* __restrict__ residual, const T* __restrict__ delta,
+// the residual is left as it is.  The row is staged in shared memory (H floats).  ``delta_scale`` (may be null): a number per
+// column that delta is multiplied by; delta is of its own type (the compute type or float).
+template <typename T, typename TD>
+__global__ void add_rmsnorm_kernel(float* __restrict__ residual, const TD* __restrict__ delta, const float* __restrict__ delta_scale,
                                    const float* __restrict__ weight, float eps, T* __restrict__ out,
                                    const int* __restrict__ rows, int H, int n_rows_total, int n_out,
                                    const void* __restrict__ upcoming, long long upcoming_bytes) {
@@ -91,11 +92,11 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ residual, const T* __rest
     int r = rows ? rows[i] : i;
     if (r < 0 || r >= n_rows_total) r = 0;          // guarded: rows are checked on the host
     float* res = residual + (size_t)r * H;
-    const T* del = delta ? delta + (size_t)r * H : nullptr;
+    const TD* del = delta ? delta + (size_t)r * H : nullptr;
     float ss = 0.f;
     for (int j = threadIdx.x; j < H; j += blockDim.x) {
         float v = res[j];
-        if (del) v += to_float(del[j]);
+        if (del) v += to_float(del[j]) * (delta_scale ? delta_scale[j] : 1.f);
         row[j] = v;
         if (!rows && del) res[j] = v;
         ss += v * v;
@@ -127,8 +128,8 @@ template <> struct Vec4<bf16> {
     }
 };
 
-template <typename T>
-__global__ void add_rmsnorm_vec_kernel(float* __restrict__ residual, const T* __restrict__ delta,
+template <typename T, typename TD>
+__global__ void add_rmsnorm_vec_kernel(float* __restrict__ residual, const TD* __restrict__ delta, const float* __restrict__ delta_scale,
                                        const float* __restrict__ weight, float eps, T* __restrict__ out,
                                        const int* __restrict__ rows, int H, int n_rows_total, int n_out,
                                        const void* __restrict__ upcoming, long long upcoming_bytes) {
@@ -145,12 +146,16 @@ __global__ void add_rmsnorm_vec_kernel(float* __restrict__ residual, const T* __
     int r = rows ? rows[i] : i;
     if (r < 0 || r >= n_rows_total) r = 0;
     float* res = residual + (size_t)r * H;
-    const T* del = delta ? delta + (size_t)r * H : nullptr;
+    const TD* del = delta ? delta + (size_t)r * H : nullptr;
     float ss = 0.f;
     for (int j = threadIdx.x * 4; j < H; j += blockDim.x * 4) {
         float4 v = *reinterpret_cast<const float4*>(res + j);
         if (del) {
-            const float4 dv = Vec4<T>::load(del + j);
+            float4 dv = Vec4<TD>::load(del + j);
+            if (delta_scale) {
+                const float4 s = *reinterpret_cast<const float4*>(delta_scale + j);
+                dv.x *= s.x; dv.y *= s.y; dv.z *= s.z; dv.w *= s.w;
+            }
             v.x += dv.x; v.y += dv.y; v.z += dv.z; v.w += dv.w;
             if (!rows) *reinterpret_cast<float4*>(res + j) = v;
         }
@@ -169,8 +174,8 @@ __global__ void add_rmsnorm_vec_kernel(float* __restrict__ residual, const T* __
 
 constexpr int PREFETCH_BLOCKS = 64;
 
-template <typename T>
-static int launch_add_rmsnorm(float* residual, const void* delta, const float* weight, float eps, void* out,
+template <typename T, typename TD>
+static int launch_add_rmsnorm(float* residual, const void* delta, const float* delta_scale, const float* weight, float eps, void* out,
                               const int* rows, int n_out, int H, int n_rows_total, const void* upcoming,
                               long long upcoming_bytes, cudaStream_t stream) {
     const int grid = n_out + (upcoming && upcoming_bytes > 0 ? PREFETCH_BLOCKS : 0);
@@ -180,15 +185,15 @@ static int launch_add_rmsnorm(float* residual, const void* delta, const float* w
     cudaError_t err = cudaSuccess;
     if (vec) {
         if (smem > 48 * 1024)
-            err = cudaFuncSetAttribute(add_rmsnorm_vec_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            err = cudaFuncSetAttribute(add_rmsnorm_vec_kernel<T, TD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         FE_REQUIRE(err == cudaSuccess, "add_rmsnorm: %s", cudaGetErrorString(err));
-        fe::launch(add_rmsnorm_vec_kernel<T>, grid, threads, smem, stream, residual, (const T*)delta, weight, eps, (T*)out,
+        fe::launch(add_rmsnorm_vec_kernel<T, TD>, grid, threads, smem, stream, residual, (const TD*)delta, delta_scale, weight, eps, (T*)out,
                    rows, H, n_rows_total, n_out, upcoming, upcoming_bytes);
     } else {
         if (smem > 48 * 1024)
-            err = cudaFuncSetAttribute(add_rmsnorm_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            err = cudaFuncSetAttribute(add_rmsnorm_kernel<T, TD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         FE_REQUIRE(err == cudaSuccess, "add_rmsnorm: %s", cudaGetErrorString(err));
-        fe::launch(add_rmsnorm_kernel<T>, grid, threads, smem, stream, residual, (const T*)delta, weight, eps, (T*)out, rows,
+        fe::launch(add_rmsnorm_kernel<T, TD>, grid, threads, smem, stream, residual, (const TD*)delta, delta_scale, weight, eps, (T*)out, rows,
                    H, n_rows_total, n_out, upcoming, upcoming_bytes);
     }
     return fe_check_launch("add_rmsnorm");
@@ -204,10 +209,26 @@ extern "C" int fe_add_rmsnorm(float* residual, const void* delta, const float* w
     FE_REQUIRE((size_t)H * sizeof(float) <= 200 * 1024,
                "add_rmsnorm: hidden size %d needs %zu bytes of shared memory (limit 204800)", H, (size_t)H * sizeof(float));
     if (dtype == FE_F32)
-        return launch_add_rmsnorm<float>(residual, delta, weight, eps, out, rows, n_out, H, n_rows_total, upcoming, upcoming_bytes, stream);
+        return launch_add_rmsnorm<float, float>(residual, delta, nullptr, weight, eps, out, rows, n_out, H, n_rows_total, upcoming, upcoming_bytes, stream);
     if (dtype == FE_BF16)
-        return launch_add_rmsnorm<bf16>(residual, delta, weight, eps, out, rows, n_out, H, n_rows_total, upcoming, upcoming_bytes, stream);
+        return launch_add_rmsnorm<bf16, bf16>(residual, delta, nullptr, weight, eps, out, rows, n_out, H, n_rows_total, upcoming, upcoming_bytes, stream);
     FE_REQUIRE(false, "add_rmsnorm: unknown dtype %d", dtype);
+}
+
+// The same for a branch that enters the stream times a number per column: residual += delta_scale * delta.  delta is of
+// delta_dtype: the compute type or float.
+extern "C" int fe_add_rmsnorm_scaled(float* residual, const void* delta, int delta_dtype, const float* delta_scale, const float* weight,
+                                     float eps, void* out, const int* rows, int n_out, int H, int n_rows_total, int dtype,
+                                     const void* upcoming, long long upcoming_bytes, cudaStream_t stream) {
+    FE_REQUIRE(n_out >= 0 && H > 0 && upcoming_bytes >= 0, "add_rmsnorm: bad sizes n=%d H=%d", n_out, H);
+    FE_REQUIRE((size_t)H * sizeof(float) <= 200 * 1024, "add_rmsnorm: hidden size %d needs too much shared memory", H);
+    FE_REQUIRE((dtype == FE_F32 || dtype == FE_BF16) && (delta_dtype == FE_F32 || delta_dtype == dtype), "add_rmsnorm: unknown dtypes %d, %d", dtype, delta_dtype);
+    if (n_out == 0) return 0;
+    if (dtype == FE_F32)
+        return launch_add_rmsnorm<float, float>(residual, delta, delta_scale, weight, eps, out, rows, n_out, H, n_rows_total, upcoming, upcoming_bytes, stream);
+    if (delta_dtype == FE_F32)
+        return launch_add_rmsnorm<bf16, float>(residual, delta, delta_scale, weight, eps, out, rows, n_out, H, n_rows_total, upcoming, upcoming_bytes, stream);
+    return launch_add_rmsnorm<bf16, bf16>(residual, delta, delta_scale, weight, eps, out, rows, n_out, H, n_rows_total, upcoming, upcoming_bytes, stream);
 }
 
 // ---------------------------------------------------------------------------------------------

@@ -169,7 +169,8 @@ __global__ void __launch_bounds__(THREADS)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                     void* __restrict__ out_raw, int M, int N_out, int K, int up_row_offset, int m_tiles, int n_tiles,
                     const int* __restrict__ g_tiles, const int* __restrict__ g_expert, const int* __restrict__ g_row0,
-                    const int* __restrict__ g_offsets, int w_rows, int gate_act, float gate_limit, int* __restrict__ status) {
+                    const int* __restrict__ g_offsets, int w_rows, int gate_act, float gate_limit, int* __restrict__ status,
+                    const float* __restrict__ row_weights, const int* __restrict__ pair_of_row) {
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     __shared__ __align__(8) unsigned long long full_bar[STAGES], empty_bar[STAGES];
     __shared__ __align__(8) unsigned long long acc_full[ACC_BUFFERS], acc_empty[ACC_BUFFERS];
@@ -267,6 +268,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
             if (!mbar_wait(&acc_full[buf], (i >> 1) & 1)) { give_up = 1; break; }
             tc_fence_after();
             const int row = m0 + quarter * 32 + lane;
+            // what this row's products are multiplied by before the activation (grouped form: an expert that reads weight * h)
+            const float rw = (row_weights && row < row_end) ? row_weights[pair_of_row[row]] : 1.f;
             const unsigned lane_addr = tmem_base + buf * BN + ((unsigned)(quarter * 32) << 16);
 #pragma unroll 1
             for (int c = 0; c < OUT_COLS; c += 32) {
@@ -276,7 +279,11 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                     float u[32];
                     tmem_load32(lane_addr + 128 + c, u);
 #pragma unroll
-                    for (int j = 0; j < 32; ++j) v[j] = gated_value(v[j], u[j], gate_act, gate_limit);
+                    for (int j = 0; j < 32; ++j) v[j] = gated_value(v[j] * rw, u[j] * rw, gate_act, gate_limit);
+                }
+                if (EPI == EPI_BF16 && row_weights) {
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) v[j] *= rw;
                 }
                 if (EPI == EPI_BF16 && gate_act == ACT_RELU2) {
 #pragma unroll
@@ -353,7 +360,8 @@ int make_map(CUtensorMap* map, const void* base, long long rows, long long cols,
 template <int EPI>
 int launch(const void* x, const void* W, void* out, int M, int N, int K, int* status, cudaStream_t stream,
            const int* g_tiles = nullptr, const int* g_expert = nullptr, const int* g_row0 = nullptr, const int* g_offsets = nullptr,
-           long long w_rows_total = 0, int gate_act = 0, float gate_limit = 0.f) {
+           long long w_rows_total = 0, int gate_act = 0, float gate_limit = 0.f, const float* row_weights = nullptr,
+           const int* pair_of_row = nullptr) {
     const int n_out = EPI == EPI_SWIGLU ? N / 2 : N;
     constexpr int OUT_COLS = EPI == EPI_SWIGLU ? 128 : 256;
     CUtensorMap map_a, map_b;
@@ -367,7 +375,7 @@ int launch(const void* x, const void* W, void* out, int M, int N, int K, int* st
     const long long total = (long long)m_tiles * n_tiles;
     const int blocks = g_tiles ? sms : (int)(total < sms ? total : sms);        // one persistent block per SM
     fe::launch(gemm_tcgen05_kernel<EPI>, blocks, THREADS, smem, stream, map_a, map_b, out, M, n_out, K, n_out,
-               m_tiles, n_tiles, g_tiles, g_expert, g_row0, g_offsets, N, gate_act, gate_limit, status);
+               m_tiles, n_tiles, g_tiles, g_expert, g_row0, g_offsets, N, gate_act, gate_limit, status, row_weights, pair_of_row);
     return fe_check_launch("gemm_tcgen05");
 }
 
@@ -395,10 +403,12 @@ extern "C" int fe_gemm_tcgen05(const void* x, const void* W, void* out, int M, i
 // then its up rows), the row tiles of 128 from a list on the device (tiles[0] of them: tile_expert, tile_row0; offsets
 // [experts + 1] are the experts' row ranges).  epilogue 1: out float [rows, N]; 2: SwiGLU, out bfloat16 [rows, N / 2]; with
 // ``limit`` > 0 the gated epilogue is the clamped one (see gated_value); 6 and 8: experts without a gate, out = relu(product)^2
-// or the exact GELU of the product as bfloat16 [rows, N].
+// or the exact GELU of the product as bfloat16 [rows, N].  row_weights (may be null; epilogues 2, 6, 8): row r's products are
+// multiplied by row_weights[pair_of_row[r]] before the activation.
 extern "C" int fe_gemm_tcgen05_grouped(const void* x, const void* W, void* out, int rows, int experts, int N, int K, int epilogue,
                                        const int* tiles, const int* tile_expert, const int* tile_row0, const int* offsets,
-                                       float limit, int* status, cudaStream_t stream) {
+                                       float limit, const float* row_weights, const int* pair_of_row, int* status, cudaStream_t stream) {
+    FE_REQUIRE(row_weights == nullptr || pair_of_row != nullptr, "gemm_tcgen05 (grouped): row weights need the rows' pairs");
     FE_REQUIRE(rows >= 1 && experts >= 1 && N >= 1 && K >= 8, "gemm_tcgen05 (grouped): bad sizes rows=%d N=%d K=%d", rows, N, K);
     FE_REQUIRE(K % 8 == 0, "gemm_tcgen05 (grouped): K = %d must be a multiple of 8 (rows must start on 16-byte boundaries)", K);
     FE_REQUIRE((((size_t)x | (size_t)W | (size_t)out) & 15) == 0, "gemm_tcgen05 (grouped): operands must be 16-byte aligned");
@@ -407,11 +417,11 @@ extern "C" int fe_gemm_tcgen05_grouped(const void* x, const void* W, void* out, 
     if (epilogue == EPI_F32) return launch<EPI_F32>(x, W, out, rows, N, K, status, stream, tiles, tile_expert, tile_row0, offsets, w_rows_total);
     if (epilogue == EPI_RELU2 || epilogue == EPI_GELU)
         return launch<EPI_BF16>(x, W, out, rows, N, K, status, stream, tiles, tile_expert, tile_row0, offsets, w_rows_total,
-                                epilogue == EPI_GELU ? ACT_GELU : ACT_RELU2);
+                                epilogue == EPI_GELU ? ACT_GELU : ACT_RELU2, 0.f, row_weights, pair_of_row);
     if (epilogue == EPI_SWIGLU) {
         FE_REQUIRE(N % 2 == 0, "gemm_tcgen05 (grouped): SwiGLU needs an even number of weight rows, got %d", N);
         return launch<EPI_SWIGLU>(x, W, out, rows, N, K, status, stream, tiles, tile_expert, tile_row0, offsets, w_rows_total,
-                                  limit > 0.f ? 2 : 0, limit);
+                                  limit > 0.f ? 2 : 0, limit, row_weights, pair_of_row);
     }
     FE_REQUIRE(false, "gemm_tcgen05 (grouped): unknown epilogue %d", epilogue);
 }

@@ -774,6 +774,7 @@ extern "C" int fe_qkv_conv_rope_norm_cache(const void* proj, long long ld, const
 //     square and multiplied by a weight of heads * dim numbers; the whole key projection likewise (kv_heads * dim);
 //   rotation (q, k), after the norm: the first ``rot`` entries of every head turn by position * inv_freq[i]; pairs are
 //     (2i, 2i + 1) when ``interleaved``, else (i, i + rot/2);
+//   ``bias`` (may be null): a number per column of q | k | v, added before everything else; ``gain`` multiplies what turns;
 //   values (v_inv_freq given): all ``vdim`` entries of every value head turn by position * v_inv_freq[m], pairs laid out
 //     the same way;
 //   q into ``q_out`` [T, heads * head], k and v into their cache slots [pages, kv_heads, ps, head], zeros beyond dim / vdim.
@@ -798,7 +799,8 @@ template <typename T>
 __global__ void qkv_norm_rope_cache_kernel(const T* __restrict__ proj, long long ld, const float* __restrict__ q_weight,
                                            const float* __restrict__ k_weight, float eps, const int* __restrict__ positions,
                                            const float* __restrict__ inv_freq, int rot, int interleaved,
-                                           const float* __restrict__ v_inv_freq, const int* __restrict__ slot_mapping,
+                                           const float* __restrict__ v_inv_freq, const float* __restrict__ bias, float gain,
+                                           const int* __restrict__ slot_mapping,
                                            T* __restrict__ kc, T* __restrict__ vc, T* __restrict__ q_out, int heads, int kv_heads,
                                            int dim, int vdim, int head, int ps, long long num_slots, int* __restrict__ status) {
     griddep_wait();
@@ -815,12 +817,17 @@ __global__ void qkv_norm_rope_cache_kernel(const T* __restrict__ proj, long long
     float* vcos = sines + half;                       // [vhalf], then [vhalf]
     float* vsin = vcos + vhalf;
     const float pos = (float)positions[tok];
-    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(pos * inv_freq[i], &sines[i], &cosines[i]);
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float si, co;
+        sincosf(pos * inv_freq[i], &si, &co);
+        sines[i] = si * gain;
+        cosines[i] = co * gain;
+    }
     for (int i = threadIdx.x; i < vhalf; i += blockDim.x) sincosf(pos * v_inv_freq[i], &vsin[i], &vcos[i]);
     const T* src = proj + (size_t)tok * ld;
     float ssq = 0.f, ssk = 0.f;
     for (int c = threadIdx.x; c < C; c += blockDim.x) {
-        const float v = to_float(src[c]);
+        const float v = to_float(src[c]) + (bias ? bias[c] : 0.f);
         row[c] = v;
         if (c < qw) ssq = fmaf(v, v, ssq);
         else if (c < qw + kw) ssk = fmaf(v, v, ssk);
@@ -891,6 +898,7 @@ __global__ void unrotate_heads_kernel(const T* __restrict__ mixed, const int* __
 
 extern "C" int fe_qkv_norm_rope_cache(const void* proj, long long ld, const float* q_weight, const float* k_weight, float eps,
                                       const int* positions, const float* inv_freq, int rot, int interleaved, const float* v_inv_freq,
+                                      const float* bias, float gain,
                                       const int* slot_mapping, void* kc, void* vc, void* q_out, int T, int heads, int kv_heads, int dim,
                                       int vdim, int head, int ps, long long num_slots, int dtype, int* status, cudaStream_t stream) {
     FE_REQUIRE((q_weight == nullptr) == (k_weight == nullptr), "qkv_norm_rope_cache: the norm weights come in pairs");
@@ -912,7 +920,7 @@ extern "C" int fe_qkv_norm_rope_cache(const void* proj, long long ld, const floa
             FE_REQUIRE(err == cudaSuccess, "qkv_norm_rope_cache: %s", cudaGetErrorString(err));                                          \
         }                                                                                                                               \
         fe::launch(qkv_norm_rope_cache_kernel<TYPE>, T, threads, smem, stream, (const TYPE*)proj, ld, q_weight, k_weight, eps, positions, \
-                   inv_freq, rot, interleaved, v_inv_freq, slot_mapping, (TYPE*)kc, (TYPE*)vc, (TYPE*)q_out, heads, kv_heads, dim, vdim,    \
+                   inv_freq, rot, interleaved, v_inv_freq, bias, gain, slot_mapping, (TYPE*)kc, (TYPE*)vc, (TYPE*)q_out, heads, kv_heads, dim, vdim,    \
                    head, ps, num_slots, status);                                                                                        \
     } while (0)
     if (dtype == FE_F32) FE_LAUNCH_QKV_NORM(float);

@@ -30,17 +30,17 @@ extern "C" int fe_gemm_tcgen05(const void* x, const void* W, void* out, int M, i
 extern "C" int fe_paged_prefill_tcgen05(const void* q, long long q_stride, void* out, long long out_stride, const void* kc,
                                         const void* vc, const int* block_table, int bt_stride, const int* cu_q,
                                         const int* q_start, int requests, int max_q_len, int nq, int nkv, int d, int ps,
-                                        int num_pages, float scale, int window, int sink, int splits, void* scratch,
+                                        int num_pages, float scale, int window, int keep, int sink, int splits, void* scratch,
                                         long long total_tokens, int* status, const float* per_head, float softcap, cudaStream_t stream);
 extern "C" int fe_paged_prefill_mma(const void* q, long long q_stride, void* out, long long out_stride, const void* kc,
                                     const void* vc, const int* block_table, int bt_stride, const int* cu_q,
                                     const int* q_start, int requests, int max_q_len, int nq, int nkv, int d, int ps,
-                                    int num_pages, float scale, int window, int sink, int* status, const float* per_head, float softcap,
+                                    int num_pages, float scale, int window, int keep, int sink, int* status, const float* per_head, float softcap,
                                     cudaStream_t stream);
 extern "C" int fe_paged_decode_cluster(const void* q, long long q_stride, void* out, long long out_stride, const void* kc,
                                        const void* vc, const int* block_table, int bt_stride, const int* cu_q,
                                        const int* q_start, int requests, int nq, int nkv, int d, int ps, int num_pages,
-                                       float scale, int window, int sink, int splits, int* status, const float* per_head, float softcap,
+                                       float scale, int window, int keep, int sink, int splits, int* status, const float* per_head, float softcap,
                                        cudaStream_t stream);
 extern "C" int fe_paged_decode_mma(const void* q, long long q_stride, void* out, long long out_stride, void* scratch,
                                    const void* kc, const void* vc, const int* block_table, int bt_stride, const int* cu_q,
@@ -194,7 +194,7 @@ extern "C" int fe_layer_forward(const FeLayer* layer, const FeStep* step, void* 
     switch (S.attention) {
         case 0:
             rc = fe_paged_decode_cluster(qkv, Wq, heads, out_stride, k_cache, v_cache, S.block_table, S.bt_stride, S.cu_q,
-                                         S.q_start, S.R, L.nq, L.nkv, L.d, S.page_size, S.num_pages, L.scale, L.window, 0, S.splits,
+                                         S.q_start, S.R, L.nq, L.nkv, L.d, S.page_size, S.num_pages, L.scale, L.window, 0, 0, S.splits,
                                          S.status, nullptr, 0.f, stream);
             break;
         case 1:
@@ -205,12 +205,12 @@ extern "C" int fe_layer_forward(const FeLayer* layer, const FeStep* step, void* 
         case 2:
             rc = fe_paged_prefill_tcgen05(qkv, Wq, heads, out_stride, k_cache, v_cache, S.block_table, S.bt_stride, S.cu_q,
                                           S.q_start, S.R, S.max_q_len, L.nq, L.nkv, L.d, S.page_size, S.num_pages, L.scale,
-                                          L.window, 0, S.splits, S.attention_scratch, T, S.status, nullptr, 0.f, stream);
+                                          L.window, 0, 0, S.splits, S.attention_scratch, T, S.status, nullptr, 0.f, stream);
             break;
         case 3:
             rc = fe_paged_prefill_mma(qkv, Wq, heads, out_stride, k_cache, v_cache, S.block_table, S.bt_stride, S.cu_q,
                                       S.q_start, S.R, S.max_q_len, L.nq, L.nkv, L.d, S.page_size, S.num_pages, L.scale, L.window,
-                                      0, S.status, nullptr, 0.f, stream);
+                                      0, 0, S.status, nullptr, 0.f, stream);
             break;
         default:
             FE_REQUIRE(false, "layer_forward: unknown attention kind %d", S.attention);

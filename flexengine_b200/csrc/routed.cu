@@ -41,7 +41,8 @@ __device__ __forceinline__ float single_activation(float z, float which) {
 // the softmax over all logits; 1: the ``top`` largest logits are chosen and the weights are the softmax over those alone.
 // ``correction`` (one number per expert, may be null; over_chosen 0 only): added to the shares for the choice, not for the
 // weights.  ``groups`` > 1: the experts form that many equal groups of neighbours; a group's score is its largest (corrected)
-// share, and only experts of the ``keep`` best groups can be chosen (ties to the lower group).
+// share, and only experts of the ``keep`` best groups can be chosen (ties to the lower group).  over_chosen 2: no softmax; the
+// ``top`` largest logits are chosen and the weights are their sigmoids, not normalised.
 __global__ void route_top_kernel(const float* __restrict__ logits, int* __restrict__ chosen, float* __restrict__ weights,
                                  int T, int experts, int top, float scale, int over_chosen, const float* __restrict__ correction,
                                  int groups, int keep) {
@@ -118,16 +119,16 @@ __global__ void route_top_kernel(const float* __restrict__ logits, int* __restri
         }
         if (at >= experts) at = 0;                // nothing left to rank (logits that are not numbers): a weight of zero
         if (lane == 0) {
-            const float share = over_chosen ? expf(best - m) : best;      // m is the largest logit, the first one chosen
+            const float share = over_chosen == 2 ? 1.f / (1.f + expf(-best)) : over_chosen ? expf(best - m) : best;      // m is the largest logit, the first one chosen
             chosen[(size_t)t * top + c] = at;
             if (corrected) weights[(size_t)t * top + c] = share_of[at] * scale;
-            else weights[(size_t)t * top + c] = over_chosen ? share : share / sum * scale;
+            else weights[(size_t)t * top + c] = over_chosen == 2 ? share * scale : over_chosen ? share : share / sum * scale;
             chosen_sum += share;
             s[at] = -CUDART_INF_F;
         }
         __syncwarp();
     }
-    if (over_chosen && lane == 0) {
+    if (over_chosen == 1 && lane == 0) {
         const float inv = scale / chosen_sum;
         for (int c = 0; c < top; ++c) weights[(size_t)t * top + c] *= inv;
     }
@@ -194,7 +195,11 @@ __global__ void route_plan_kernel(const int* __restrict__ chosen, int pairs, int
 // The two grouped products.  Tile 64 rows x 64 columns, 16 of K a stage, 256 threads with 4 x 4 outputs each; float
 // accumulation in ascending k.  MODE 1 (GATED): columns n and n + F of the expert's matrix are taken together and
 // silu(gate) * up is written (compute type); MODE 2: an expert without a gate, single_activation is written (compute type);
-// MODE 0: the plain product is written in float.
+// MODE 0: the plain product is written in float.  ``row_weights`` (one per (token, choice) pair; null: 1) multiplies what an expert
+// reads: the products of the first kernel are multiplied by it before the activation.
+__device__ __forceinline__ float weight_of_row(const float* __restrict__ row_weights, const int* __restrict__ pair_of_row, int row) {
+    return row_weights ? row_weights[pair_of_row[row]] : 1.f;
+}
 namespace {
 constexpr int BM = 64, BN = 64, BK = 16, TM = 4, TN = 4;
 
@@ -202,7 +207,8 @@ template <typename T, int MODE>
 __global__ void __launch_bounds__(256)
 routed_product_kernel(const T* __restrict__ A, const int* __restrict__ pair_of_row, int top, const T* __restrict__ W,
                       void* __restrict__ out, const int* __restrict__ offsets, const int* __restrict__ tiles,
-                      const int* __restrict__ tile_expert, const int* __restrict__ tile_row0, int N, int K, float limit) {
+                      const int* __restrict__ tile_expert, const int* __restrict__ tile_row0, int N, int K, float limit,
+                          const float* __restrict__ row_weights) {
     griddep_wait();
     griddep_launch_dependents();
     constexpr bool GATED = MODE == 1;
@@ -264,16 +270,17 @@ routed_product_kernel(const T* __restrict__ A, const int* __restrict__ pair_of_r
     for (int i = 0; i < TM; ++i) {
         const int r = ty * TM + i;
         if (r >= rows) continue;
+        const float rw = MODE == 0 ? 1.f : weight_of_row(row_weights, pair_of_row, row0 + r);
 #pragma unroll
         for (int j = 0; j < TN; ++j) {
             const int gn = n0 + tx * TN + j;
             if (gn >= N) continue;
             const size_t at = (size_t)(row0 + r) * N + gn;
             if (GATED) {
-                const float g = acc[i][j];
-                reinterpret_cast<T*>(out)[at] = from_float<T>(expert_activation(g, acu[i][j], limit));
+                const float g = acc[i][j] * rw;
+                reinterpret_cast<T*>(out)[at] = from_float<T>(expert_activation(g, acu[i][j] * rw, limit));
             } else if (MODE == 2) {
-                reinterpret_cast<T*>(out)[at] = from_float<T>(single_activation(acc[i][j], limit));
+                reinterpret_cast<T*>(out)[at] = from_float<T>(single_activation(acc[i][j] * rw, limit));
             } else {
                 reinterpret_cast<float*>(out)[at] = acc[i][j];
             }
@@ -292,7 +299,8 @@ template <typename T, int MODE, int ROWS>
 __global__ void __launch_bounds__(FEW_WARPS * 32)
 routed_product_few_kernel(const T* __restrict__ A, const int* __restrict__ pair_of_row, int top, const T* __restrict__ W,
                           void* __restrict__ out, const int* __restrict__ offsets, const int* __restrict__ tiles,
-                          const int* __restrict__ tile_expert, const int* __restrict__ tile_row0, int N, int K, float limit) {
+                          const int* __restrict__ tile_expert, const int* __restrict__ tile_row0, int N, int K, float limit,
+                          const float* __restrict__ row_weights) {
     griddep_wait();
     griddep_launch_dependents();
     constexpr bool GATED = MODE == 1;
@@ -370,8 +378,9 @@ routed_product_few_kernel(const T* __restrict__ A, const int* __restrict__ pair_
 #pragma unroll
             for (int r = 0; r < ROWS; ++r) {
                 if (r >= rows) continue;
-                const float g = warp_sum(acc[c][r]);
-                const float u = GATED ? warp_sum(acu[c][r]) : 0.f;
+                const float rw = MODE == 0 ? 1.f : weight_of_row(row_weights, pair_of_row, row0 + r);
+                const float g = warp_sum(acc[c][r]) * rw;
+                const float u = GATED ? warp_sum(acu[c][r]) * rw : 0.f;
                 if (lane == 0 && nbase + c < N) {
                     const size_t at = (size_t)(row0 + r) * N + nbase + c;
                     if (GATED) reinterpret_cast<T*>(out)[at] = from_float<T>(expert_activation(g, u, limit));
@@ -404,8 +413,9 @@ routed_product_few_kernel(const T* __restrict__ A, const int* __restrict__ pair_
         }
 #pragma unroll
         for (int r = 0; r < ROWS; ++r) {
-            const float g = warp_sum(acc[r]);
-            const float u = GATED ? warp_sum(acu[r]) : 0.f;
+            const float rw = (MODE == 0 || r >= rows) ? 1.f : weight_of_row(row_weights, pair_of_row, row0 + r);
+            const float g = warp_sum(acc[r]) * rw;
+            const float u = GATED ? warp_sum(acu[r]) * rw : 0.f;
             if (lane == 0 && r < rows) {
                 const size_t at = (size_t)(row0 + r) * N + n;
                 if (GATED) reinterpret_cast<T*>(out)[at] = from_float<T>(expert_activation(g, u, limit));
@@ -424,7 +434,8 @@ template <int MODE, bool GATED = (MODE == 1)>
 __global__ void __launch_bounds__(128)
 routed_product_mma_kernel(const bf16* __restrict__ A, const int* __restrict__ pair_of_row, int top, const bf16* __restrict__ W,
                           void* __restrict__ out, const int* __restrict__ offsets, const int* __restrict__ tiles,
-                          const int* __restrict__ tile_expert, const int* __restrict__ tile_row0, int N, int K, float limit) {
+                          const int* __restrict__ tile_expert, const int* __restrict__ tile_row0, int N, int K, float limit,
+                          const float* __restrict__ row_weights) {
     using namespace nvcuda;
     griddep_wait();
     griddep_launch_dependents();
@@ -514,8 +525,9 @@ routed_product_mma_kernel(const bf16* __restrict__ A, const int* __restrict__ pa
                 const int r = wm * 32 + i * 16 + rr, gn = n0 + wn * 32 + j * 16 + cc;
                 if (r < rows && gn < N) {
                     const size_t at = (size_t)(row0 + r) * N + gn;
-                    const float g = stage[warp][0][rr][cc];
-                    if (GATED) reinterpret_cast<bf16*>(out)[at] = __float2bfloat16_rn(expert_activation(g, stage[warp][GATED ? 1 : 0][rr][cc], limit));
+                    const float rw = MODE == 0 ? 1.f : weight_of_row(row_weights, pair_of_row, row0 + r);
+                    const float g = stage[warp][0][rr][cc] * rw;
+                    if (GATED) reinterpret_cast<bf16*>(out)[at] = __float2bfloat16_rn(expert_activation(g, stage[warp][GATED ? 1 : 0][rr][cc] * rw, limit));
                     else if (MODE == 2) reinterpret_cast<bf16*>(out)[at] = __float2bfloat16_rn(single_activation(g, limit));
                     else reinterpret_cast<float*>(out)[at] = g;
                 }
@@ -542,7 +554,8 @@ template <int MODE, bool GATED = (MODE == 1)>
 __global__ void __launch_bounds__(256)
 routed_product_pipe_kernel(const bf16* __restrict__ A, const int* __restrict__ pair_of_row, int top, const bf16* __restrict__ W,
                            void* __restrict__ out, const int* __restrict__ offsets, const int* __restrict__ tiles,
-                           const int* __restrict__ tile_expert, const int* __restrict__ tile_row0, int N, int K, float limit) {
+                           const int* __restrict__ tile_expert, const int* __restrict__ tile_row0, int N, int K, float limit,
+                          const float* __restrict__ row_weights) {
     using namespace nvcuda;
     griddep_wait();
     griddep_launch_dependents();
@@ -637,8 +650,9 @@ routed_product_pipe_kernel(const bf16* __restrict__ A, const int* __restrict__ p
                 const int r = wm * 32 + i * 16 + rr, gn = n0 + wn * 32 + j * 16 + cc;
                 if (r < rows && gn < N) {
                     const size_t at = (size_t)(row0 + r) * N + gn;
-                    const float g = mine[rr * 20 + cc];
-                    if (GATED) reinterpret_cast<bf16*>(out)[at] = __float2bfloat16_rn(expert_activation(g, mine[16 * 20 + rr * 20 + cc], limit));
+                    const float rw = MODE == 0 ? 1.f : weight_of_row(row_weights, pair_of_row, row0 + r);
+                    const float g = mine[rr * 20 + cc] * rw;
+                    if (GATED) reinterpret_cast<bf16*>(out)[at] = __float2bfloat16_rn(expert_activation(g, mine[16 * 20 + rr * 20 + cc] * rw, limit));
                     else if (MODE == 2) reinterpret_cast<bf16*>(out)[at] = __float2bfloat16_rn(single_activation(g, limit));
                     else reinterpret_cast<float*>(out)[at] = g;
                 }
@@ -648,7 +662,7 @@ routed_product_pipe_kernel(const bf16* __restrict__ A, const int* __restrict__ p
 }
 
 // out[t] = sum_c weights[t][c] * y[row_of_pair[t top + c]] (+ shared[t]); a choice of an expert that returns its input
-// (row -2) adds weights[t][c] * h[t]
+// (row -2) adds weights[t][c] * h[t].  weights null: every y counts once (the experts' inputs were weighed)
 template <typename T>
 __global__ void routed_combine_kernel(const float* __restrict__ y, const int* __restrict__ row_of_pair,
                                       const float* __restrict__ weights, const T* __restrict__ shared, T* __restrict__ out,
@@ -660,8 +674,8 @@ __global__ void routed_combine_kernel(const float* __restrict__ y, const int* __
         float total = 0.f;
         for (int c = 0; c < top; ++c) {
             const int row = row_of_pair[(size_t)t * top + c];
-            if (row >= 0) total = fmaf(weights[(size_t)t * top + c], y[(size_t)row * D + j], total);
-            else if (row == -2 && h) total = fmaf(weights[(size_t)t * top + c], to_float(h[(size_t)t * D + j]), total);
+            if (row >= 0) total = fmaf(weights ? weights[(size_t)t * top + c] : 1.f, y[(size_t)row * D + j], total);
+            else if (row == -2 && h && weights) total = fmaf(weights[(size_t)t * top + c], to_float(h[(size_t)t * D + j]), total);
         }
         if (shared) total += to_float(shared[(size_t)t * D + j]);
         out[(size_t)t * D + j] = from_float<T>(total);
@@ -680,11 +694,15 @@ extern "C" long long fe_routed_experts_workspace(int T, int top, int experts, in
 // h [T, D]; chosen, weights [T, top]; gate_up [experts, 2F, D]; down [experts, D, F]; shared [T, D] or null; out [T, D].
 // limit: 0 for silu(gate) * up, else the clamped activation (see expert_activation).  single 1 or 2: the experts have no
 // gate, gate_up is [experts, F, D] and an expert is down(relu(up h)^2) (1) or down(gelu(up h)) (2, the exact form).  identity: choices in [experts, experts + identity) stand
-// for experts that return their input.
+// for experts that return their input.  weigh_input: the weights multiply what the experts read, and their outputs are plainly added.
 extern "C" int fe_routed_experts(const void* h, const int* chosen, const float* weights, const void* gate_up, const void* down,
                                  const void* shared, void* out, void* workspace, long long workspace_bytes, int T, int top,
                                  int experts, int D, int F, int dtype, float limit, int* status, int single, int identity,
-                                 cudaStream_t stream) {
+                                 int weigh_input, cudaStream_t stream) {
+    FE_REQUIRE(!weigh_input || identity == 0, "routed_experts: experts that return their input are weighed at their output");
+    const float* row_weights = weigh_input ? weights : nullptr;
+    const float* out_weights = weigh_input ? nullptr : weights;
+    const float* no_weights = nullptr;
     FE_REQUIRE(limit >= 0.f, "routed_experts: the activation's limit is 0 (plain silu) or positive");
     FE_REQUIRE(T >= 0 && top >= 1 && experts >= 1 && experts <= ROUTE_MAX_EXPERTS && D > 0 && F > 0, "routed_experts: bad sizes");
     FE_REQUIRE(dtype == FE_F32 || dtype == FE_BF16, "routed_experts: unknown dtype %d", dtype);
@@ -720,9 +738,9 @@ extern "C" int fe_routed_experts(const void* h, const int* chosen, const float* 
     const int *c_offsets = offsets, *c_tiles = tiles, *c_expert = tile_expert, *c_row0 = tile_row0;
 #define FE_ROUTED_PRODUCTS(KERNEL1, KERNEL2, TYPE, GRID1, GRID2, THREADS, SMEM1, SMEM2)                                                   \
     fe::launch(KERNEL1, GRID1, THREADS, SMEM1, stream, (const TYPE*)h, c_pairs, top, (const TYPE*)gate_up, (void*)act, c_offsets, c_tiles, \
-               c_expert, c_row0, F, D, act_of);                                                                                            \
+               c_expert, c_row0, F, D, act_of, row_weights);                                                                               \
     fe::launch(KERNEL2, GRID2, THREADS, SMEM2, stream, (const TYPE*)act, c_none, top, (const TYPE*)down, (void*)y, c_offsets, c_tiles,    \
-               c_expert, c_row0, D, F, 0.f)
+               c_expert, c_row0, D, F, 0.f, no_weights)
     if (few) {
         const int few_tiles = (int)((pairs + few_rows - 1) / few_rows + experts);
         const int per_block = FEW_WARPS * FEW_COLS;
@@ -775,10 +793,10 @@ extern "C" int fe_routed_experts(const void* h, const int* chosen, const float* 
     const int stretches = T >= 512 ? 1 : (D + threads - 1) / threads;          // few tokens: one column a thread
     const dim3 combine(T, stretches < 65535 ? stretches : 65535);
     if (dtype == FE_F32)
-        fe::launch(routed_combine_kernel<float>, combine, threads, 0, stream, (const float*)y, (const int*)row_of_pair, weights,
+        fe::launch(routed_combine_kernel<float>, combine, threads, 0, stream, (const float*)y, (const int*)row_of_pair, out_weights,
                    (const float*)shared, (float*)out, top, D, identity ? (const float*)h : (const float*)nullptr);
     else
-        fe::launch(routed_combine_kernel<bf16>, combine, threads, 0, stream, (const float*)y, (const int*)row_of_pair, weights,
+        fe::launch(routed_combine_kernel<bf16>, combine, threads, 0, stream, (const float*)y, (const int*)row_of_pair, out_weights,
                    (const bf16*)shared, (bf16*)out, top, D, identity ? (const bf16*)h : (const bf16*)nullptr);
     return fe_check_launch("routed_experts");
 }

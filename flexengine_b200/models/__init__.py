@@ -1,1 +1,1 @@
-from . import bebulorn, fedutar, fuvozen, fuvuvik, qwen2, rikolix  # noqa: F401  (register Bebulorn, Fedutar, Fuvozen, Fuvuvik, Rikolix and Qwen2ForCausalLM)
+from . import bebulorn, fedutar, fuvozen, fuvuvik, qwen2, ribozen, rikolix  # noqa: F401  (register Bebulorn, Fedutar, Fuvozen, Fuvuvik, Ribozen, Rikolix and Qwen2ForCausalLM)

@@ -182,13 +182,14 @@ def scale_softcap(logits, scale, cap):
     return logits
 
 
-def add_rmsnorm(residual, delta, weight, eps, out_dtype, rows=None, upcoming=None, post=None):
+def add_rmsnorm(residual, delta, weight, eps, out_dtype, rows=None, upcoming=None, post=None, delta_scale=None):
     """Fused residual add + RMSNorm.  rows=None: residual += delta in place (all rows) and every row
     is normalised; rows given: only those rows are read (residual[rows] + delta[rows]), nothing is
     written back.  ``upcoming``: the weight matrix that the next kernel streams; in a decode step extra
     blocks of this kernel, which barely touches memory, ask for its start to be brought into L2.
     ``post`` = (weight, eps, bias or None): the branch output goes through a norm of its own on its way into the stream,
-    w_b (delta + bias) / rms(delta + bias); delta may then be float32 whatever the compute dtype."""
+    w_b (delta + bias) / rms(delta + bias); delta may then be float32 whatever the compute dtype.  ``delta_scale`` (float32 [H]):
+    residual += delta_scale * delta; delta may then be float32 too."""
     if post is not None and delta is not None:
         T, H = residual.shape
         n_out = T if rows is None else rows.numel()
@@ -198,6 +199,17 @@ def add_rmsnorm(residual, delta, weight, eps, out_dtype, rows=None, upcoming=Non
     T, H = residual.shape
     if residual.dtype != torch.float32 or weight.dtype != torch.float32:
         raise TypeError("the residual stream and norm weights are float32")
+    if delta_scale is not None and delta is not None:
+        _need_cuda(delta_scale)
+        if delta.dtype not in (torch.float32, out_dtype) or delta.shape != residual.shape or not delta.is_contiguous() \
+                or delta_scale.dtype != torch.float32 or delta_scale.numel() != H or not residual.is_contiguous():
+            raise ValueError("add_rmsnorm: a scaled branch is contiguous, shaped like the residual, float32 or in the compute dtype; its "
+                             "scale float32 [H]")
+        n_out = T if rows is None else rows.numel()
+        out = torch.empty((n_out, H), dtype=out_dtype, device=residual.device)
+        _run(_core(), "fe_add_rmsnorm_scaled", _ptr(residual), _ptr(delta), _c_int(_code(delta.dtype)), _ptr(delta_scale), _ptr(weight),
+             _c_float(eps), _ptr(out), _ptr(rows), _c_int(n_out), _c_int(H), _c_int(T), _c_int(_code(out_dtype)), *_upcoming(upcoming, T), _stream())
+        return out
     if delta is not None and (delta.dtype != out_dtype or delta.shape != residual.shape or not delta.is_contiguous()):
         raise ValueError("add_rmsnorm: delta must be contiguous, shaped like the residual, in the compute dtype")
     n_out = T if rows is None else rows.numel()
@@ -311,8 +323,8 @@ def linear(x, w, bias=None, out_float32=False, follow=None, upcoming=None):
         return y if out_float32 or not wide else y.to(torch.bfloat16)
     if x.dim() != 2 or w.dim() != 2 or x.shape[1] != w.shape[1]:
         raise ValueError(f"linear: shapes {tuple(x.shape)} x {tuple(w.shape)}")
-    if not x.is_contiguous():
-        x = x.contiguous()
+    if not x.is_contiguous() and (w.dtype == torch.float32 or x.stride(1) != 1):
+        x = x.contiguous()                           # the library's products take rows of any stride
     if w.dtype == torch.float32:
         y = gemm_fp32(x if x.dtype == torch.float32 else x.float(), w, bias)
         return y if (out_float32 or x.dtype == torch.float32) else y.to(x.dtype)
@@ -536,14 +548,14 @@ def _score_map(sigmoid, head_bias, softcap, head_scales):
 
 def paged_attention_simt(q, q_stride, k_cache, v_cache, block_table, cu_q, q_start, token_request, T, nq, nkv, d,
                          page_size, scale, window, sink=False, sigmoid=False, head_bias=None, softcap=0.0,
-                         head_scales=None):
+                         head_scales=None, keep=0):
     out = torch.empty((T, nq * d), dtype=k_cache.dtype, device=k_cache.device)
     mapped, per_head, softcap = _score_map(sigmoid, head_bias, softcap, head_scales)
     mode = _attention_mode(sink, sigmoid, mapped)
     _run(_core(), "fe_paged_attention_simt", _ptr(q), _c_ll(q_stride), _ptr(out), _c_ll(nq * d), _ptr(k_cache),
          _ptr(v_cache), _ptr(block_table), _c_int(block_table.shape[1]), _ptr(cu_q), _ptr(q_start),
          _ptr(token_request), _c_int(T), _c_int(nq), _c_int(nkv), _c_int(d), _c_int(page_size),
-         _c_int(k_cache.shape[0]), _c_float(scale), _c_int(window), _c_int(mode), _c_int(_code(k_cache.dtype)),
+         _c_int(k_cache.shape[0]), _c_float(scale), _c_int(window), _c_int(keep), _c_int(mode), _c_int(_code(k_cache.dtype)),
          _ptr(status_word(k_cache.device)), _ptr(per_head), _c_float(softcap), _stream())
     return out
 
@@ -605,7 +617,7 @@ def decode_splits(requests: int, nkv: int, max_ctx_len: int, sms: int | None = N
 
 def paged_decode_mma(q, q_stride, k_cache, v_cache, block_table, cu_q, q_start, requests, nq, nkv, d, page_size,
                      scale, window, splits, out=None, upcoming=None, sink=False, sigmoid=False, head_bias=None, softcap=0.0,
-                     head_scales=None):
+                     head_scales=None, keep=0):
     """Tensor-core decode attention (one token per request), keys split ``splits`` ways.  ``upcoming``: the
     matrix that the next kernel streams (the output projection); extra blocks of the merge kernel ask for its
     start to be brought into L2."""
@@ -618,7 +630,7 @@ def paged_decode_mma(q, q_stride, k_cache, v_cache, block_table, cu_q, q_start, 
     _run(lib, "fe_paged_decode_mma_upcoming", _ptr(q), _c_ll(q_stride), _ptr(out), _c_ll(out.stride(0)), _ptr(work),
          _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _c_int(block_table.shape[1]), _ptr(cu_q), _ptr(q_start),
          _c_int(requests), _c_int(nq), _c_int(nkv), _c_int(d), _c_int(page_size), _c_int(k_cache.shape[0]),
-         _c_float(scale), _c_int(window), _c_int(_attention_mode(sink, sigmoid, mapped)), _c_int(splits),
+         _c_float(scale), _c_int(window), _c_int(keep), _c_int(_attention_mode(sink, sigmoid, mapped)), _c_int(splits),
          *_upcoming(upcoming, requests, UPCOMING_BYTES_MERGE),
          _ptr(status_word(k_cache.device)), _ptr(per_head), _c_float(softcap), _stream())
     return out
@@ -666,7 +678,7 @@ def decode_cluster_splits(splits: int, max_ctx_len: int, clusters: int = 0, resi
 
 def paged_decode_cluster(q, q_stride, k_cache, v_cache, block_table, cu_q, q_start, requests, nq, nkv, d, page_size,
                          scale, window, splits, out=None, sink=False, sigmoid=False, head_bias=None, softcap=0.0,
-                         head_scales=None):
+                         head_scales=None, keep=0):
     """Decode attention with the splits of each (request, key/value head) as one thread-block cluster that merges
     its partial results through distributed shared memory: one launch, no scratch memory; splits <= 16."""
     if out is None:
@@ -674,21 +686,21 @@ def paged_decode_cluster(q, q_stride, k_cache, v_cache, block_table, cu_q, q_sta
     mapped, per_head, softcap = _score_map(sigmoid, head_bias, softcap, head_scales)
     _run(_bf16(), "fe_paged_decode_cluster", _ptr(q), _c_ll(q_stride), _ptr(out), _c_ll(out.stride(0)), _ptr(k_cache),
          _ptr(v_cache), _ptr(block_table), _c_int(block_table.shape[1]), _ptr(cu_q), _ptr(q_start), _c_int(requests),
-         _c_int(nq), _c_int(nkv), _c_int(d), _c_int(page_size), _c_int(k_cache.shape[0]), _c_float(scale), _c_int(window),
+         _c_int(nq), _c_int(nkv), _c_int(d), _c_int(page_size), _c_int(k_cache.shape[0]), _c_float(scale), _c_int(window), _c_int(keep),
          _c_int(_attention_mode(sink, sigmoid, mapped)), _c_int(splits), _ptr(status_word(k_cache.device)), _ptr(per_head), _c_float(softcap), _stream())
     return out
 
 
 def paged_prefill_mma(q, q_stride, k_cache, v_cache, block_table, cu_q, q_start, T, requests, max_q_len, nq, nkv, d,
                       page_size, scale, window, sink=False, sigmoid=False, head_bias=None, softcap=0.0,
-                      head_scales=None):
+                      head_scales=None, keep=0):
     """Tensor-core attention for portions of any length (decoded tokens are portions of one)."""
     out = torch.empty((T, nq * d), dtype=torch.bfloat16, device=k_cache.device)
     mapped, per_head, softcap = _score_map(sigmoid, head_bias, softcap, head_scales)
     _run(_bf16(), "fe_paged_prefill_mma", _ptr(q), _c_ll(q_stride), _ptr(out), _c_ll(nq * d), _ptr(k_cache),
          _ptr(v_cache), _ptr(block_table), _c_int(block_table.shape[1]), _ptr(cu_q), _ptr(q_start), _c_int(requests),
          _c_int(max_q_len), _c_int(nq), _c_int(nkv), _c_int(d), _c_int(page_size), _c_int(k_cache.shape[0]),
-         _c_float(scale), _c_int(window), _c_int(_attention_mode(sink, sigmoid, mapped)), _ptr(status_word(k_cache.device)), _ptr(per_head),
+         _c_float(scale), _c_int(window), _c_int(keep), _c_int(_attention_mode(sink, sigmoid, mapped)), _ptr(status_word(k_cache.device)), _ptr(per_head),
          _c_float(softcap), _stream())
     return out
 
@@ -734,7 +746,7 @@ def prefill_splits(lengths, starts, nq, nkv, window=0, sms: int | None = None) -
 
 def paged_prefill_tcgen05(q, q_stride, k_cache, v_cache, block_table, cu_q, q_start, T, requests, max_q_len, nq, nkv, d,
                           page_size, scale, window, splits=1, sink=False, sigmoid=False, head_bias=None, softcap=0.0,
-                          head_scales=None):
+                          head_scales=None, keep=0):
     """Prefill attention on tcgen05 tensor cores: 128 (query, head) rows a block, head sizes 64 and 128.
     ``splits`` > 1 shares the keys of each pair of row tiles out over that many blocks and merges their results."""
     out = torch.empty((T, nq * d), dtype=torch.bfloat16, device=k_cache.device)
@@ -743,17 +755,17 @@ def paged_prefill_tcgen05(q, q_stride, k_cache, v_cache, block_table, cu_q, q_st
     _run(_bf16(), "fe_paged_prefill_tcgen05", _ptr(q), _c_ll(q_stride), _ptr(out), _c_ll(nq * d), _ptr(k_cache),
          _ptr(v_cache), _ptr(block_table), _c_int(block_table.shape[1]), _ptr(cu_q), _ptr(q_start), _c_int(requests),
          _c_int(max_q_len), _c_int(nq), _c_int(nkv), _c_int(d), _c_int(page_size), _c_int(k_cache.shape[0]),
-         _c_float(scale), _c_int(window), _c_int(_attention_mode(sink, sigmoid, mapped)), _c_int(splits), _ptr(part),
+         _c_float(scale), _c_int(window), _c_int(keep), _c_int(_attention_mode(sink, sigmoid, mapped)), _c_int(splits), _ptr(part),
          _c_ll(T), _ptr(status_word(k_cache.device)), _ptr(per_head), _c_float(softcap), _stream())
     return out
 
 
 def paged_attention(qkv, k_cache, v_cache, block_table, ctx, nq, nkv, d, page_size, scale, window, upcoming=None, sink=False,
-                    weights="softmax", head_bias=None, softcap=0.0, head_scales=None):
+                    weights="softmax", head_bias=None, softcap=0.0, head_scales=None, keep_first=0):
     """Causal grouped-query attention of the step's tokens over their requests' pages.
     qkv [T, >= nq d] holds the (rotated) queries in its first nq d columns; returns [T, nq d].
     ``window``: what a query sees of the earlier keys: 0 all of them, w > 0 the last w, -c < 0 those of its own chunk of
-    c positions (counted from position 0).  ``sink``: 1 is added to the softmax's denominator.
+    c positions (counted from position 0).  ``keep_first`` (with a window): the sequence's first so many keys are seen as well.  ``sink``: 1 is added to the softmax's denominator.
     ``weights`` "sigmoid": no softmax; a visible key weighs sigmoid(score + head_bias[head]) (``head_bias`` float32 [nq] or
     None), not normalised over the keys.  ``head_scales`` (float32 [nq]): scores are multiplied by the head's number as well as
     by ``scale``; ``softcap`` > 0: they then become softcap * tanh(score / softcap), before the softmax.
@@ -775,14 +787,16 @@ def paged_attention(qkv, k_cache, v_cache, block_table, ctx, nq, nkv, d, page_si
         _need_cuda(head_scales)
         if head_scales.dtype != torch.float32 or head_scales.numel() != nq:
             raise ValueError("paged_attention: head scales are float32 [heads]")
-    score = {"softcap": softcap, "head_scales": head_scales}
+    if keep_first < 0 or (keep_first and window <= 0):
+        raise ValueError("paged_attention: kept first keys go with a window")
+    score = {"softcap": softcap, "head_scales": head_scales, "keep": keep_first}
     if qkv.dtype == torch.float32 or d > 256:          # the tensor-core kernels take head sizes up to 256
         return paged_attention_simt(qkv, qkv.stride(0), k_cache, v_cache, block_table, ctx.cu_q, ctx.q_start,
                                     ctx.token_request, T, nq, nkv, d, page_size, scale, window, sink, sigmoid, head_bias, **score)
     requests = ctx.cu_q.numel() - 1
     if ctx.max_q_len == 1 and nq // nkv <= 16:
         # a window or a chunk bounds the keys a token walks (plus the tile of 32 that its first key lies in)
-        span = ctx.max_ctx_len if window == 0 else min(ctx.max_ctx_len, abs(window) + 31)
+        span = ctx.max_ctx_len if window == 0 else min(ctx.max_ctx_len, abs(window) + 31 + -(-keep_first // 32) * 32)
         splits = decode_splits(requests, nkv, span)
         clustered = decode_cluster_splits(splits, span, requests * nkv,
                                           lambda s: clusters_resident(requests, nq, nkv, d, s))
@@ -915,15 +929,16 @@ ROTATION_PAIRS = {"halves": 0, "interleaved": 1}
 
 
 def qkv_norm_rope_cache(projected, q_weight, k_weight, eps, positions, inv_freq, rot_dims, pairs, value_inv_freq, slot_mapping,
-                        k_cache, v_cache, heads, kv_heads, dim, vdim, head, page_size):
+                        k_cache, v_cache, heads, kv_heads, dim, vdim, head, page_size, bias=None, rot_gain=1.0):
     """What attention does between its projection and its scores, second form (csrc/hyper_ops.cu).  ``projected``
     [T, >= channels] holds q | k | v.  One RMS norm over the WHOLE query projection with ``q_weight`` (float32
     [heads dim]) and one over the whole key projection with ``k_weight`` ([kv_heads dim]; both None: no norm), then the
     first ``rot_dims`` entries of every query and key head turned by position * inv_freq, ``pairs`` "interleaved"
     (2i with 2i + 1) or "halves" (i with i + rot_dims/2); the values turned over all ``vdim`` entries by position *
     value_inv_freq (None: as they are); keys and values into their cache slots (slot_mapping None: no write) and the
-    queries returned [T, heads head], all padded with zeros to ``head``."""
-    _need_cuda(projected, q_weight, k_weight, positions, inv_freq, value_inv_freq, slot_mapping, k_cache, v_cache)
+    queries returned [T, heads head], all padded with zeros to ``head``.  ``bias`` (float32 [channels]) is added to q | k | v before
+    everything else; ``rot_gain`` multiplies the turned entries of queries and keys."""
+    _need_cuda(projected, q_weight, k_weight, positions, inv_freq, value_inv_freq, slot_mapping, k_cache, v_cache, bias)
     T = projected.shape[0]
     channels = (heads + kv_heads) * dim + kv_heads * vdim
     if projected.dim() != 2 or projected.shape[1] < channels or projected.stride(1) != 1:
@@ -941,10 +956,12 @@ def qkv_norm_rope_cache(projected, q_weight, k_weight, eps, positions, inv_freq,
         raise ValueError("value_inv_freq must be float32 [vdim / 2]")
     if pairs not in ROTATION_PAIRS:
         raise ValueError(f"unknown layout of rotation pairs {pairs!r}; known: {sorted(ROTATION_PAIRS)}")
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != channels):
+        raise ValueError("qkv_norm_rope_cache: the bias is float32 [channels]")
     queries = torch.empty((T, heads * head), dtype=projected.dtype, device=projected.device)
     _run(_core(), "fe_qkv_norm_rope_cache", _ptr(projected), _c_ll(projected.stride(0)), _ptr(q_weight), _ptr(k_weight), _c_float(eps),
          _ptr(positions), _ptr(inv_freq), _c_int(rot_dims if inv_freq is not None else 0), _c_int(ROTATION_PAIRS[pairs]),
-         _ptr(value_inv_freq), _ptr(slot_mapping), _ptr(k_cache), _ptr(v_cache), _ptr(queries), _c_int(T), _c_int(heads), _c_int(kv_heads),
+         _ptr(value_inv_freq), _ptr(bias), _c_float(rot_gain), _ptr(slot_mapping), _ptr(k_cache), _ptr(v_cache), _ptr(queries), _c_int(T), _c_int(heads), _c_int(kv_heads),
          _c_int(dim), _c_int(vdim), _c_int(head), _c_int(page_size), _c_ll(k_cache.shape[0] * page_size), _c_int(_code(projected.dtype)),
          _ptr(status_word(projected.device)), _stream())
     return queries
@@ -1315,6 +1332,163 @@ def delta_decode(projected, conv, state, history_at, state_slots, a_log, dt_bias
     return out
 
 
+# ---- scans with a decay and a weight per token: state-space layers, a matrix memory ------------------------------
+def _rows_ok(t, columns, dtype=torch.float32) -> bool:
+    return t.dim() == 2 and t.dtype == dtype and t.stride(1) == 1 and t.shape[1] >= columns
+
+
+def conv_silu(u, conv, bias, state, history_at, state_slots, cu_q, out_float32=False, steps=None, max_q_len=0):
+    """silu(bias + a causal convolution over time) of every channel of ``u`` [T, channels] (any row stride); ``conv`` float32
+    [taps, channels], tap by tap, the last the current token's; a request's last taps - 1 inputs lie in state[seat, history_at:]
+    (zeros and nothing kept for a seat below 0) and are brought up to date.  Rows come out in u's dtype.  ``steps`` = (rows
+    [T, heads], bias [heads], minus_a [heads]), float32: also float32 [2, T, heads] comes back, the logarithms of the decays
+    minus_a * dt and the step sizes dt = softplus(rows + bias) (csrc/state_space.cu).  Returns (rows, those or None)."""
+    _need_cuda(u, conv, bias, state, state_slots, cu_q)
+    T = u.shape[0]
+    taps, C = conv.shape
+    if u.dim() != 2 or u.shape[1] != C or u.stride(1) != 1 or conv.dtype != torch.float32 or not conv.is_contiguous() or bias.dtype != torch.float32 \
+            or bias.numel() != C or state.dtype != torch.float32 or state.stride(-1) != 1 or state.shape[-1] < history_at + (taps - 1) * C \
+            or (out_float32 and u.dtype != torch.float32):
+        raise ValueError("conv_silu: u [T, channels] with unit column stride, conv float32 [taps, channels], bias float32 [channels], a float32 "
+                         "state row that holds the history")
+    out = torch.empty((T, C), dtype=u.dtype, device=u.device)
+    rows = step_bias = minus_a = gates = None
+    heads = 0
+    if steps is not None:
+        rows, step_bias, minus_a = steps
+        heads = minus_a.numel()
+        _need_cuda(rows, step_bias, minus_a)
+        if not _rows_ok(rows, heads) or step_bias.dtype != torch.float32 or step_bias.numel() != heads or minus_a.dtype != torch.float32:
+            raise ValueError("conv_silu: the steps' rows are float32 [T, heads], bias and minus_a float32 [heads]")
+        gates = torch.empty((2, T, heads), dtype=torch.float32, device=u.device)
+    _run(_core(), "fe_conv_silu", _ptr(u), _c_ll(u.stride(0)), _c_int(_code(u.dtype)), _ptr(conv), _ptr(bias), _c_int(taps), _ptr(state),
+         _c_ll(state.stride(0)), _c_ll(history_at), _ptr(state_slots), _ptr(cu_q), _ptr(out), _c_int(_code(out.dtype)), _c_int(cu_q.numel() - 1),
+         _c_int(max_q_len or T), _c_int(C), _c_int(state.shape[0]), _ptr(rows), _c_ll(rows.stride(0) if rows is not None else 0),
+         _ptr(step_bias), _ptr(minus_a), _ptr(gates), _c_ll(T * heads), _c_int(heads), _stream())
+    return out, gates
+
+
+def memory_gates(rows, bias, cap, state, maxima_at, state_slots, cu_q, heads):
+    """The gates of a matrix memory: rows float32 [T, i | f] (any row stride), bias float32 [2 heads]; i = cap tanh((i + b) / cap),
+    f = log sigmoid(cap tanh((f + b) / cap)), m' = max(f + m, i) from token to token with m in state[seat, maxima_at:] (0 and
+    nothing kept for a seat below 0).  float32 [3, T, heads]: f + m - m', exp(i - m'), exp(-m') (csrc/head_scan.cu)."""
+    _need_cuda(rows, bias, state, state_slots, cu_q)
+    T = rows.shape[0]
+    if not _rows_ok(rows, 2 * heads) or bias.dtype != torch.float32 or bias.numel() != 2 * heads or state.dtype != torch.float32 \
+            or state.stride(-1) != 1 or state.shape[-1] < maxima_at + heads:
+        raise ValueError("memory_gates: rows float32 [T, 2 heads] with unit column stride, bias float32 [2 heads], a float32 state row")
+    gates = torch.empty((3, T, heads), dtype=torch.float32, device=rows.device)
+    _run(_core(), "fe_memory_gates", _ptr(rows), _c_ll(rows.stride(0)), _ptr(bias), _c_float(cap), _ptr(state), _c_ll(state.stride(0)),
+         _c_ll(maxima_at), _ptr(state_slots), _ptr(cu_q), _ptr(gates), _c_ll(T * heads), _c_int(cu_q.numel() - 1), _c_int(heads),
+         _c_int(state.shape[0]), _stream())
+    return gates
+
+
+def head_scan(q, k, v, gates, state, state_slots, cu_q, heads, groups, dim, vdim, query_scale=1.0, skip=None, divided=None, max_q_len=0):
+    """S <- exp(gates[0]) S + gates[1] k v^T, o = S^T (query_scale q) (+ skip v) per request and head over the step's tokens
+    (csrc/head_scan.cu); S [dim, vdim] float32 lives in state[seat, : heads dim vdim] (zeros and nothing kept for a seat below 0).
+    q, k float32 [T, groups dim], v float32 [T, heads vdim] (any row strides); head h reads group h // (heads / groups); gates float32
+    [2 or 3, T, heads], logarithms of the decays and weights; ``skip`` float32 [heads].  ``divided`` (a floor): a memory n [dim] of the
+    keys alone lies behind the heads' S, and o is divided by max(|n . q|, gates[2]) + floor.  Returns float32 [T, heads vdim]."""
+    _need_cuda(q, k, v, gates, state, state_slots, cu_q, skip)
+    T, requests = v.shape[0], cu_q.numel() - 1
+    per = heads * dim * vdim + (heads * dim if divided is not None else 0)
+    if not (_rows_ok(q, groups * dim) and _rows_ok(k, groups * dim) and _rows_ok(v, heads * vdim)) or gates.dtype != torch.float32 \
+            or tuple(gates.shape[1:]) != (T, heads) or gates.shape[0] < (2 if divided is None else 3) or not gates.is_contiguous() \
+            or state.dtype != torch.float32 or state.stride(-1) != 1 or state.shape[-1] < per \
+            or (skip is not None and (skip.dtype != torch.float32 or skip.numel() != heads)):
+        raise ValueError("head_scan: q, k float32 [T, groups dim], v float32 [T, heads vdim], gates float32 [2 or 3, T, heads], the state float32")
+    out = torch.empty((T, heads * vdim), dtype=torch.float32, device=v.device)
+    lib = _core()
+    if max_q_len == 1 and divided is None:
+        _run(lib, "fe_head_step", _ptr(q), _c_ll(q.stride(0)), _c_float(query_scale), _ptr(k), _c_ll(k.stride(0)), _ptr(v), _c_ll(v.stride(0)),
+             _ptr(gates), _c_ll(T * heads), _ptr(skip), _ptr(state), _c_ll(state.stride(0)), _ptr(state_slots), _ptr(out), _c_int(requests),
+             _c_int(heads), _c_int(groups), _c_int(dim), _c_int(vdim), _c_int(state.shape[0]), _stream())
+        return out
+    rows = T // lib.fe_head_scan_chunk_tokens() + requests
+    sums = torch.empty((rows, per), dtype=torch.float32, device=v.device)
+    totals = torch.empty((rows, heads), dtype=torch.float32, device=v.device)
+    _run(lib, "fe_head_scan", _ptr(q), _c_ll(q.stride(0)), _c_float(query_scale), _ptr(k), _c_ll(k.stride(0)), _ptr(v), _c_ll(v.stride(0)),
+         _ptr(gates), _c_ll(T * heads), _ptr(skip), _ptr(state), _c_ll(state.stride(0)), _ptr(state_slots), _ptr(cu_q), _ptr(out), _ptr(sums),
+         _ptr(totals), _c_int(requests), _c_int(max_q_len or T), _c_int(heads), _c_int(groups), _c_int(dim), _c_int(vdim),
+         _c_int(state.shape[0]), _c_int(0 if divided is None else 1), _c_float(divided or 0.0), _stream())
+    return out
+
+
+def memory_decode(projected, bias, cap, query_scale, floor, state, state_slots, norm_weight, eps, heads, dim, vdim, out_dtype):
+    """A step of ONE token a request of a matrix memory, everything between the projection and the output product in one kernel
+    (csrc/head_scan.cu): ``projected`` float32 [R, q | k | v | g | i | f]; ``memory_gates`` and ``head_scan`` divided with ``floor``, then
+    every head divided by its root mean square, times ``norm_weight`` (float32 [heads vdim]), times sigmoid(g)."""
+    _need_cuda(projected, bias, state, state_slots, norm_weight)
+    R = projected.shape[0]
+    if not _rows_ok(projected, 2 * heads * dim + 2 * heads * vdim + 2 * heads) or bias.dtype != torch.float32 or bias.numel() != 2 * heads \
+            or norm_weight.dtype != torch.float32 or norm_weight.numel() != heads * vdim or state.dtype != torch.float32 or state.stride(-1) != 1 \
+            or state.shape[-1] < heads * (dim * vdim + dim + 1) or state_slots.numel() < R:
+        raise ValueError("memory_decode: projected float32 [R, q | k | v | g | i | f], bias [2 heads], the norm weight [heads vdim], a seat per row")
+    out = torch.empty((R, heads * vdim), dtype=out_dtype, device=projected.device)
+    _run(_core(), "fe_memory_decode", _ptr(projected), _c_ll(projected.stride(0)), _ptr(bias), _c_float(cap), _c_float(query_scale),
+         _c_float(floor), _ptr(state), _c_ll(state.stride(0)), _ptr(state_slots), _ptr(norm_weight), _c_float(eps), _ptr(out), _c_int(R),
+         _c_int(heads), _c_int(dim), _c_int(vdim), _c_int(state.shape[0]), _c_int(_code(out_dtype)), _stream())
+    return out
+
+
+def gated_group_rmsnorm(y, z, weight, eps, groups, out_dtype):
+    """y silu(z), then each of ``groups`` equal parts of a row divided by its own root mean square, times ``weight``; y float32
+    [T, inner], z float32 (any row stride)."""
+    _need_cuda(y, z, weight)
+    T, inner = y.shape
+    if y.dtype != torch.float32 or not y.is_contiguous() or not _rows_ok(z, inner) or z.shape[0] != T or weight.dtype != torch.float32 \
+            or weight.numel() != inner or inner % groups:
+        raise ValueError("gated_group_rmsnorm: y and z float32 [T, inner], weight float32 [inner], groups equal parts")
+    out = torch.empty((T, inner), dtype=out_dtype, device=y.device)
+    _run(_core(), "fe_gated_group_rmsnorm", _ptr(y), _ptr(z), _c_ll(z.stride(0)), _ptr(weight), _c_float(eps), _ptr(out), _c_int(T),
+         _c_int(inner), _c_int(groups), _c_int(_code(out_dtype)), _stream())
+    return out
+
+
+def _selective_out(what, x, dt_bias, minus_a, skip, z, state, into):
+    (T, inner), N = x.shape, minus_a.shape[1]
+    if not x.is_contiguous() or tuple(minus_a.shape) != (inner, N) or not minus_a.is_contiguous() or not _rows_ok(z, inner, x.dtype) \
+            or any(t.dtype != torch.float32 for t in (dt_bias, minus_a, skip, state)) or dt_bias.numel() != inner or skip.numel() != inner \
+            or state.stride(-1) != 1 or state.shape[-1] < inner * N:
+        raise ValueError(f"{what}: x and z [T, inner] in one dtype, minus_a float32 [inner, N], bias, skip [inner] and the state float32")
+    out = into if into is not None else torch.empty((T, inner), dtype=x.dtype, device=x.device)
+    if tuple(out.shape) != (T, inner) or out.dtype != x.dtype or out.stride(1) != 1:
+        raise ValueError(f"{what}: the rows go to [T, inner] in the compute dtype with unit column stride")
+    return out
+
+
+def selective_scan(x, dt, dt_bias, minus_a, bc, skip, z, state, state_slots, cu_q, scale=1.0, into=None):
+    """dt <- softplus(dt + dt_bias); S[c, n] <- exp(dt_c minus_a[c, n]) S[c, n] + dt_c x_c B_n; y_c = sum_n S[c, n] C_n + skip_c x_c; y silu(z)
+    times ``scale``, per request over the step's tokens (csrc/state_space.cu); S [inner, N] float32 lives in state[seat, : inner N] (zeros
+    and nothing kept for a seat below 0).  x [T, inner], bc [T, B | C] and z in the compute dtype, dt float32 [T, inner]; ``into``: where
+    the rows go (a view with any row stride)."""
+    _need_cuda(x, dt, dt_bias, minus_a, bc, skip, z, state, state_slots, cu_q, into)
+    out = _selective_out("selective_scan", x, dt_bias, minus_a, skip, z, state, into)
+    (T, inner), N = x.shape, minus_a.shape[1]
+    if dt.dtype != torch.float32 or tuple(dt.shape) != (T, inner) or not dt.is_contiguous() or not _rows_ok(bc, 2 * N, x.dtype):
+        raise ValueError("selective_scan: dt is contiguous float32 [T, inner], bc [T, 2 N] in the compute dtype")
+    _run(_core(), "fe_selective_scan", _ptr(x), _ptr(dt), _ptr(dt_bias), _ptr(minus_a), _ptr(bc), _c_ll(bc.stride(0)), _ptr(skip), _ptr(z),
+         _c_ll(z.stride(0)), _ptr(state), _c_ll(state.stride(0)), _ptr(state_slots), _ptr(cu_q), _ptr(out), _c_ll(out.stride(0)), _c_float(scale),
+         _c_int(cu_q.numel() - 1), _c_int(inner), _c_int(N), _c_int(state.shape[0]), _c_int(_code(x.dtype)), _stream())
+    return out
+
+
+def selective_decode(x, low, dt_weight, dt_bias, minus_a, skip, z, state, state_slots, scale=1.0, into=None):
+    """``selective_scan`` for a step of ONE token a request, with the step sizes' projection in the same kernel: low [R, rank | B | C],
+    dt = softplus(dt_weight low + dt_bias), dt_weight [inner, rank] in the compute dtype."""
+    _need_cuda(x, low, dt_weight, dt_bias, minus_a, skip, z, state, state_slots, into)
+    out = _selective_out("selective_decode", x, dt_bias, minus_a, skip, z, state, into)
+    (R, inner), N, rank = x.shape, minus_a.shape[1], dt_weight.shape[1]
+    if not _rows_ok(low, rank + 2 * N, x.dtype) or tuple(dt_weight.shape) != (inner, rank) or dt_weight.dtype != x.dtype or not dt_weight.is_contiguous() \
+            or state_slots.numel() < R:
+        raise ValueError("selective_decode: low [R, rank + 2 N] and dt_weight [inner, rank] in the compute dtype, a seat per row")
+    _run(_core(), "fe_selective_decode", _ptr(x), _ptr(low), _c_ll(low.stride(0)), _ptr(dt_weight), _ptr(dt_bias), _ptr(minus_a), _ptr(skip),
+         _ptr(z), _c_ll(z.stride(0)), _ptr(state), _c_ll(state.stride(0)), _ptr(state_slots), _ptr(out), _c_ll(out.stride(0)), _c_float(scale),
+         _c_int(R), _c_int(inner), _c_int(N), _c_int(rank), _c_int(state.shape[0]), _c_int(_code(x.dtype)), _stream())
+    return out
+
+
 # ---- attention over a cached latent ------------------------------------------------------------------------------
 def batched_linear(x, w, token_major=False):
     """x [B, M, K] (a view with any row and batch strides, unit stride along K) times w [B, N, K]^T, one small matrix a
@@ -1369,12 +1543,13 @@ def latent_prepare(q, q_latent, down, norm_weight, eps, positions, inv_freq, rot
 
 
 # ---- a routed feed-forward ---------------------------------------------------------------------------------------
-def route_top(logits, top, scale, over_chosen=False, correction=None, groups=(1, 1)):
+def route_top(logits, top, scale, over_chosen=False, correction=None, groups=(1, 1), sigmoid=False):
     """(int32 [T, top], float32 [T, top]): per token the ``top`` largest softmax scores over all experts (float32, ties
     to the lower index) times ``scale``, and their experts.  ``over_chosen``: the ``top`` largest logits are chosen and the
     weights are the softmax over those alone (times ``scale``).  ``correction`` (float32, a number per expert) is added to
     the scores for the choice only.  ``groups`` = (count, keep): the experts form ``count`` equal groups of neighbours, a
-    group's score is its largest (corrected) score, and only experts of the ``keep`` best groups can be chosen."""
+    group's score is its largest (corrected) score, and only experts of the ``keep`` best groups can be chosen.  ``sigmoid``: the
+    scores are the sigmoids of the logits, and the weights the chosen scores, not normalised (times ``scale``)."""
     _need_cuda(logits, correction)
     T, experts = logits.shape
     if logits.dtype != torch.float32 or not logits.is_contiguous():
@@ -1385,7 +1560,7 @@ def route_top(logits, top, scale, over_chosen=False, correction=None, groups=(1,
     chosen = torch.empty((T, top), dtype=torch.int32, device=logits.device)
     weights = torch.empty((T, top), dtype=torch.float32, device=logits.device)
     _run(_core(), "fe_route_top", _ptr(logits), _ptr(chosen), _ptr(weights), _c_int(T), _c_int(experts), _c_int(top),
-         _c_float(scale), _c_int(1 if over_chosen else 0), _ptr(correction), _c_int(count), _c_int(keep), _stream())
+         _c_float(scale), _c_int(2 if sigmoid else 1 if over_chosen else 0), _ptr(correction), _c_int(count), _c_int(keep), _stream())
     return chosen, weights
 
 
@@ -1403,7 +1578,7 @@ def routed_tcgen05_ok(h, pairs, H, F) -> bool:
             and min(H, F) >= ROUTED_TCGEN05_MIN_K and h.data_ptr() % 16 == 0)
 
 
-def _routed_experts_tcgen05(h, chosen, weights, gate_up, down, shared, limit=0.0, single=None, identity=0):
+def _routed_experts_tcgen05(h, chosen, weights, gate_up, down, shared, limit=0.0, single=None, identity=0, weigh_input=False):
     """The routed feed-forward with its products on tcgen05 tensor cores: plan (counting sort, row tiles of 128 per
     expert), the rows of h gathered into sorted order, gate/up with the activation in the epilogue, down into float32,
     combination.  Everything stays on the device."""
@@ -1426,24 +1601,26 @@ def _routed_experts_tcgen05(h, chosen, weights, gate_up, down, shared, limit=0.0
          _ptr(offsets[experts:]), _stream())
     act = torch.empty((pairs, F), dtype=torch.bfloat16, device=dev)
     _run(tensor, "fe_gemm_tcgen05_grouped", _ptr(rows), _ptr(gate_up), _ptr(act), _c_int(pairs), _c_int(experts), _c_int(F if single else 2 * F),
-         _c_int(H), _c_int(SINGLE_EPILOGUES[single] if single else EPI_SWIGLU), _ptr(tiles), _ptr(tile_expert), _ptr(tile_row0), _ptr(offsets), _c_float(limit), _ptr(status), _stream())
+         _c_int(H), _c_int(SINGLE_EPILOGUES[single] if single else EPI_SWIGLU), _ptr(tiles), _ptr(tile_expert), _ptr(tile_row0), _ptr(offsets), _c_float(limit),
+         _ptr(weights) if weigh_input else None, _ptr(pair_of_row), _ptr(status), _stream())
     y = torch.empty((pairs, H), dtype=torch.float32, device=dev)
     _run(tensor, "fe_gemm_tcgen05_grouped", _ptr(act), _ptr(down), _ptr(y), _c_int(pairs), _c_int(experts), _c_int(H), _c_int(F),
-         _c_int(EPI_F32), _ptr(tiles), _ptr(tile_expert), _ptr(tile_row0), _ptr(offsets), _c_float(0.0), _ptr(status), _stream())
+         _c_int(EPI_F32), _ptr(tiles), _ptr(tile_expert), _ptr(tile_row0), _ptr(offsets), _c_float(0.0), None, None, _ptr(status), _stream())
     out = torch.empty((T, H), dtype=h.dtype, device=dev)
-    _run(core, "fe_routed_combine", _ptr(y), _ptr(row_of_pair), _ptr(weights), _ptr(shared), _ptr(out), _c_int(T), _c_int(top),
+    _run(core, "fe_routed_combine", _ptr(y), _ptr(row_of_pair), None if weigh_input else _ptr(weights), _ptr(shared), _ptr(out), _c_int(T), _c_int(top),
          _c_int(H), _c_int(_code(h.dtype)), _ptr(h) if identity else None, _stream())
     return out
 
 
-def routed_experts(h, chosen, weights, gate_up, down, shared=None, activation="silu", limit=0.0, identity=0):
+def routed_experts(h, chosen, weights, gate_up, down, shared=None, activation="silu", limit=0.0, identity=0, weigh_input=False):
     """out[t] = sum_c weights[t, c] * down_e( silu(gate_e h_t) * up_e h_t ) with e = chosen[t, c], plus ``shared`` [T, H] if
     given; gate_up [experts, 2F, H] ([gate; up] per expert), down [experts, H, F].  ``activation`` "clamped": with
     g = min(gate_e h_t, limit) and u = clamp(up_e h_t, -limit, limit) an expert is down_e( g sigmoid(1.702 g) (u + 1) ).
     The (token, choice) pairs are sorted by expert on the device and every expert multiplies its own rows (csrc/routed.cu):
     nothing comes back to the host.  ``activation`` "relu2", "gelu": experts without a gate; ``gate_up`` is then [experts, F, H]
     and an expert is down_e( act(up_e h_t) ), act the square of relu or the exact GELU.  ``identity``: choices in [experts, experts + identity) stand for experts that
-    return their input: out[t] += weight * h_t."""
+    return their input: out[t] += weight * h_t.  ``weigh_input``: the weights multiply what the experts read, expert(weight * h), and
+    their outputs are plainly added."""
     _need_cuda(h, chosen, weights, gate_up, down, shared)
     T, H = h.shape
     experts, F2, _ = gate_up.shape
@@ -1458,14 +1635,15 @@ def routed_experts(h, chosen, weights, gate_up, down, shared=None, activation="s
         raise ValueError("routed_experts: the activation is 'silu', 'relu2', 'gelu' or 'clamped' with a positive limit")
     limit = float(limit) if activation == "clamped" else 0.0
     if routed_tcgen05_ok(h, T * top, H, F):
-        return _routed_experts_tcgen05(h, chosen, weights, gate_up, down, shared, limit, single, identity)
+        return _routed_experts_tcgen05(h, chosen, weights, gate_up, down, shared, limit, single, identity, weigh_input)
     lib = _core()
     need = lib.fe_routed_experts_workspace(_c_int(T), _c_int(top), _c_int(experts), _c_int(H), _c_int(F), _c_int(_code(h.dtype)))
     work = torch.empty(need, dtype=torch.uint8, device=h.device)
     out = torch.empty((T, H), dtype=h.dtype, device=h.device)
     _run(lib, "fe_routed_experts", _ptr(h), _ptr(chosen), _ptr(weights), _ptr(gate_up), _ptr(down), _ptr(shared), _ptr(out),
          _ptr(work), _c_ll(need), _c_int(T), _c_int(top), _c_int(experts), _c_int(H), _c_int(F), _c_int(_code(h.dtype)),
-         _c_float(limit), _ptr(status_word(h.device)), _c_int(1 + ROUTED_SINGLE.index(single) if single else 0), _c_int(identity), _stream())
+         _c_float(limit), _ptr(status_word(h.device)), _c_int(1 + ROUTED_SINGLE.index(single) if single else 0), _c_int(identity),
+         _c_int(1 if weigh_input else 0), _stream())
     return out
 
 

@@ -117,6 +117,11 @@ class GatedAttentionMixer(Mixer):
     ``value_norm``: every value head is divided by its root mean square over ``vdim`` (``eps`` inside the root) and cached so.
     ``head_scales``: scores are multiplied by a learned number per query head as well as by ``scale``.
     ``softcap`` > 0: scores, scaled, then become softcap * tanh(score / softcap).
+    ``bias``: the projections of q, k and v have biases (``qkv.bias``; with ``norm_scope`` "all").
+    ``rot_scaling`` = (factor, original, fast, slow) (with ``norm_scope`` "all"): the rotation's frequencies as YaRN blends them: pairs
+    that turn more than ``fast`` times over ``original`` positions keep theirs, pairs that turn less than ``slow`` times have
+    theirs divided by ``factor``, with a ramp between, and the turned entries are multiplied by 0.1 ln(factor) + 1.
+    ``keep_first`` (mask "window"): a query also sees the first so many keys of its sequence, however far back they are.
 
     q, k, v and the head gates are one product; convolution, rotation, unit norm and the cache write are one kernel;
     angles, norms, scores and softmax are float32."""
@@ -131,7 +136,8 @@ class GatedAttentionMixer(Mixer):
                  rot_dims: int = 0, conv: int = 0, qk_norm: bool = False, eps: float = 1e-6, mask: str = "full", mask_size: int = 0,
                  sink: bool = False, conv_group: int = -1, conv_slot: int = -1, norm_weights: bool = False, temp_coef: float = 0.0,
                  temp_every: int = 1, gate: str = "head", norm_scope: str = "head", rot_pairs: str = "halves", rotate_values: bool = False,
-                 weights: str = "softmax", value_norm: bool = False, head_scales: bool = False, softcap: float = 0.0):
+                 weights: str = "softmax", value_norm: bool = False, head_scales: bool = False, softcap: float = 0.0, bias: bool = False,
+                 rot_scaling=None, keep_first: int = 0):
         if heads % kv_heads:
             raise ValueError("Invalid GQA head ratio")
         if mask not in self.MASKS or (mask != "full" and mask_size <= 0):
@@ -168,6 +174,15 @@ class GatedAttentionMixer(Mixer):
             raise ValueError("the value norm goes with neither a norm over the whole projection, nor neighbouring pairs, nor turned values")
         if self.softcap < 0.0 or ((self.softcap > 0.0 or self.has_head_scales) and weights == "sigmoid"):
             raise ValueError("softcap and head scales belong to a softmax; softcap is not negative")
+        self.has_bias, self.keep_first = bool(bias), int(keep_first)
+        self.rot_scaling = None if rot_scaling is None else tuple(float(x) for x in rot_scaling)
+        if (self.has_bias or self.rot_scaling is not None) and not self.wide_prepare:
+            raise ValueError("biases and a scaled rotation go with a norm over the whole projection, neighbouring pairs or turned values")
+        if self.rot_scaling is not None and self.rotate_values:
+            raise ValueError("a scaled rotation does not turn values")
+        if self.keep_first < 0 or (self.keep_first and mask != "window"):
+            raise ValueError("keep_first belongs to a window")
+        self.qkv_bias = None
         self.score_bias = self.head_scales = None
         self._inv_freq_v = {}
         if self.temp_every < 1:
@@ -209,6 +224,8 @@ class GatedAttentionMixer(Mixer):
             every = self.norm_scope == "all"
             shapes["q_norm.weight"] = ((self.heads * self.dim if every else self.dim,), "vector")
             shapes["k_norm.weight"] = ((self.kv_heads * self.dim if every else self.dim,), "vector")
+        if self.has_bias:
+            shapes["qkv.bias"] = ((self.channels,), "vector")
         if self.weights == "sigmoid":
             shapes["score_bias"] = ((self.heads,), "vector")
         if self.has_head_scales:
@@ -224,15 +241,32 @@ class GatedAttentionMixer(Mixer):
         return self.qkvg_weight
 
     def cache_need(self):
-        return {"kind": self.mask, "kv_heads": self.kv_heads, "head_dim": self.head, "window": self.mask_size}
+        return {"kind": self.mask, "kv_heads": self.kv_heads, "head_dim": self.head, "window": self.mask_size, "keep": self.keep_first}
 
     def inverse_frequencies(self, device):
         key = str(device)
         if key not in self._inv_freq:
             i = torch.arange(self.rot_dims // 2, dtype=torch.float64)
             table = torch.pow(torch.tensor(self.rot_base, dtype=torch.float64), -2.0 * i / max(self.rot_dims, 1))
+            if self.rot_scaling is not None:
+                table = self._blended(table)
             self._inv_freq[key] = table.to(torch.float32).to(device).contiguous()
         return self._inv_freq[key]
+
+    def _blended(self, table):
+        factor, original, fast, slow = self.rot_scaling
+        dims = self.rot_dims
+
+        def place(turns):                 # the (fractional) pair that turns so many times over the original length
+            return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.rot_base))
+
+        lo, hi = max(math.floor(place(fast)), 0), min(math.ceil(place(slow)), dims - 1)
+        ramp = ((torch.arange(dims // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        return table / factor * ramp + table * (1.0 - ramp)
+
+    @property
+    def rot_gain(self) -> float:
+        return 1.0 if self.rot_scaling is None else 0.1 * math.log(self.rot_scaling[0]) + 1.0
 
     def value_inverse_frequencies(self, device):
         """The values' rotation: pair m of ``vdim`` / 2 turns by position * rot_base^(-2m/vdim)."""
@@ -263,12 +297,17 @@ class GatedAttentionMixer(Mixer):
             more.update(temp=(self.temp_coef, self.temp_every))
         if self.value_norm:
             more.update(value_norm=True)
+        wide = {}
+        if self.has_bias:
+            wide.update(bias=self.qkv_bias)
+        if self.rot_scaling is not None:
+            wide.update(rot_gain=self.rot_gain)
         turned = self.value_inverse_frequencies(projected.device) if self.rotate_values else None
         if self.wide_prepare:
             queries = ops.qkv_norm_rope_cache(
                 projected, self.q_norm_weight, self.k_norm_weight, self.eps, ctx.positions,
                 self.inverse_frequencies(projected.device) if self.rot_dims else None, self.rot_dims, self.rot_pairs, turned,
-                slot_mapping, k_cache, v_cache, self.heads, self.kv_heads, self.dim, self.vdim, self.head, group.page_size)
+                slot_mapping, k_cache, v_cache, self.heads, self.kv_heads, self.dim, self.vdim, self.head, group.page_size, **wide)
         else:
             queries = ops.qkv_conv_rope_norm_cache(
                 projected, self._conv_by_tap, history, self.conv, ctx.state_slots, ctx.cu_q, ctx.token_request, ctx.positions,
@@ -281,6 +320,8 @@ class GatedAttentionMixer(Mixer):
                                         group.page_size, self.scale, visibility, weights="sigmoid", head_bias=self.score_bias)
         else:
             scores = {"softcap": self.softcap, "head_scales": self.head_scales} if self.softcap > 0.0 or self.has_head_scales else {}
+            if self.keep_first:
+                scores.update(keep_first=self.keep_first)
             mixed = ops.paged_attention(queries, k_cache, v_cache, group.block_table, ctx, self.heads, self.kv_heads, self.head,
                                         group.page_size, self.scale, visibility, sink=self.sink, **scores)
         head = self.head

@@ -114,6 +114,53 @@ class PreNormBlock:
         return part.forward(*args, follow=follow)
 
 
+class ChannelScale:
+    """A learned number per channel that a branch's output is multiplied by; a part, so that it is bound by name."""
+
+    def __init__(self, hidden_size: int):
+        self.hidden_size = int(hidden_size)
+        self.weight = None
+
+    def parameter_shapes(self) -> dict:
+        return {"weight": ((self.hidden_size,), "vector")}
+
+    def bind(self, tensors: dict) -> None:
+        from .base import Part
+        Part.bind(self, tensors)
+
+    def reads_first(self):
+        return None
+
+
+class ScaledPreNormBlock:
+    """The pre-norm arrangement with a learned number per channel on every branch (layer scale):
+        x <- x + s1 * mixer(norm1(x));  x <- x + s2 * feed_forward(norm2(x))   (the second where the layer has one).
+    A branch's output is handed on as ``pending`` (``ScaledBranch``): the kernel of the norm that reads the stream next
+    multiplies and adds it."""
+
+    def __init__(self, layer_spec):
+        width = int(dict(layer_spec.block_params)["hidden_size"])
+        self.input_norm = build_part("norm", layer_spec.norm)
+        self.mixer, self.mixer_scale = build_part("mixer", layer_spec.mixer), ChannelScale(width)
+        self.feed_forward = build_part("feed_forward", layer_spec.feed_forward) if layer_spec.feed_forward is not None else None
+        self.part_names = ("input_norm", "mixer", "mixer_scale")
+        if self.feed_forward is not None:
+            self.post_mixer_norm, self.feed_forward_scale = build_part("norm", layer_spec.norm), ChannelScale(width)
+            self.part_names += ("post_mixer_norm", "feed_forward", "feed_forward_scale")
+
+    def parts(self) -> dict:
+        return {name: getattr(self, name) for name in self.part_names}
+
+    def forward(self, ctx, residual, pending, entry):
+        from .norm import ScaledBranch
+        h = _norm(self.input_norm, ctx, residual, pending, self.mixer.reads_first())
+        pending = ScaledBranch(self.mixer.forward(ctx, h, entry), self.mixer_scale.weight)
+        if self.feed_forward is None:
+            return pending
+        h = _norm(self.post_mixer_norm, ctx, residual, pending, self.feed_forward.reads_first())
+        return ScaledBranch(self.feed_forward.forward(ctx, h), self.feed_forward_scale.weight)
+
+
 def _norm(norm, ctx, residual, delta, upcoming):
     """A norm of another kind need not know the hint: it is passed only to a ``forward`` that names it."""
     if upcoming is not None and _accepts(norm.forward, "upcoming"):
@@ -255,6 +302,7 @@ class SandwichBlock:
 
 
 register_block("prenorm", PreNormBlock)
+register_block("scaled_prenorm", ScaledPreNormBlock)
 register_block("sandwich", SandwichBlock)
 register_block("hyper_gated", HyperGatedBlock)
 register_block("parallel_depth_average", ParallelDepthAverageBlock)

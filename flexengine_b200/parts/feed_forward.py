@@ -102,13 +102,13 @@ class RoutedExperts(FeedForward):
     none) that every token runs.  Tokens are sorted by expert on the device and each expert multiplies its own
     rows (``ops.routed_experts``): no count ever comes back to the host, so the step can be a CUDA graph."""
 
-    ROUTERS = ("softmax_all", "softmax_chosen")
+    ROUTERS = ("softmax_all", "softmax_chosen", "sigmoid")
     ACTIVATIONS = ("silu", "clamped", "relu2", "gelu")
     SINGLE = ("relu2", "gelu")            # experts (and a shared one) without a gate: one matrix up, one down
 
     def __init__(self, hidden_size: int, experts: int, top: int, expert_size: int, scale: float = 1.0, shared_size: int = 0,
                  router: str = "softmax_all", activation: str = "silu", limit: float = 0.0, identity: int = 0,
-                 correction: bool = False, groups: int = 1, keep: int = 1):
+                 correction: bool = False, groups: int = 1, keep: int = 1, weigh: str = "output"):
         """``router`` "softmax_all": as above; "softmax_chosen": the ``top`` largest logits are chosen and the weights are
         the softmax over the chosen logits only (the same as the softmax over all, divided by the sum of the chosen shares).  ``activation`` "silu": as above; "clamped": with g = min(gate h, limit)
         and u = clamp(up h, -limit, limit) an expert is down( g * sigmoid(1.702 g) * (u + 1) ); "relu2", "gelu": an expert (and
@@ -117,7 +117,9 @@ class RoutedExperts(FeedForward):
         their input (times the weight); they have no tensors.  ``correction``: a learned number per router output is added
         to the scores for the choice only; the weights are the uncorrected scores.  ``groups``, ``keep``: the router's
         outputs form ``groups`` equal groups of neighbours, a group's score is its largest (corrected) score, and only
-        outputs of the ``keep`` best groups can be chosen."""
+        outputs of the ``keep`` best groups can be chosen.  ``router`` "sigmoid": the scores are sigmoid(z), the ``top`` largest are
+        chosen and used as weights as they are (times ``scale``).  ``weigh`` "input": a weight multiplies what its expert reads, not
+        what it returns: the output is the plain sum of expert(weight * h)."""
         self.hidden_size, self.experts, self.top = int(hidden_size), int(experts), int(top)
         self.expert_size, self.scale, self.shared_size = int(expert_size), float(scale), int(shared_size)
         if router not in self.ROUTERS or activation not in self.ACTIVATIONS:
@@ -131,6 +133,9 @@ class RoutedExperts(FeedForward):
             raise ValueError("the groups must share the router's outputs out equally, and 1 <= keep <= groups")
         if (self.correction or self.groups > 1) and router != "softmax_all":
             raise ValueError("a correction and groups go with the softmax over all router outputs")
+        if weigh not in ("output", "input") or (weigh == "input" and self.identity):
+            raise ValueError("weights multiply an expert's 'output' or its 'input'; experts that return their input take 'output'")
+        self.weigh = weigh
         self.single = activation in self.SINGLE
         self.router_weight = self.router_correction = self.experts_gate_up_weight = self.experts_up_weight = self.experts_down_weight = None
         self.shared_gate_up_weight = self.shared_up_weight = self.shared_down_weight = None
@@ -165,6 +170,13 @@ class RoutedExperts(FeedForward):
         elif self.shared_size:
             shared = ops.linear(ops.linear_swiglu(h, self.shared_gate_up_weight, self.shared_size), self.shared_down_weight)
         down = self.experts_down_weight.view(e, d, f)
+        if self.router == "sigmoid" or self.weigh == "input":
+            options = {"sigmoid": True} if self.router == "sigmoid" else {"over_chosen": self.router == "softmax_chosen"}
+            chosen, weights = ops.route_top(logits, self.top, self.scale, correction=self.router_correction, groups=(self.groups, self.keep),
+                                            **options)
+            first = self.experts_up_weight.view(e, f, d) if self.single else self.experts_gate_up_weight.view(e, 2 * f, d)
+            return ops.routed_experts(h, chosen, weights, first, down, shared, activation=self.activation, limit=self.limit,
+                                      identity=self.identity, weigh_input=self.weigh == "input")
         if self.single or self.identity or self.correction or self.groups > 1:
             chosen, weights = ops.route_top(logits, self.top, self.scale, over_chosen=self.router == "softmax_chosen",
                                             correction=self.router_correction, groups=(self.groups, self.keep))

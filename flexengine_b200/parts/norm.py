@@ -26,6 +26,15 @@ class PostNormed:
         self.norm_bias, self.scale, self.plus = norm_bias, float(scale), plus
 
 
+class ScaledBranch:
+    """A branch's output on its way into the residual stream times a learned number per channel: the stream receives
+    weight * y.  The kernel of the norm that reads the stream next does it.  ``y`` is float32 or in the compute dtype."""
+    __slots__ = ("y", "weight")
+
+    def __init__(self, y, weight):
+        self.y, self.weight = y, weight
+
+
 class RMSNorm(Norm):
     """``unit_offset``: the checkpoint stores the weight around zero and the norm multiplies by (1 + w).  The sum is taken
     once, in float32, when the weights are bound; the kernels see a plain weight."""
@@ -45,6 +54,8 @@ class RMSNorm(Norm):
             self.weight = self.weight.to(torch.float32) + 1.0
 
     def forward(self, ctx, residual, delta, rows=None, upcoming=None):
+        if isinstance(delta, ScaledBranch):
+            return ctx.ops.add_rmsnorm(residual, delta.y, self.weight, self.eps, ctx.dtype, rows, upcoming=upcoming, delta_scale=delta.weight)
         if isinstance(delta, PostNormed):
             # the branch before ends in a norm of its own (a layer with norms on both sides of a sublayer): one kernel
             # norms the branch's output, adds it to the stream and norms the sum

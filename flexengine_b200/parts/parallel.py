@@ -4,8 +4,8 @@
 
 Each side is a mixer of its own kind with its own cache group and slot (a run entry names the first side's place in
 ``cache_group``/``cache_slot`` and the others' in ``more``).  A side is a mixer that can work between shared products: it
-has ``input_width``, ``inner_width`` and ``mix(ctx, projected, entry, out, scale)`` besides ``qkvg.weight`` and
-``o.weight``.  The sides' input projections are ONE product, their gated rows are written side by side (each times its
+has ``input_width``, ``inner_width`` and ``mix(ctx, projected, entry, out, scale)`` besides its input matrix (``qkvg.weight``, or what its
+class names as ``input_parameter``) and ``o.weight``.  The sides' input projections are ONE product, their gated rows are written side by side (each times its
 scale), and their output projections are one product over the concatenated rows, so that the weighted sum costs nothing.
 The sides keep their parameters' names, behind the side's name (``left.qkvg.weight``); when the tensors are bound, the
 matrices are laid out side by side once and the sides' own matrices become views of that storage.
@@ -47,11 +47,12 @@ class ParallelMixer(Mixer):
         for name, side in zip(self.names, self.sides):
             side.bind({k[len(name) + 1:]: t for k, t in tensors.items() if k.startswith(name + ".")})
         # one matrix for all input projections, one for all output projections; the sides see views of them
-        self.in_weight = torch.cat([s.qkvg_weight for s in self.sides], dim=0).contiguous()
+        names = [getattr(s, "input_parameter", "qkvg.weight").replace(".", "_") for s in self.sides]
+        self.in_weight = torch.cat([getattr(s, name) for s, name in zip(self.sides, names)], dim=0).contiguous()
         self.o_weight = torch.cat([s.o_weight for s in self.sides], dim=1).contiguous()
         row = col = 0
-        for s in self.sides:
-            s.qkvg_weight = self.in_weight[row:row + s.input_width]
+        for s, name in zip(self.sides, names):
+            setattr(s, name, self.in_weight[row:row + s.input_width])
             s.o_weight = self.o_weight[:, col:col + s.inner_width]
             row, col = row + s.input_width, col + s.inner_width
         for name, side in zip(self.names, self.sides):

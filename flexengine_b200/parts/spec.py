@@ -26,7 +26,8 @@ class CacheGroupSpec:
 
     kind "full":   paged keys/values, every key kept.
     kind "window": paged keys/values, only the last ``window`` keys are visible; pages
-                   that the window has passed are given back.
+                   that the window has passed are given back.  ``keep``: the first so many keys of the
+                   sequence stay visible (and their pages stay).
     kind "chunk":  paged keys/values, a query sees only the earlier keys of its own chunk of ``window``
                    positions (counted from position 0 of the sequence); pages that lie wholly before the
                    chunk of the next token are given back.
@@ -51,8 +52,11 @@ class CacheGroupSpec:
     page_size: int = 0
     chunk_granularity: int = 1
     planes: int = 2
+    keep: int = 0
 
     def __post_init__(self):
+        if self.keep < 0 or (self.keep and self.kind != "window"):
+            raise ValueError("keep >= 0, and only a window group keeps its first keys")
         if self.planes not in (1, 2):
             raise ValueError("a paged group keeps one or two tensors per token")
         if self.page_size < 0 or self.chunk_granularity < 1:

@@ -29,7 +29,9 @@ def _post_normed(delta, post):
     return y * torch.rsqrt(y.pow(2).mean(dim=-1, keepdim=True) + eps) * weight.float()
 
 
-def add_rmsnorm(residual, delta, weight, eps, out_dtype, rows=None, upcoming=None, post=None):
+def add_rmsnorm(residual, delta, weight, eps, out_dtype, rows=None, upcoming=None, post=None, delta_scale=None):
+    if delta_scale is not None and delta is not None:
+        delta = delta.float() * delta_scale.float()
     if post is not None and delta is not None:
         delta = _post_normed(delta if rows is None else delta[rows.long()], post)
         if rows is None:
@@ -160,8 +162,8 @@ def qkv_projection(h, w, bias, positions, inv_freq, rot, slot_mapping, k_cache, 
 
 
 def paged_attention(qkv, k_cache, v_cache, block_table, ctx, nq, nkv, d, page_size, scale, window, upcoming=None, sink=False,
-                    weights="softmax", head_bias=None, softcap=0.0, head_scales=None):
-    """``head_scales`` (one number per query head) multiplies the scores as ``scale`` does; ``softcap`` > 0: they then become
+                    weights="softmax", head_bias=None, softcap=0.0, head_scales=None, keep_first=0):
+    """``keep_first``: under a window the first so many keys are seen as well.  ``head_scales`` (one number per query head) multiplies the scores as ``scale`` does; ``softcap`` > 0: they then become
     softcap * tanh(score / softcap).  ``window`` > 0: the last ``window`` keys; < 0: the earlier keys of the query's chunk of -window positions.
     ``sink``: 1 is added to the softmax's denominator.  ``weights`` "sigmoid": a visible key weighs
     sigmoid(score + head_bias[head]), not normalised over the keys."""
@@ -178,14 +180,16 @@ def paged_attention(qkv, k_cache, v_cache, block_table, ctx, nq, nkv, d, page_si
         length = starts[r] + n
         lo = max(0, starts[r] - window + 1) if window > 0 else (starts[r] // chunk * chunk if chunk else 0)
         lo_page = lo // page_size
-        pages = block_table[r, lo_page:-(-length // page_size)].long()
+        kept_pages = min(-(-keep_first // page_size), lo_page) if window > 0 else 0
+        places = torch.tensor(list(range(kept_pages)) + list(range(lo_page, -(-length // page_size))), device=q.device)
+        pages = block_table[r, places].long()
         k = k_cache[pages].float().permute(0, 2, 1, 3).reshape(-1, nkv, d)      # [tokens, nkv, d]
         v = v_cache[pages].float().permute(0, 2, 1, 3).reshape(-1, nkv, d)
-        key_pos = torch.arange(lo_page * page_size, lo_page * page_size + k.shape[0], device=q.device)
+        key_pos = (places[:, None] * page_size + torch.arange(page_size, device=q.device)).reshape(-1)
         q_pos = torch.arange(starts[r], length, device=q.device)
         visible = (key_pos[None, :] <= q_pos[:, None]) & (key_pos[None, :] < length)
         if window > 0:
-            visible &= key_pos[None, :] > q_pos[:, None] - window
+            visible &= (key_pos[None, :] > q_pos[:, None] - window) | (key_pos[None, :] < keep_first)
         if chunk:
             visible &= key_pos[None, :] // chunk == q_pos[:, None] // chunk
         kh = k.repeat_interleave(ratio, dim=1)
@@ -336,14 +340,17 @@ def _turn(x, positions, inv_freq, dims, pairs, sign=1.0):
 
 
 def qkv_norm_rope_cache(projected, q_weight, k_weight, eps, positions, inv_freq, rot_dims, pairs, value_inv_freq, slot_mapping,
-                        k_cache, v_cache, heads, kv_heads, dim, vdim, head, page_size):
-    """projected [T, >= channels] holds q | k | v.  One RMS norm over the whole query projection and one over the whole key
+                        k_cache, v_cache, heads, kv_heads, dim, vdim, head, page_size, bias=None, rot_gain=1.0):
+    """``bias`` (float32 [channels]) is added to q | k | v first; ``rot_gain`` multiplies the turned entries.
+    projected [T, >= channels] holds q | k | v.  One RMS norm over the whole query projection and one over the whole key
     projection (weights of their full widths; None: no norm), then the rotation of the first ``rot_dims`` entries of every
     query and key head, the values turned over all ``vdim`` entries (``value_inv_freq`` None: as they are), keys and values
     into the cache and the queries out, padded with zeros to ``head`` entries a head."""
     T = projected.shape[0]
     qw, kw = heads * dim, kv_heads * dim
-    u = projected.float()
+    u = projected[:, :qw + kw + kv_heads * vdim].float()
+    if bias is not None:
+        u = u + bias.float()
     q, k, v = u[:, :qw], u[:, qw:qw + kw], u[:, qw + kw:qw + kw + kv_heads * vdim]
     if q_weight is not None:
         q = q * torch.rsqrt(q.pow(2).mean(dim=-1, keepdim=True) + eps) * q_weight.float()
@@ -351,6 +358,9 @@ def qkv_norm_rope_cache(projected, q_weight, k_weight, eps, positions, inv_freq,
     q, k, v = q.reshape(T, heads, dim), k.reshape(T, kv_heads, dim), v.reshape(T, kv_heads, vdim)
     if inv_freq is not None and rot_dims > 0:
         q, k = _turn(q, positions, inv_freq, rot_dims, pairs), _turn(k, positions, inv_freq, rot_dims, pairs)
+        if rot_gain != 1.0:
+            q[..., :rot_dims] *= rot_gain
+            k[..., :rot_dims] *= rot_gain
     if value_inv_freq is not None:
         v = _turn(v, positions, value_inv_freq, vdim, pairs)
     dt = projected.dtype
@@ -679,6 +689,133 @@ def head_rmsnorm_gate(out, weight, g, eps, heads, out_dtype, scale=1.0, into=Non
     return into
 
 
+# ---- scans with a decay and a weight per token ------------------------------------------------------------
+def conv_silu(u, conv, bias, state, history_at, state_slots, cu_q, out_float32=False, steps=None, max_q_len=0):
+    """silu(bias + causal convolution) of u [T, channels] (``conv`` [taps, channels]; a request's last taps - 1 rows in
+    state[seat, history_at:], brought up to date).  ``steps`` = (rows [T, heads], bias, minus_a): also float32 [2, T, heads]:
+    the logarithms of the decays minus_a * dt and the step sizes dt = softplus(rows + bias)."""
+    T = u.shape[0]
+    taps, C = conv.shape
+    uf = u.float()
+    y = bias.float().repeat(T, 1)
+    cu, seats, back = cu_q.tolist(), state_slots.tolist(), taps - 1
+    for r in range(len(seats)):
+        a, b = cu[r], cu[r + 1]
+        past = torch.zeros(back, C, dtype=torch.float32, device=u.device)
+        if seats[r] >= 0 and back:
+            past = state[seats[r], history_at:history_at + back * C].view(back, C).clone()
+        rows = torch.cat([past, uf[a:b]])
+        for j in range(taps):
+            y[a:b] += conv[j] * rows[j:j + b - a]
+        if seats[r] >= 0 and back:
+            state[seats[r], history_at:history_at + back * C] = rows[rows.shape[0] - back:].reshape(-1)
+    y = (y / (1.0 + torch.exp(-y))).to(torch.float32 if out_float32 else u.dtype)
+    if steps is None:
+        return y, None
+    rows, dt_bias, minus_a = steps
+    dt = torch.nn.functional.softplus(rows.float() + dt_bias.float())
+    return y, torch.stack([minus_a.float() * dt, dt])
+
+
+def memory_gates(rows, bias, cap, state, maxima_at, state_slots, cu_q, heads):
+    """float32 [3, T, heads] from the rows i | f: the logarithms of the decays f + m - m', the weights exp(i - m') and exp(-m'),
+    with the running maximum m in state[seat, maxima_at:]."""
+    T = rows.shape[0]
+    z = cap * torch.tanh((rows[:, :2 * heads].float() + bias.float()) / cap)
+    log_i, log_f = z[:, :heads], torch.nn.functional.logsigmoid(z[:, heads:])
+    out = torch.zeros(3, T, heads, dtype=torch.float32, device=rows.device)
+    cu, seats = cu_q.tolist(), state_slots.tolist()
+    for r in range(len(seats)):
+        m = state[seats[r], maxima_at:maxima_at + heads].clone() if seats[r] >= 0 else torch.zeros(heads, device=rows.device)
+        for t in range(cu[r], cu[r + 1]):
+            new = torch.maximum(log_f[t] + m, log_i[t])
+            out[0, t], out[1, t], out[2, t] = log_f[t] + m - new, torch.exp(log_i[t] - new), torch.exp(-new)
+            m = new
+        if seats[r] >= 0:
+            state[seats[r], maxima_at:maxima_at + heads] = m
+    return out
+
+
+def head_scan(q, k, v, gates, state, state_slots, cu_q, heads, groups, dim, vdim, query_scale=1.0, skip=None, divided=None, max_q_len=0):
+    """S <- exp(gates[0]) S + gates[1] k v^T, o = S^T q (+ skip v) per request and head; head h reads group h // (heads / groups) of
+    q and k.  ``divided`` (a floor): a memory n of the keys alone behind the heads' S, and o / (max(|n . q|, gates[2]) + floor)."""
+    T = v.shape[0]
+    ratio = heads // groups
+    qf = (q.float() * query_scale).reshape(T, groups, dim).repeat_interleave(ratio, dim=1)
+    kf = k.float().reshape(T, groups, dim).repeat_interleave(ratio, dim=1)
+    vf = v.float().reshape(T, heads, vdim)
+    decay = torch.exp(gates[0])
+    out = torch.zeros(T, heads, vdim, dtype=torch.float32, device=v.device)
+    cu, seats = cu_q.tolist(), state_slots.tolist()
+    m = heads * dim * vdim
+    for r in range(len(seats)):
+        S = state[seats[r], :m].view(heads, dim, vdim).clone() if seats[r] >= 0 else torch.zeros(heads, dim, vdim, device=v.device)
+        n = torch.zeros(heads, dim, device=v.device)
+        if divided is not None and seats[r] >= 0:
+            n = state[seats[r], m:m + heads * dim].view(heads, dim).clone()
+        for t in range(cu[r], cu[r + 1]):
+            w = gates[1, t][:, None] * kf[t]
+            S = decay[t, :, None, None] * S + w[:, :, None] * vf[t][:, None, :]
+            out[t] = torch.einsum("hdv,hd->hv", S, qf[t])
+            if divided is not None:
+                n = decay[t, :, None] * n + w
+                out[t] /= (torch.maximum((n * qf[t]).sum(dim=-1).abs(), gates[2, t]) + divided)[:, None]
+            if skip is not None:
+                out[t] += skip[:, None] * vf[t]
+        if seats[r] >= 0:
+            state[seats[r], :m] = S.reshape(-1)
+            if divided is not None:
+                state[seats[r], m:m + heads * dim] = n.reshape(-1)
+    return out.view(T, heads * vdim)
+
+
+def memory_decode(projected, bias, cap, query_scale, floor, state, state_slots, norm_weight, eps, heads, dim, vdim, out_dtype):
+    R, qk, inner = projected.shape[0], heads * dim, heads * vdim
+    cu = torch.arange(R + 1, dtype=torch.int32, device=projected.device)
+    gates = memory_gates(projected[:, 2 * qk + 2 * inner:], bias, cap, state, heads * (dim * vdim + dim), state_slots, cu, heads)
+    o = head_scan(projected[:, :qk], projected[:, qk:2 * qk], projected[:, 2 * qk:2 * qk + inner], gates, state, state_slots, cu, heads, heads,
+                  dim, vdim, query_scale=query_scale, divided=floor)
+    return head_rmsnorm_gate(o, norm_weight, projected[:, 2 * qk + inner:2 * qk + 2 * inner], eps, heads, out_dtype, gate="sigmoid")
+
+
+def gated_group_rmsnorm(y, z, weight, eps, groups, out_dtype):
+    T, inner = y.shape
+    zf = z.float()
+    x = (y * (zf / (1.0 + torch.exp(-zf)))).view(T, groups, inner // groups)
+    x = x * torch.rsqrt(x.pow(2).mean(dim=-1, keepdim=True) + eps)
+    return (x.reshape(T, inner) * weight.float()).to(out_dtype)
+
+
+def selective_scan(x, dt, dt_bias, minus_a, bc, skip, z, state, state_slots, cu_q, scale=1.0, into=None):
+    """dt <- softplus(dt + dt_bias); S[c, n] <- exp(dt_c minus_a[c, n]) S + dt_c x_c B_n; y = S C + skip x; y silu(z) scale.  ``bc`` [T, B | C]."""
+    T, inner = x.shape
+    N = minus_a.shape[1]
+    dtf = torch.nn.functional.softplus(dt.float() + dt_bias.float())
+    xf, B, C = x.float(), bc[:, :N].float(), bc[:, N:2 * N].float()
+    y = torch.zeros(T, inner, dtype=torch.float32, device=x.device)
+    cu, seats = cu_q.tolist(), state_slots.tolist()
+    for r in range(len(seats)):
+        S = state[seats[r], :inner * N].view(inner, N).clone() if seats[r] >= 0 else torch.zeros(inner, N, device=x.device)
+        for t in range(cu[r], cu[r + 1]):
+            S = torch.exp(dtf[t][:, None] * minus_a) * S + (dtf[t] * xf[t])[:, None] * B[t]
+            y[t] = S @ C[t] + skip * xf[t]
+        if seats[r] >= 0:
+            state[seats[r], :inner * N] = S.reshape(-1)
+    zf = z.float()
+    rows = (y * (zf / (1.0 + torch.exp(-zf))) * scale).to(x.dtype)
+    if into is None:
+        return rows
+    into.copy_(rows)
+    return into
+
+
+def selective_decode(x, low, dt_weight, dt_bias, minus_a, skip, z, state, state_slots, scale=1.0, into=None):
+    R, rank = x.shape[0], dt_weight.shape[1]
+    dt = low[:, :rank].float() @ dt_weight.float().T
+    cu = torch.arange(R + 1, dtype=torch.int32, device=x.device)
+    return selective_scan(x, dt, dt_bias, minus_a, low[:, rank:], skip, z, state, state_slots, cu, scale=scale, into=into)
+
+
 # ---- attention over a cached latent -------------------------------------------------------------------
 def batched_linear(x, w, token_major=False):
     """x [B, M, K] (any strides) times w [B, N, K]^T -> [B, M, N], or [M, B N] with ``token_major``."""
@@ -721,11 +858,14 @@ def latent_prepare(q, q_latent, down, norm_weight, eps, positions, inv_freq, rot
 
 
 # ---- routed feed-forward ------------------------------------------------------------------------------
-def route_top(logits, top, scale, over_chosen=False, correction=None, groups=(1, 1)):
-    """``correction`` (float32, one number per router output) is added to the scores for the choice only; ``groups`` =
+def route_top(logits, top, scale, over_chosen=False, correction=None, groups=(1, 1), sigmoid=False):
+    """``sigmoid``: the scores are sigmoid(z), not normalised.  ``correction`` (float32, one number per router output) is added to the scores for the choice only; ``groups`` =
     (count, keep): only outputs of the ``keep`` groups (of ``count`` equal groups of neighbours) with the largest corrected
     score can be chosen.  Ties go to the lower index."""
     count, keep = groups
+    if sigmoid:
+        best = torch.sort(logits.float(), dim=-1, descending=True, stable=True)
+        return best.indices[:, :top].to(torch.int32), (torch.sigmoid(best.values[:, :top]) * scale).float()
     if correction is not None or count > 1:
         scores = torch.softmax(logits.float(), dim=-1)
         choice = scores if correction is None else scores + correction.float()
@@ -746,8 +886,8 @@ def route_top(logits, top, scale, over_chosen=False, correction=None, groups=(1,
     return best.indices.to(torch.int32), (best.values * scale).float()
 
 
-def routed_experts(h, chosen, weights, gate_up, down, shared=None, activation="silu", limit=0.0, identity=0):
-    """``activation`` "relu2" or "gelu": ``gate_up`` is [experts, F, H], an expert is down(act(up h)).  ``identity``: choices from
+def routed_experts(h, chosen, weights, gate_up, down, shared=None, activation="silu", limit=0.0, identity=0, weigh_input=False):
+    """``weigh_input``: the weights multiply what the experts read.  ``activation`` "relu2" or "gelu": ``gate_up`` is [experts, F, H], an expert is down(act(up h)).  ``identity``: choices from
     ``experts`` on stand for experts that return their input."""
     T, D = h.shape
     f = down.shape[2]
@@ -762,10 +902,13 @@ def routed_experts(h, chosen, weights, gate_up, down, shared=None, activation="s
                     total[rows] += weights[rows, slot, None] * hf[rows]
                 continue
             gu = hf[rows] @ gate_up[e].float().T
+            share = weights[rows, slot, None]
+            if weigh_input:
+                gu, share = gu * share, 1.0
             if activation in ("relu2", "gelu"):
                 z = torch.relu(gu) ** 2 if activation == "relu2" else 0.5 * gu * (1.0 + torch.erf(gu * math.sqrt(0.5)))
                 act = z.to(h.dtype).float()
-                total[rows] += weights[rows, slot, None] * (act @ down[e].float().T)
+                total[rows] += share * (act @ down[e].float().T)
                 continue
             g, u = gu[:, :f], gu[:, f:]
             if activation == "clamped":
@@ -773,7 +916,7 @@ def routed_experts(h, chosen, weights, gate_up, down, shared=None, activation="s
                 act = (g / (1.0 + torch.exp(-1.702 * g)) * (u + 1.0)).to(h.dtype).float()
             else:
                 act = (g / (1.0 + torch.exp(-g)) * u).to(h.dtype).float()
-            total[rows] += weights[rows, slot, None] * (act @ down[e].float().T)
+            total[rows] += share * (act @ down[e].float().T)
     if shared is not None:
         total += shared.float()
     return total.to(h.dtype)
