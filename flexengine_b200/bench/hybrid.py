@@ -1,9 +1,10 @@
-"""``--workload fuvozen|fuvuvik|fedutar|rikolix|bebulorn``: prefill and decode throughput of one of these designs at a few sizes that resemble a
+"""``--workload fuvozen|fuvuvik|fedutar|rikolix|bebulorn|ribozen``: prefill and decode throughput of one of these designs at a few sizes that resemble a
 real model's layers (random weights), beside the closest existing model at equal width, depth and vocabulary (a Qwen2
 decoder; for Fedutar the Fuvozen design, which also has a recurrence with a matrix state and routed experts; for Rikolix the
 Fuvozen design too, which also has attention over a cached latent, routed experts and a dense feed-forward without a gate; for
 Bebulorn the Fedutar design, which also has norms on both sides of a sublayer, linear attention with a state matrix, routed experts
-and a repeated span), and, at one size, an
+and a repeated span; for Ribozen the Bebulorn design, which also has attention under a window with squashed scores, recurrences with a
+state matrix, short convolutions and routed experts beside a shared one), and, at one size, an
 operation-by-operation table of both: time, the bytes and flops of the work, and how far each operation is from the
 roofline of the measured peaks (time / max(bytes / copy rate, flops / bf16 rate)).
 
@@ -131,8 +132,33 @@ def bebulorn_config(width, layers, vocab, heads):
             "loop": {"start": 0, "stop": max(1, layers - distinct), "times": 2 if layers > distinct else 1}, "layers": stack}
 
 
+def ribozen_config(width, layers, vocab, heads):
+    """Layers in turns of three: a state-space layer (2 x width channels in heads of 64, a state of 128, eight groups of keys, four
+    taps), a matrix memory (width / 128 heads of 64 key x 128 value channels, as the lightning attention of the Bebulorn model
+    beside it), and two mixers side by side: softmax attention under a window of 1,024 that keeps four tokens (heads of 128 in
+    groups of four, squashed scores) beside a selective scan over ``width`` channels of 16 state entries.  Every feed-forward has 8
+    experts of 1.25 x width of which a token uses 2, beside a shared one of the same size."""
+    stack = []
+    mlp = {"kind": "moe", "expert": {"ff": width * 5 // 4}, "router": {"experts": 8, "top": 2}, "shared": {"ff": width * 5 // 4}}
+    for i in range(layers):
+        turn = i % 3
+        if turn == 0:
+            mixer = {"type": "mamba2", "mixer": {"heads": width // 32, "vdim": 64, "state": 128, "groups": 8, "norm_groups": 8, "conv": 4}}
+        elif turn == 1:
+            mixer = {"type": "mlstm", "mixer": {"heads": max(1, width // 128), "dim": 64, "vdim": 128, "gate_cap": 15.0}}
+        else:
+            mixer = {"type": "parallel", "mixer": {
+                "left": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "mask": {"size": 1024, "keep_first": 4},
+                         "rot": {"base": 10000.0, "dims": 128, "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}},
+                         "scale": 128 ** -0.5, "softcap": 30.0},
+                "right": {"inner": width, "state": 16, "dt_rank": max(8, width // 16), "conv": 4}, "left_scale": 0.7, "right_scale": 0.7}}
+        stack.append(dict(mixer, mlp=mlp))
+    return {"architecture": "Ribozen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5}, "layers": stack}
+
+
 DESIGNS = {"fuvozen": ("Fuvozen", fuvozen_config), "fuvuvik": ("Fuvuvik", fuvuvik_config), "fedutar": ("Fedutar", fedutar_config),
-           "rikolix": ("Rikolix", rikolix_config), "bebulorn": ("Bebulorn", bebulorn_config)}
+           "rikolix": ("Rikolix", rikolix_config), "bebulorn": ("Bebulorn", bebulorn_config),
+           "ribozen": ("Ribozen", ribozen_config)}
 
 
 def qwen2_config(width, layers, vocab, heads):
@@ -146,7 +172,7 @@ def qwen2_config(width, layers, vocab, heads):
 
 # the model a design is measured beside (default: the Qwen2 decoder)
 BESIDE = {"fedutar": ("fuvozen", "Fuvozen", fuvozen_config), "rikolix": ("fuvozen", "Fuvozen", fuvozen_config),
-          "bebulorn": ("fedutar", "Fedutar", fedutar_config)}
+          "bebulorn": ("fedutar", "Fedutar", fedutar_config), "ribozen": ("bebulorn", "Bebulorn", bebulorn_config)}
 
 SIZES = {"1k": (1024, 8, 32000, 8), "2k": (2048, 8, 32000, 16), "4k": (4096, 4, 32000, 32)}
 
@@ -238,6 +264,36 @@ class TimedOps:
                     nbytes = tokens * 4 * (2 * C + 4 * heads)
                 else:
                     flops, nbytes = 6.0 * tokens * heads * d * dv, tokens * (args[0].shape[1] * 4 + heads * dv * out.element_size()) + states
+            elif name in ("head_scan", "memory_decode", "memory_gates"):
+                # the state's update and its product with the query a token and head; a request's state read and written once
+                if name == "memory_gates":
+                    nbytes = args[0].shape[0] * args[7] * 4 * 5
+                elif name == "head_scan":
+                    heads, groups, d, dv = args[7:11]
+                    tokens, requests = args[2].shape[0], (args[2].shape[0] if kwargs.get("max_q_len") == 1 else args[6].numel() - 1)
+                    flops, nbytes = 4.0 * tokens * heads * d * dv, tokens * 4 * (2 * groups * d + 2 * heads * dv + 2 * heads) + 8.0 * requests * heads * d * dv
+                else:
+                    heads, d, dv = args[9:12]
+                    rows = args[0].shape[0]
+                    flops = 4.0 * rows * heads * d * dv
+                    nbytes = rows * (args[0].shape[1] * 4 + heads * dv * out.element_size() + 8 * heads * (d * dv + d))
+            elif name == "conv_silu":
+                nbytes = 2.0 * args[0].numel() * args[0].element_size()
+            elif name == "gated_group_rmsnorm":
+                nbytes = args[0].numel() * (8 + out.element_size())
+            elif name in ("selective_scan", "selective_decode"):
+                # a token's input, gate and output rows, its step sizes (of which a decode step makes its own), B and C; the states
+                tokens, inner = args[0].shape
+                N = (args[3] if name == "selective_scan" else args[4]).shape[1]
+                requests = args[9].numel() - 1 if name == "selective_scan" else tokens
+                width = args[0].element_size()
+                nbytes = tokens * (inner * (3 * width + (4 if name == "selective_scan" else 0)) + 2 * N * width) + 8.0 * requests * inner * N
+                if name == "selective_decode":
+                    nbytes += args[2].numel() * width
+            elif name == "qkv_norm_rope_cache":
+                heads, kv, d, dv, head = args[12:17]
+                tokens, width = args[0].shape[0], args[0].element_size()
+                nbytes = tokens * width * ((heads + kv) * d + kv * dv + (heads + 2 * kv) * head)
             elif name == "qkv_conv_rope_norm_cache":
                 # the projection's rows read, keys and values into the cache, queries out (not where they stay in place)
                 heads, kv, d, dv, head = args[15:20]
@@ -358,8 +414,8 @@ def run(args) -> int:
     if args.kernels:
         width, layers, vocab, heads = SIZES[sizes[-1] if getattr(args, "size", None) else "2k"]
         # as many layers as show every kind of layer the design has
-        tables[key] = measure(design_config(width, {"fuvozen": 2, "bebulorn": 8}.get(key, 4), vocab, heads), vocab, TimedOps(ops, torch))
-        tables[other] = measure(other_config(width, 4 if other == "fedutar" else 2, vocab, heads), vocab, TimedOps(ops, torch))
+        tables[key] = measure(design_config(width, {"fuvozen": 2, "bebulorn": 8, "ribozen": 3}.get(key, 4), vocab, heads), vocab, TimedOps(ops, torch))
+        tables[other] = measure(other_config(width, {"fedutar": 4, "bebulorn": 8}.get(other, 2), vocab, heads), vocab, TimedOps(ops, torch))
     sampler.stop()
     first = results[sizes[0]][key]
     line = {"metric": f"decode tokens/s ({design} design, size {sizes[0]}, batch {BATCH}, {PROMPT}-token prompts)",
