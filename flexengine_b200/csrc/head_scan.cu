@@ -26,55 +26,6 @@ __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - l
 __device__ __forceinline__ float capped(float z, float cap) { return cap * tanhf(z / cap); }
 
 // ---------------------------------------------------------------------------------------------
-// A warp per (request, head), 32 tokens at a time: the gates side by side, the maximum one token after the other.
-constexpr int GATE_WARPS = 4;
-
-__global__ void __launch_bounds__(GATE_WARPS * 32)
-memory_gates_kernel(const float* __restrict__ rows, long long ld, const float* __restrict__ bias, float cap, float* state,
-                    long long state_stride, long long maxima_at, const int* __restrict__ seats, const int* __restrict__ cu_q,
-                    float* __restrict__ gates, long long plane, int heads, int n_seats) {
-    griddep_wait();
-    griddep_launch_dependents();
-    const int lane = threadIdx.x & 31, head = blockIdx.y * GATE_WARPS + (threadIdx.x >> 5), r = blockIdx.x;
-    if (head >= heads) return;
-    const int begin = cu_q[r], end = cu_q[r + 1];
-    const int seat = seats[r];
-    float* kept = (seat >= 0 && seat < n_seats) ? state + (size_t)seat * state_stride + maxima_at + head : nullptr;
-    float m = kept ? *kept : 0.f;
-    const float bi = bias[head], bf = bias[heads + head];
-    float zi = 0.f, zf = 0.f;
-    if (begin + lane < end) {
-        zi = rows[(size_t)(begin + lane) * ld + head];
-        zf = rows[(size_t)(begin + lane) * ld + heads + head];
-    }
-    for (int t0 = begin; t0 < end; t0 += 32) {
-        const int t = t0 + lane;
-        const bool in = t < end;
-        const float i = in ? capped(zi + bi, cap) : -CUDART_INF_F;
-        const float f = in ? log_sigmoid(capped(zf + bf, cap)) : 0.f;
-        if (t + 32 < end) {                               // the next tokens' rows are asked for ahead of the walk
-            zi = rows[(size_t)(t + 32) * ld + head];
-            zf = rows[(size_t)(t + 32) * ld + heads + head];
-        }
-        float before = 0.f, after = 0.f;
-#pragma unroll
-        for (int j = 0; j < 32; ++j) {
-            const float fj = __shfl_sync(0xffffffffu, f, j), ij = __shfl_sync(0xffffffffu, i, j);
-            const float next = fmaxf(fj + m, ij);
-            if (lane == j) before = m, after = next;
-            m = next;
-        }
-        if (in) {
-            const size_t at = (size_t)t * heads + head;
-            gates[at] = (f + before) - after;
-            gates[plane + at] = expf(i - after);
-            gates[2 * plane + at] = expf(-after);
-        }
-    }
-    if (kept && lane == 0 && end > begin) *kept = m;
-}
-
-// ---------------------------------------------------------------------------------------------
 // Blocks of CHUNK tokens.  Block c of request r has row cu_q[r] / CHUNK + r + c of ``sums`` and ``totals``: the rows of different
 // requests never meet, and T / CHUNK + requests rows hold a step.  A row of sums is a seat's layout: [heads][d][dv], then with a
 // divisor [heads][d]; a row of totals the blocks' decays exp(L_C) [heads].
@@ -85,6 +36,99 @@ static_assert(CHUNK == TILE, "a block of tokens and a tile of channels are loade
 
 __device__ __forceinline__ size_t chunk_row(const int* __restrict__ cu_q, int r) { return (size_t)(cu_q[r] / CHUNK + r); }
 
+// ---------------------------------------------------------------------------------------------
+// The gates of a matrix memory, in blocks of CHUNK tokens.  Over a block the running maximum goes from m to max(m + F, G) with F the
+// sum of the block's f and G what it comes to from minus infinity.  The first kernel makes the gates and F and G; the second one
+// folds the blocks before its own and walks its tokens one after the other.  A block's last token takes the folded value, which the
+// next block (and the seat) starts from.  Planes 0 and 1 of ``gates`` hold f and i in between.  Grid (block of tokens, request).
+constexpr int GATE_THREADS = 256;
+
+__global__ void __launch_bounds__(GATE_THREADS)
+memory_gates_local_kernel(const float* __restrict__ rows, long long ld, const float* __restrict__ bias, float cap, const float* __restrict__ state,
+                          long long state_stride, long long maxima_at, const int* __restrict__ seats, const int* __restrict__ cu_q,
+                          float* __restrict__ gates, long long plane, float* __restrict__ totals, float* __restrict__ starts, int heads,
+                          int n_seats) {
+    griddep_wait();
+    griddep_launch_dependents();
+    extern __shared__ float smem[];
+    float *is = smem, *fs = smem + CHUNK * heads;          // [CHUNK][heads]
+    const int c = blockIdx.x, r = blockIdx.y;
+    const int begin = cu_q[r] + c * CHUNK, end = cu_q[r + 1];
+    if (begin >= end) return;
+    const int len = min(CHUNK, end - begin);
+    for (int e = threadIdx.x; e < len * 2 * heads; e += GATE_THREADS) {
+        const int t = e / (2 * heads), col = e - t * 2 * heads;
+        const float z = capped(rows[(size_t)(begin + t) * ld + col] + bias[col], cap);
+        if (col < heads) {
+            is[t * heads + col] = z;
+            gates[plane + (size_t)(begin + t) * heads + col] = z;
+        } else {
+            const float f = log_sigmoid(z);
+            fs[t * heads + col - heads] = f;
+            gates[(size_t)(begin + t) * heads + col - heads] = f;
+        }
+    }
+    __syncthreads();
+    const size_t row = chunk_row(cu_q, r) + c;
+    const int seat = seats[r];
+    for (int h = threadIdx.x; h < heads; h += GATE_THREADS) {
+        float F = 0.f, G = -CUDART_INF_F;
+#pragma unroll 8
+        for (int t = 0; t < len; ++t) {
+            const float f = fs[t * heads + h];
+            G = fmaxf(G + f, is[t * heads + h]);
+            F += f;
+        }
+        totals[(2 * row) * heads + h] = F;
+        totals[(2 * row + 1) * heads + h] = G;
+        if (c == 0) starts[(size_t)r * heads + h] = (seat >= 0 && seat < n_seats) ? state[(size_t)seat * state_stride + maxima_at + h] : 0.f;
+    }
+}
+
+__global__ void __launch_bounds__(GATE_THREADS)
+memory_gates_walk_kernel(float* state, long long state_stride, long long maxima_at, const int* __restrict__ seats, const int* __restrict__ cu_q,
+                         float* __restrict__ gates, long long plane, const float* __restrict__ totals, const float* __restrict__ starts, int heads,
+                         int n_seats) {
+    griddep_wait();
+    griddep_launch_dependents();
+    extern __shared__ float smem[];
+    float *is = smem, *fs = smem + CHUNK * heads, *ms = fs + CHUNK * heads;        // [CHUNK][heads] twice, the maxima [CHUNK + 1][heads]
+    const int c = blockIdx.x, r = blockIdx.y;
+    const int begin = cu_q[r] + c * CHUNK, end = cu_q[r + 1];
+    if (begin >= end) return;
+    const int len = min(CHUNK, end - begin), count = len * heads;
+    float *decays = gates + (size_t)begin * heads, *weights = decays + plane, *floors = weights + plane;
+    for (int e = threadIdx.x; e < count; e += GATE_THREADS) {
+        fs[e] = decays[e];
+        is[e] = weights[e];
+    }
+    __syncthreads();
+    const size_t row0 = chunk_row(cu_q, r);
+    const int seat = seats[r];
+    for (int h = threadIdx.x; h < heads; h += GATE_THREADS) {
+        float m = starts[(size_t)r * heads + h];
+#pragma unroll 8
+        for (int b = 0; b < c; ++b) m = fmaxf(m + totals[2 * (row0 + b) * heads + h], totals[(2 * (row0 + b) + 1) * heads + h]);
+        const float after = fmaxf(m + totals[2 * (row0 + c) * heads + h], totals[(2 * (row0 + c) + 1) * heads + h]);
+        ms[h] = m;
+#pragma unroll 8
+        for (int t = 0; t < len - 1; ++t) {
+            m = fmaxf(fs[t * heads + h] + m, is[t * heads + h]);
+            ms[(t + 1) * heads + h] = m;
+        }
+        ms[len * heads + h] = after;
+        if (begin + len == end && seat >= 0 && seat < n_seats) state[(size_t)seat * state_stride + maxima_at + h] = after;
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < count; e += GATE_THREADS) {
+        const float next = ms[e + heads];
+        decays[e] = (fs[e] + ms[e]) - next;
+        weights[e] = expf(is[e] - next);
+        floors[e] = expf(-next);
+    }
+}
+
+// ---------------------------------------------------------------------------------------------
 // cum[n] = l_0 + .. + l_n of the block's tokens (tokens from len on repeat the last sum); the first CHUNK threads work.
 __device__ __forceinline__ void cumulate(const float* __restrict__ gates, int begin, int len, int heads, int head, double* cum, double* half) {
     const int tid = threadIdx.x;
@@ -463,15 +507,26 @@ int launch_step(const float* q, long long ldq, float query_scale, const float* k
 }  // namespace
 
 // rows float [T, >= 2 heads] (i, then f; rows ld entries long); bias float [2 heads]; gates float [3][plane] with plane >= T heads: the
-// decays' logarithms, the weights, exp(-m); the running maxima [heads] of a seat lie at state[seat][maxima_at].
+// decays' logarithms, the weights, exp(-m); the running maxima [heads] of a seat lie at state[seat][maxima_at].  totals float [tokens /
+// 64 + requests, 2, heads] and starts float [requests, heads] are scratch; most_tokens: the longest portion of the step or more.
 extern "C" int fe_memory_gates(const float* rows, long long ld, const float* bias, float cap, float* state, long long state_stride,
-                               long long maxima_at, const int* seats, const int* cu_q, float* gates, long long plane, int requests, int heads,
-                               int n_seats, cudaStream_t stream) {
+                               long long maxima_at, const int* seats, const int* cu_q, float* gates, long long plane, float* totals, float* starts,
+                               int requests, int most_tokens, int heads, int n_seats, cudaStream_t stream) {
     FE_REQUIRE(requests >= 0 && heads > 0 && ld >= 2 * heads && cap > 0.f && n_seats >= 0 && maxima_at >= 0 && maxima_at + heads <= state_stride,
                "memory_gates: bad sizes (%d heads)", heads);
-    if (requests == 0) return 0;
-    fe::launch(memory_gates_kernel, dim3(requests, (heads + GATE_WARPS - 1) / GATE_WARPS), GATE_WARPS * 32, 0, stream, rows, ld, bias, cap,
-               state, state_stride, maxima_at, seats, cu_q, gates, plane, heads, n_seats);
+    if (requests == 0 || most_tokens == 0) return 0;
+    FE_REQUIRE(requests <= 65535 && heads <= 256, "memory_gates: %d requests or %d heads (up to 256)", requests, heads);
+    const dim3 grid((most_tokens + CHUNK - 1) / CHUNK, requests);
+    const size_t local = (size_t)2 * CHUNK * heads * sizeof(float), walk = (size_t)(3 * CHUNK + 1) * heads * sizeof(float);
+    if (walk > 48 * 1024) {
+        cudaError_t err = cudaFuncSetAttribute(memory_gates_local_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)local);
+        if (err == cudaSuccess) err = cudaFuncSetAttribute(memory_gates_walk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)walk);
+        FE_REQUIRE(err == cudaSuccess, "memory_gates: %s", cudaGetErrorString(err));
+    }
+    fe::launch(memory_gates_local_kernel, grid, GATE_THREADS, local, stream, rows, ld, bias, cap, (const float*)state, state_stride, maxima_at,
+               seats, cu_q, gates, plane, totals, starts, heads, n_seats);
+    fe::launch(memory_gates_walk_kernel, grid, GATE_THREADS, walk, stream, state, state_stride, maxima_at, seats, cu_q, gates, plane,
+               (const float*)totals, (const float*)starts, heads, n_seats);
     return fe_check_launch("memory_gates");
 }
 

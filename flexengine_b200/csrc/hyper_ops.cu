@@ -870,6 +870,138 @@ __global__ void qkv_norm_rope_cache_kernel(const T* __restrict__ proj, long long
     }
 }
 
+// The same where the pairs are halves, nothing of the values turns and everything comes in fours (sizes, half a rotation, strides):
+// a thread loads, turns and stores four neighbouring entries at a time, of both halves of a pair together.
+template <typename T> struct Four;
+template <> struct Four<float> {
+    static __device__ __forceinline__ float4 load(const float* p) { return *reinterpret_cast<const float4*>(p); }
+    static __device__ __forceinline__ void store(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+};
+template <> struct Four<bf16> {
+    static __device__ __forceinline__ float4 load(const bf16* p) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(p);
+        return make_float4(__uint_as_float(raw.x << 16), __uint_as_float(raw.x & 0xffff0000u), __uint_as_float(raw.y << 16),
+                           __uint_as_float(raw.y & 0xffff0000u));
+    }
+    static __device__ __forceinline__ void store(bf16* p, float4 v) {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+        uint2 raw;
+        raw.x = *reinterpret_cast<const unsigned*>(&a), raw.y = *reinterpret_cast<const unsigned*>(&b);
+        *reinterpret_cast<uint2*>(p) = raw;
+    }
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+qkv_norm_rope_cache_four_kernel(const T* __restrict__ proj, long long ld, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
+                                float eps, const int* __restrict__ positions, const float* __restrict__ inv_freq, int rot,
+                                const float* __restrict__ bias, float gain, const int* __restrict__ slot_mapping, T* __restrict__ kc,
+                                T* __restrict__ vc, T* __restrict__ q_out, int heads, int kv_heads, int dim, int vdim, int head, int ps,
+                                long long num_slots, int* __restrict__ status) {
+    griddep_wait();
+    griddep_launch_dependents();
+    extern __shared__ __align__(16) float staged[];
+    __shared__ float sums[2][8];
+    const int tok = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int qw = heads * dim, kw = kv_heads * dim, qk = qw + kw;
+    const int half = rot >> 1;
+    float* row = staged;                              // [qk] queries and keys
+    float* cosines = staged + qk;                     // [half], then the sines [half]
+    float* sines = cosines + half;
+    const T* src = proj + (size_t)tok * ld;
+    float ssq = 0.f, ssk = 0.f;
+    for (int c = tid * 4; c < qk; c += 1024) {
+        float4 v = Four<T>::load(src + c);
+        if (bias) {
+            const float4 b = *reinterpret_cast<const float4*>(bias + c);
+            v.x += b.x, v.y += b.y, v.z += b.z, v.w += b.w;
+        }
+        *reinterpret_cast<float4*>(row + c) = v;
+        const float s = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        if (c < qw) ssq += s;
+        else ssk += s;
+    }
+    const float pos = (float)positions[tok];
+    for (int i = tid; i < half; i += 256) {
+        float si, co;
+        sincosf(pos * inv_freq[i], &si, &co);
+        sines[i] = si * gain;
+        cosines[i] = co * gain;
+    }
+    T* kdst = nullptr;
+    T* vdst = nullptr;
+    if (slot_mapping) {
+        const int slot = slot_mapping[tok];
+        if (slot >= 0) {
+            if (slot >= num_slots) {
+                if (tid == 0 && status) atomicOr(status, FE_STATUS_BAD_SLOT);
+            } else {
+                const long long page = slot / ps, off = slot % ps;
+                kdst = kc + ((page * kv_heads) * ps + off) * head;          // head 0; the next head is ps * head further
+                vdst = vc + ((page * kv_heads) * ps + off) * head;
+            }
+        }
+    }
+    if (vdst) {                                        // values need only their bias
+        const int per = head >> 2;
+        for (int e = tid; e < kv_heads * per; e += 256) {
+            const int index = e / per, c = (e - index * per) * 4;
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (c < vdim) {
+                const int at = qk + index * vdim + c;
+                v = Four<T>::load(src + at);
+                if (bias) {
+                    const float4 b = *reinterpret_cast<const float4*>(bias + at);
+                    v.x += b.x, v.y += b.y, v.z += b.z, v.w += b.w;
+                }
+            }
+            Four<T>::store(vdst + (size_t)index * ps * head + c, v);
+        }
+    }
+    float inv_q = 1.f, inv_k = 1.f;
+    ssq = warp_sum(ssq);
+    ssk = warp_sum(ssk);
+    if (lane == 0) sums[0][warp] = ssq, sums[1][warp] = ssk;
+    __syncthreads();
+    if (q_weight) {
+        ssq = ssk = 0.f;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) ssq += sums[0][w], ssk += sums[1][w];
+        inv_q = rsqrtf(ssq / (float)qw + eps);
+        inv_k = rsqrtf(ssk / (float)kw + eps);
+    }
+    // units of four entries: of a head, the pairs' first halves (with the second ones), then what passes and the padding
+    const int turning = half >> 2, rest = (head - rot) >> 2, per = turning + rest;
+    T* qdst = q_out + (size_t)tok * heads * head;
+    for (int e = tid; e < (heads + kv_heads) * per; e += 256) {
+        const int hs = e / per, unit = e - hs * per;
+        const bool is_q = hs < heads;
+        T* dst = is_q ? qdst + (size_t)hs * head : (kdst ? kdst + (size_t)(hs - heads) * ps * head : nullptr);
+        if (!dst) continue;
+        const float inv = is_q ? inv_q : inv_k;
+        const int at = hs * dim;                       // keys follow the queries
+        const float* weight = q_weight ? (is_q ? q_weight + at : k_weight + (at - qw)) : nullptr;
+        auto normed = [&](int c) {
+            float4 v = *reinterpret_cast<const float4*>(row + at + c);
+            if (weight) {
+                const float4 w = *reinterpret_cast<const float4*>(weight + c);
+                v.x *= inv * w.x, v.y *= inv * w.y, v.z *= inv * w.z, v.w *= inv * w.w;
+            }
+            return v;
+        };
+        if (unit < turning) {
+            const int c = unit * 4;
+            const float4 u = normed(c), v = normed(c + half);
+            const float4 co = *reinterpret_cast<const float4*>(cosines + c), si = *reinterpret_cast<const float4*>(sines + c);
+            Four<T>::store(dst + c, make_float4(fmaf(u.x, co.x, -v.x * si.x), fmaf(u.y, co.y, -v.y * si.y), fmaf(u.z, co.z, -v.z * si.z), fmaf(u.w, co.w, -v.w * si.w)));
+            Four<T>::store(dst + c + half, make_float4(fmaf(v.x, co.x, u.x * si.x), fmaf(v.y, co.y, u.y * si.y), fmaf(v.z, co.z, u.z * si.z), fmaf(v.w, co.w, u.w * si.w)));
+        } else {
+            const int c = rot + (unit - turning) * 4;
+            Four<T>::store(dst + c, c < dim ? normed(c) : make_float4(0.f, 0.f, 0.f, 0.f));
+        }
+    }
+}
+
 // out[t, h, :vdim] = the first vdim entries of head h of mixed[t] turned BACK by the token's position (pair m by
 // -position * inv_freq[m]), times ``scale``; the padding of the attention kernels' head size is dropped on the way.
 template <typename T>
@@ -912,6 +1044,26 @@ extern "C" int fe_qkv_norm_rope_cache(const void* proj, long long ld, const floa
     const size_t smem = ((size_t)C + rot + (v_inv_freq ? vdim : 0)) * sizeof(float);
     FE_REQUIRE(smem <= 200 * 1024, "qkv_norm_rope_cache: a token's projections need %zu bytes of shared memory (limit 204800)", smem);
     FE_REQUIRE(dtype == FE_F32 || dtype == FE_BF16, "qkv_norm_rope_cache: unknown dtype %d", dtype);
+    const size_t align = dtype == FE_F32 ? 16 : 8;
+    if (!interleaved && v_inv_freq == nullptr && head % 4 == 0 && dim % 4 == 0 && vdim % 4 == 0 && rot % 8 == 0 && ld % 4 == 0 &&
+        (size_t)proj % align == 0 && (((size_t)q_weight | (size_t)k_weight | (size_t)bias) & 15) == 0 &&
+        (((size_t)kc | (size_t)vc | (size_t)q_out) % align) == 0) {
+        const size_t four_smem = ((size_t)(heads + kv_heads) * dim + rot) * sizeof(float);
+#define FE_LAUNCH_QKV_FOUR(TYPE)                                                                                                        \
+    do {                                                                                                                                \
+        if (four_smem > 48 * 1024) {                                                                                                    \
+            cudaError_t err = cudaFuncSetAttribute(qkv_norm_rope_cache_four_kernel<TYPE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)four_smem); \
+            FE_REQUIRE(err == cudaSuccess, "qkv_norm_rope_cache: %s", cudaGetErrorString(err));                                          \
+        }                                                                                                                               \
+        fe::launch(qkv_norm_rope_cache_four_kernel<TYPE>, T, 256, four_smem, stream, (const TYPE*)proj, ld, q_weight, k_weight, eps,      \
+                   positions, inv_freq, rot, bias, gain, slot_mapping, (TYPE*)kc, (TYPE*)vc, (TYPE*)q_out, heads, kv_heads, dim, vdim,    \
+                   head, ps, num_slots, status);                                                                                        \
+    } while (0)
+        if (dtype == FE_F32) FE_LAUNCH_QKV_FOUR(float);
+        else FE_LAUNCH_QKV_FOUR(bf16);
+#undef FE_LAUNCH_QKV_FOUR
+        return fe_check_launch("qkv_norm_rope_cache");
+    }
     const int threads = C >= 2048 ? 512 : 256;
 #define FE_LAUNCH_QKV_NORM(TYPE)                                                                                                        \
     do {                                                                                                                                \

@@ -134,6 +134,84 @@ __global__ void route_top_kernel(const float* __restrict__ logits, int* __restri
     }
 }
 
+// Router logits: out[t, e] = h[t] . W[e] in float, h float or bfloat16.  A block takes LOGIT_ROWS tokens; its warps share out K (a lane
+// walks it in fours), take eight experts at a time, and their sums meet in shared memory.  A token's sum is taken in the same
+// order whatever else is in the batch.
+constexpr int LOGIT_ROWS = 4, LOGIT_WARPS = 8, LOGIT_EXPERTS = 8;
+
+template <typename T> __device__ __forceinline__ float4 load_four(const T* p);
+template <> __device__ __forceinline__ float4 load_four<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <> __device__ __forceinline__ float4 load_four<bf16>(const bf16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(raw.x << 16), __uint_as_float(raw.x & 0xffff0000u), __uint_as_float(raw.y << 16),
+                       __uint_as_float(raw.y & 0xffff0000u));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(LOGIT_WARPS * 32)
+router_logits_kernel(const T* __restrict__ h, const float* __restrict__ W, float* __restrict__ out, int T_tokens, int experts, int K) {
+    griddep_wait();
+    griddep_launch_dependents();
+    __shared__ float part[LOGIT_WARPS][32];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int t0 = blockIdx.x * LOGIT_ROWS;
+    const T* row[LOGIT_ROWS];
+#pragma unroll
+    for (int r = 0; r < LOGIT_ROWS; ++r) row[r] = h + (size_t)min(t0 + r, T_tokens - 1) * K;
+    for (int e0 = 0; e0 < experts; e0 += LOGIT_EXPERTS) {
+        float acc[LOGIT_ROWS * LOGIT_EXPERTS];
+#pragma unroll
+        for (int i = 0; i < LOGIT_ROWS * LOGIT_EXPERTS; ++i) acc[i] = 0.f;
+        for (int k = (warp * 32 + lane) * 4; k < K; k += LOGIT_WARPS * 128) {
+            float4 a[LOGIT_ROWS];
+#pragma unroll
+            for (int r = 0; r < LOGIT_ROWS; ++r) a[r] = load_four<T>(row[r] + k);
+#pragma unroll
+            for (int e = 0; e < LOGIT_EXPERTS; ++e) {
+                const float4 w = *reinterpret_cast<const float4*>(W + (size_t)min(e0 + e, experts - 1) * K + k);
+#pragma unroll
+                for (int r = 0; r < LOGIT_ROWS; ++r) {
+                    float& x = acc[r * LOGIT_EXPERTS + e];
+                    x = fmaf(a[r].x, w.x, x), x = fmaf(a[r].y, w.y, x), x = fmaf(a[r].z, w.z, x), x = fmaf(a[r].w, w.w, x);
+                }
+            }
+        }
+        // 32 sums over 32 lanes: rounds in which a lane gives half of its sums away; lane i ends with sum i
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const bool up = lane & o;
+#pragma unroll
+            for (int i = 0; i < 16; ++i) {
+                if (i >= o) break;
+                const float keep = up ? acc[o + i] : acc[i], give = up ? acc[i] : acc[o + i];
+                acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+            }
+        }
+        part[warp][lane] = acc[0];
+        __syncthreads();
+        if (warp == 0) {
+            float sum = 0.f;
+#pragma unroll
+            for (int w = 0; w < LOGIT_WARPS; ++w) sum += part[w][lane];
+            const int t = t0 + lane / LOGIT_EXPERTS, e = e0 + lane % LOGIT_EXPERTS;
+            if (t < T_tokens && e < experts) out[(size_t)t * experts + e] = sum;
+        }
+        __syncthreads();
+    }
+}
+
+// h [T, K] in ``dtype``, W float [experts, K], out float [T, experts]; K a multiple of four, rows on 16-byte (bfloat16: 8-byte) boundaries.
+extern "C" int fe_router_logits(const void* h, const float* W, float* out, int T, int experts, int K, int dtype, cudaStream_t stream) {
+    FE_REQUIRE(T >= 0 && experts >= 1 && K >= 4 && K % 4 == 0, "router_logits: bad sizes (experts %d, width %d in steps of 4)", experts, K);
+    FE_REQUIRE(((size_t)W & 15) == 0 && ((size_t)h & (dtype == FE_F32 ? 15 : 7)) == 0, "router_logits: operands must be aligned");
+    FE_REQUIRE(dtype == FE_F32 || dtype == FE_BF16, "router_logits: unknown dtype %d", dtype);
+    if (T == 0) return 0;
+    const int blocks = (T + LOGIT_ROWS - 1) / LOGIT_ROWS;
+    if (dtype == FE_F32) fe::launch(router_logits_kernel<float>, blocks, LOGIT_WARPS * 32, 0, stream, (const float*)h, W, out, T, experts, K);
+    else fe::launch(router_logits_kernel<bf16>, blocks, LOGIT_WARPS * 32, 0, stream, (const bf16*)h, W, out, T, experts, K);
+    return fe_check_launch("router_logits");
+}
+
 extern "C" int fe_route_top(const float* logits, int* chosen, float* weights, int T, int experts, int top, float scale,
                             int over_chosen, const float* correction, int groups, int keep, cudaStream_t stream) {
     FE_REQUIRE(T >= 0 && experts >= 1 && experts <= ROUTE_MAX_EXPERTS && top >= 1 && top <= experts,

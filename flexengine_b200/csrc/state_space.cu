@@ -186,62 +186,97 @@ __global__ void gated_group_rmsnorm_kernel(const float* __restrict__ y, const fl
 
 // ---------------------------------------------------------------------------------------------
 // The selective scan.  LANES neighbouring lanes share a channel, each with NPT neighbouring entries of its state in registers
-// (entries beyond N have B = C = 0 and stay zero); EXACT takes the decays to half an ulp (exp_decay), else they are the hardware's
-// 2^x; a block has 128 / LANES channels of one request and walks its portion in
-// tiles of TT tokens staged in shared memory; the rows of the next tile are on their way (in registers) while one is walked.
-// Four tokens at a time share the rounds of the sum over the lanes.
+// (entries beyond N have B = C = 0 and stay zero); the true 32-bit path takes the decays to half an ulp (exp_decay), the other one
+// with the hardware's 2^x; a block has 128 / LANES channels of one request and walks its tokens in tiles of TT staged in shared
+// memory; the rows of the next tile are on their way (in registers, as they lie in memory) while one is walked.  Four tokens at a
+// time share the rounds of the sum over the lanes.
+// A long portion of few channels would leave most of the device idle: it is cut into segments that are walked side by side.  MODE
+// WALK: a portion from its seat to its seat.  Else three launches: FOLD walks every segment from a state of zero, without outputs,
+// and leaves the state it ends with and the sum of its step sizes (and, in place of the step sizes' rows, the step sizes);
+// the chain makes of them the state before every segment, S <- exp(A sum) S + fold; OUT walks every segment from there.  Segment
+// s of request r has row cu_q[r] / SEGMENT + r + s of ``folds`` and ``sums``.
 constexpr int SCAN_THREADS = 128;
+constexpr int SEGMENT = 128;
+enum ScanMode { WALK, FOLD, OUT };
 
-template <typename TX, bool EXACT, int LANES, int NPT, int TT>
+__device__ __forceinline__ size_t segment_row(const int* __restrict__ cu_q, int r) { return (size_t)(cu_q[r] / SEGMENT + r); }
+
+struct SelectiveScan {
+    float* dt;                  // [T, inner]: before bias and softplus; FOLD leaves the step sizes there
+    const float* dt_bias;
+    const float* minus_a;       // [inner, N]
+    const float* skip;
+    float* state;
+    long long state_stride;
+    const int* seats;
+    const int* cu_q;
+    float* folds;               // [rows][inner N]
+    float* sums;                // [rows][inner]
+    float scale;
+    int inner, N, n_seats;
+};
+
+template <typename TX, ScanMode MODE, int LANES, int NPT, int TT>
 __global__ void __launch_bounds__(SCAN_THREADS)
-selective_scan_kernel(const TX* __restrict__ x, const float* __restrict__ dt, const float* __restrict__ dt_bias, const float* __restrict__ minus_a,
-                      const TX* __restrict__ bc, long long ldbc, const float* __restrict__ skip, const TX* __restrict__ z, long long ldz,
-                      float* state, long long state_stride, const int* __restrict__ seats, const int* __restrict__ cu_q, TX* __restrict__ out,
-                      long long ldo, float scale, int inner, int N, int n_seats) {
+selective_scan_kernel(const TX* __restrict__ x, const TX* __restrict__ bc, long long ldbc, const TX* __restrict__ z, long long ldz,
+                      TX* __restrict__ out, long long ldo, SelectiveScan sc) {
     griddep_wait();
     griddep_launch_dependents();
-    constexpr int CH = SCAN_THREADS / LANES, NP = LANES * NPT;
-    constexpr int PER_X = (TT * CH + SCAN_THREADS - 1) / SCAN_THREADS, PER_B = (TT * 2 * NP + SCAN_THREADS - 1) / SCAN_THREADS;
+    constexpr bool EXACT = sizeof(TX) == 4;        // the true 32-bit path
+    constexpr int CH = SCAN_THREADS / LANES, NP = LANES * NPT, KEYS = MODE == FOLD ? NP : 2 * NP;       // B, or B and C
+    constexpr int PER_X = (TT * CH + SCAN_THREADS - 1) / SCAN_THREADS, PER_B = (TT * KEYS + SCAN_THREADS - 1) / SCAN_THREADS;
     extern __shared__ __align__(16) float smem[];
     float* dts = smem;                              // [TT][CH] step sizes
     float* dxs = dts + TT * CH;                     // [TT][CH] step size times input
-    float* xs = dxs + TT * CH;                      // [TT][CH] inputs
-    float* ys = xs + TT * CH;                       // [TT][CH]
-    float* bs = ys + TT * CH;                       // [TT][NP]
+    float* bs = dxs + TT * CH;                      // [TT][NP]
     float* cs = bs + TT * NP;                       // [TT][NP]
+    float* xs = cs + TT * NP;                       // [TT][CH] inputs
+    float* ys = xs + TT * CH;                       // [TT][CH]
+    const int inner = sc.inner, N = sc.N;
     const int tid = threadIdx.x, r = blockIdx.y, c0 = blockIdx.x * CH;
     const int l = tid % LANES, cl = tid / LANES, ch = c0 + cl;
-    const int begin = cu_q[r], end = cu_q[r + 1];
+    const int first = sc.cu_q[r], last = sc.cu_q[r + 1];
+    const int begin = MODE == WALK ? first : first + (int)blockIdx.z * SEGMENT;
+    const int end = MODE == WALK ? last : min(last, begin + SEGMENT);
     if (begin >= end) return;
-    const int seat = seats[r];
-    float* mine = (seat >= 0 && seat < n_seats && ch < inner) ? state + (size_t)seat * state_stride + (size_t)ch * N : nullptr;
+    const size_t seg_row = MODE == WALK ? 0 : segment_row(sc.cu_q, r) + blockIdx.z;
+    const int seat = sc.seats[r];
+    float* mine = (seat >= 0 && seat < sc.n_seats && ch < inner) ? sc.state + (size_t)seat * sc.state_stride + (size_t)ch * N : nullptr;
+    float* fold = (MODE != WALK && ch < inner) ? sc.folds + seg_row * ((size_t)inner * N) + (size_t)ch * N : nullptr;
+    const float* from = MODE == WALK ? mine : MODE == OUT ? fold : nullptr;
     float S[NPT], A[NPT];
 #pragma unroll
     for (int e = 0; e < NPT; ++e) {
         const int i = l * NPT + e;
-        S[e] = (mine && i < N) ? mine[i] : 0.f;
-        A[e] = (ch < inner && i < N) ? minus_a[(size_t)ch * N + i] * (EXACT ? 1.f : LOG2E) : 0.f;
+        S[e] = (from && i < N) ? from[i] : 0.f;
+        A[e] = (ch < inner && i < N) ? sc.minus_a[(size_t)ch * N + i] * (EXACT ? 1.f : LOG2E) : 0.f;
     }
     // element e of a tile's [TT][CH] rows belongs to thread e % 128; a thread's channel is the same in all of them
     const int my_c = tid % CH, my_t = tid / CH;
     const bool in_c = c0 + my_c < inner;
-    const float my_bias = in_c ? dt_bias[c0 + my_c] : 0.f, my_skip = in_c ? skip[c0 + my_c] : 0.f;
-    float px[PER_X], pd[PER_X], pz[PER_X], pb[PER_B];
+    const float my_bias = in_c ? sc.dt_bias[c0 + my_c] : 0.f, my_skip = in_c ? sc.skip[c0 + my_c] : 0.f;
+    TX px[PER_X], pz[PER_X], pb[PER_B];
+    float pd[PER_X];
     auto fetch = [&](int t0) {
 #pragma unroll
         for (int i = 0; i < PER_X; ++i) {
             const int t = t0 + my_t + i * (SCAN_THREADS / CH);
             const bool in = in_c && my_t + i * (SCAN_THREADS / CH) < TT && t < end;
-            px[i] = in ? to_float(x[(size_t)t * inner + c0 + my_c]) : 0.f;
-            pd[i] = in ? dt[(size_t)t * inner + c0 + my_c] : 0.f;
+            px[i] = TX(0.f);
+            pd[i] = 0.f;
+            if (in) {
+                px[i] = x[(size_t)t * inner + c0 + my_c];
+                pd[i] = sc.dt[(size_t)t * inner + c0 + my_c];
+            }
         }
 #pragma unroll
         for (int i = 0; i < PER_B; ++i) {
-            const int e = tid + i * SCAN_THREADS, tt = e / (2 * NP), n = e % (2 * NP), at = n % NP;
-            const bool in = tt < TT && t0 + tt < end && at < N;
-            pb[i] = in ? to_float(bc[(size_t)(t0 + tt) * ldbc + (n < NP ? at : N + at)]) : 0.f;
+            const int e = tid + i * SCAN_THREADS, tt = e / KEYS, n = e % KEYS, at = n % NP;
+            pb[i] = TX(0.f);
+            if (tt < TT && t0 + tt < end && at < N) pb[i] = bc[(size_t)(t0 + tt) * ldbc + (n < NP ? at : N + at)];
         }
     };
+    float dt_sum = 0.f;
     fetch(begin);
     for (int t0 = begin; t0 < end; t0 += TT) {
         const int count = min(TT, end - t0);
@@ -250,22 +285,31 @@ selective_scan_kernel(const TX* __restrict__ x, const float* __restrict__ dt, co
             const int tt = my_t + i * (SCAN_THREADS / CH);
             if (tt >= TT) break;
             // tokens beyond the end have a step size of zero: the state stays as it is
-            const float d = (in_c && tt < count) ? softplus(pd[i] + my_bias) : 0.f;
+            const bool in = in_c && tt < count;
+            const float d = in ? (MODE == OUT ? pd[i] : softplus(pd[i] + my_bias)) : 0.f;
+            const float xv = to_float(px[i]);
             dts[tt * CH + my_c] = d;
-            dxs[tt * CH + my_c] = d * px[i];
-            xs[tt * CH + my_c] = px[i];
+            dxs[tt * CH + my_c] = d * xv;
+            if (MODE == FOLD) {
+                if (in) sc.dt[(size_t)(t0 + tt) * inner + c0 + my_c] = d;
+            } else {
+                xs[tt * CH + my_c] = xv;
+            }
         }
 #pragma unroll
         for (int i = 0; i < PER_B; ++i) {
-            const int e = tid + i * SCAN_THREADS, tt = e / (2 * NP), n = e % (2 * NP);
-            if (tt < TT) (n < NP ? bs : cs)[tt * NP + n % NP] = pb[i];
+            const int e = tid + i * SCAN_THREADS, tt = e / KEYS, n = e % KEYS;
+            if (tt < TT) (n < NP ? bs : cs)[tt * NP + n % NP] = to_float(pb[i]);
         }
         __syncthreads();
         // the gates of this tile and the rows of the next one
+        if (MODE != FOLD) {
 #pragma unroll
-        for (int i = 0; i < PER_X; ++i) {
-            const int tt = my_t + i * (SCAN_THREADS / CH);
-            pz[i] = (in_c && tt < count) ? to_float(z[(size_t)(t0 + tt) * ldz + c0 + my_c]) : 0.f;
+            for (int i = 0; i < PER_X; ++i) {
+                const int tt = my_t + i * (SCAN_THREADS / CH);
+                pz[i] = TX(0.f);
+                if (in_c && tt < count) pz[i] = z[(size_t)(t0 + tt) * ldz + c0 + my_c];
+            }
         }
         if (t0 + TT < end) fetch(t0 + TT);
 #pragma unroll 1
@@ -279,73 +323,120 @@ selective_scan_kernel(const TX* __restrict__ x, const float* __restrict__ dt, co
 #pragma unroll
                 for (int e = 0; e < NPT; e += 4) {
                     const float4 b4 = *reinterpret_cast<const float4*>(bs + tt * NP + l * NPT + e);
-                    const float4 q4 = *reinterpret_cast<const float4*>(cs + tt * NP + l * NPT + e);
-                    const float bb[4] = {b4.x, b4.y, b4.z, b4.w}, qq[4] = {q4.x, q4.y, q4.z, q4.w};
+                    const float bb[4] = {b4.x, b4.y, b4.z, b4.w};
 #pragma unroll
-                    for (int i = 0; i < 4; ++i) {
-                        S[e + i] = fmaf(EXACT ? exp_decay(d * A[e + i]) : exp2f(d * A[e + i]), S[e + i], dx * bb[i]);
-                        y = fmaf(S[e + i], qq[i], y);
+                    for (int i = 0; i < 4; ++i) S[e + i] = fmaf(EXACT ? exp_decay(d * A[e + i]) : exp2f(d * A[e + i]), S[e + i], dx * bb[i]);
+                    if (MODE != FOLD) {
+                        const float4 q4 = *reinterpret_cast<const float4*>(cs + tt * NP + l * NPT + e);
+                        const float qq[4] = {q4.x, q4.y, q4.z, q4.w};
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) y = fmaf(S[e + i], qq[i], y);
                     }
                 }
                 y4[q] = y;
+                if (MODE == FOLD) dt_sum += d;
             }
-            // the sums over the lanes: two rounds in which a lane gives half of its tokens away, then plain rounds; the lane ends
-            // with token (l & 1) * 2 + ((l >> 1) & 1)
-            float y2[2];
+            if constexpr (MODE != FOLD) {
+                // the sums over the lanes: two rounds in which a lane gives half of its tokens away, then plain rounds; the lane
+                // ends with token (l & 1) * 2 + ((l >> 1) & 1)
+                float y2[2];
 #pragma unroll
-            for (int i = 0; i < 2; ++i) {
-                const float keep = l & 1 ? y4[2 + i] : y4[i], give = l & 1 ? y4[i] : y4[2 + i];
-                y2[i] = keep + __shfl_xor_sync(0xffffffffu, give, 1);
+                for (int i = 0; i < 2; ++i) {
+                    const float keep = l & 1 ? y4[2 + i] : y4[i], give = l & 1 ? y4[i] : y4[2 + i];
+                    y2[i] = keep + __shfl_xor_sync(0xffffffffu, give, 1);
+                }
+                const float keep = l & 2 ? y2[1] : y2[0], give = l & 2 ? y2[0] : y2[1];
+                float y = keep + __shfl_xor_sync(0xffffffffu, give, 2);
+#pragma unroll
+                for (int o = 4; o < LANES; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+                if (l < 4) ys[(tq + (l & 1) * 2 + ((l >> 1) & 1)) * CH + cl] = y;
             }
-            const float keep = l & 2 ? y2[1] : y2[0], give = l & 2 ? y2[0] : y2[1];
-            float y = keep + __shfl_xor_sync(0xffffffffu, give, 2);
-#pragma unroll
-            for (int o = 4; o < LANES; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-            if (l < 4) ys[(tq + (l & 1) * 2 + ((l >> 1) & 1)) * CH + cl] = y;
         }
         __syncthreads();
+        if (MODE != FOLD) {
 #pragma unroll
-        for (int i = 0; i < PER_X; ++i) {
-            const int tt = my_t + i * (SCAN_THREADS / CH);
-            if (in_c && tt < count)
-                out[(size_t)(t0 + tt) * ldo + c0 + my_c] = from_float<TX>(fmaf(my_skip, xs[tt * CH + my_c], ys[tt * CH + my_c]) * silu(pz[i]) * scale);
+            for (int i = 0; i < PER_X; ++i) {
+                const int tt = my_t + i * (SCAN_THREADS / CH);
+                if (in_c && tt < count)
+                    out[(size_t)(t0 + tt) * ldo + c0 + my_c] =
+                        from_float<TX>(fmaf(my_skip, xs[tt * CH + my_c], ys[tt * CH + my_c]) * silu(to_float(pz[i])) * sc.scale);
+            }
+            __syncthreads();                        // everyone is done with this tile before it is filled again
         }
-        __syncthreads();                            // everyone is done with this tile before it is filled again
     }
-    if (mine) {
+    float* to = MODE == FOLD ? fold : (MODE == WALK || end == last) ? mine : nullptr;
+    if (to) {
 #pragma unroll
         for (int e = 0; e < NPT; ++e) {
             const int i = l * NPT + e;
-            if (i < N) mine[i] = S[e];
+            if (i < N) to[i] = S[e];
+        }
+    }
+    if (MODE == FOLD && l == 0 && ch < inner) sc.sums[seg_row * inner + ch] = dt_sum;
+}
+
+// One thread an entry of the state: from the seat over the portion's segments, leaving in each one's fold the state before it.
+__global__ void __launch_bounds__(256)
+selective_chain_kernel(SelectiveScan sc) {
+    griddep_wait();
+    griddep_launch_dependents();
+    const int r = blockIdx.x;
+    const size_t per = (size_t)sc.inner * sc.N, e = (size_t)blockIdx.y * 256 + threadIdx.x;
+    const int n = sc.cu_q[r + 1] - sc.cu_q[r];
+    if (e >= per || n <= 0) return;
+    const int segments = (n + SEGMENT - 1) / SEGMENT, seat = sc.seats[r];
+    const size_t row = segment_row(sc.cu_q, r);
+    float S = (seat >= 0 && seat < sc.n_seats) ? sc.state[(size_t)seat * sc.state_stride + e] : 0.f;
+    const float a = sc.minus_a[e];
+    float* p = sc.folds + row * per + e;
+    const float* sum = sc.sums + row * sc.inner + e / sc.N;
+    constexpr int AHEAD = 8;                      // the folds of so many segments are asked for at once: the chain waits on memory
+    for (int s0 = 0; s0 < segments; s0 += AHEAD, p += AHEAD * per, sum += (size_t)AHEAD * sc.inner) {
+        float u[AHEAD], d[AHEAD];
+#pragma unroll
+        for (int x = 0; x < AHEAD; ++x) {
+            const bool in = s0 + x < segments;
+            u[x] = in ? p[x * per] : 0.f;
+            d[x] = in ? sum[(size_t)x * sc.inner] : 0.f;
+        }
+#pragma unroll
+        for (int x = 0; x < AHEAD; ++x) {
+            if (s0 + x >= segments) break;
+            p[x * per] = S;
+            S = fmaf(exp_decay(a * d[x]), S, u[x]);
         }
     }
 }
 
 template <typename TX, int LANES, int NPT, int TT>
-int launch_selective(const void* x, const float* dt, const float* dt_bias, const float* minus_a, const void* bc, long long ldbc,
-                     const float* skip, const void* z, long long ldz, float* state, long long state_stride, const int* seats, const int* cu_q,
-                     void* out, long long ldo, float scale, int requests, int inner, int N, int n_seats, cudaStream_t stream) {
+int launch_selective(const void* x, const void* bc, long long ldbc, const void* z, long long ldz, void* out, long long ldo, SelectiveScan sc,
+                     int requests, int segments, cudaStream_t stream) {
     constexpr int CH = SCAN_THREADS / LANES, NP = LANES * NPT;
     constexpr size_t smem = (size_t)(4 * TT * CH + 2 * TT * NP) * sizeof(float);
     static_assert(smem <= 48 * 1024, "a tile of the selective scan fits the shared memory every block has");
-    constexpr bool EXACT = sizeof(TX) == 4;        // the true 32-bit path
-    fe::launch(selective_scan_kernel<TX, EXACT, LANES, NPT, TT>, dim3((inner + CH - 1) / CH, requests), SCAN_THREADS, smem, stream, (const TX*)x, dt,
-               dt_bias, minus_a, (const TX*)bc, ldbc, skip, (const TX*)z, ldz, state, state_stride, seats, cu_q, (TX*)out, ldo, scale, inner, N,
-               n_seats);
+    const int blocks = (sc.inner + CH - 1) / CH;
+#define FE_SELECTIVE_LAUNCH(MODE, SEGMENTS)                                                                                            \
+    fe::launch(selective_scan_kernel<TX, MODE, LANES, NPT, TT>, dim3(blocks, requests, SEGMENTS), SCAN_THREADS, smem, stream, (const TX*)x, \
+               (const TX*)bc, ldbc, (const TX*)z, ldz, (TX*)out, ldo, sc)
+    if (segments <= 1) {
+        FE_SELECTIVE_LAUNCH(WALK, 1);
+    } else {
+        FE_SELECTIVE_LAUNCH(FOLD, segments);
+        fe::launch(selective_chain_kernel, dim3(requests, (unsigned)(((long long)sc.inner * sc.N + 255) / 256)), 256, 0, stream, sc);
+        FE_SELECTIVE_LAUNCH(OUT, segments);
+    }
+#undef FE_SELECTIVE_LAUNCH
     return fe_check_launch("selective_scan");
 }
 
 template <typename TX>
-int dispatch_selective(const void* x, const float* dt, const float* dt_bias, const float* minus_a, const void* bc, long long ldbc,
-                       const float* skip, const void* z, long long ldz, float* state, long long state_stride, const int* seats, const int* cu_q,
-                       void* out, long long ldo, float scale, int requests, int inner, int N, int n_seats, cudaStream_t stream) {
-#define FE_SELECTIVE(LANES, NPT, TT)                                                                                                      \
-    return launch_selective<TX, LANES, NPT, TT>(x, dt, dt_bias, minus_a, bc, ldbc, skip, z, ldz, state, state_stride, seats, cu_q, out, ldo, \
-                                                scale, requests, inner, N, n_seats, stream)
-    if (N <= 16) FE_SELECTIVE(4, 4, 32);
-    if (N <= 32) FE_SELECTIVE(8, 4, 32);
-    if (N <= 64) FE_SELECTIVE(16, 4, 32);
-    if (N <= 128) FE_SELECTIVE(32, 4, 16);
+int dispatch_selective(const void* x, const void* bc, long long ldbc, const void* z, long long ldz, void* out, long long ldo, SelectiveScan sc,
+                       int requests, int segments, cudaStream_t stream) {
+#define FE_SELECTIVE(LANES, NPT, TT) return launch_selective<TX, LANES, NPT, TT>(x, bc, ldbc, z, ldz, out, ldo, sc, requests, segments, stream)
+    if (sc.N <= 16) FE_SELECTIVE(4, 4, 32);
+    if (sc.N <= 32) FE_SELECTIVE(8, 4, 32);
+    if (sc.N <= 64) FE_SELECTIVE(16, 4, 32);
+    if (sc.N <= 128) FE_SELECTIVE(32, 4, 16);
     FE_SELECTIVE(32, 16, 8);
 #undef FE_SELECTIVE
 }
@@ -493,22 +584,26 @@ extern "C" int fe_gated_group_rmsnorm(const float* y, const float* z, long long 
     return fe_check_launch("gated_group_rmsnorm");
 }
 
-// x [T, inner] in ``dtype``; dt float [T, inner] before its bias and softplus; minus_a float [inner, N]; bc [T, >= 2 N] = B | C in ``dtype``
-// (rows ldbc entries long); z, out [T, >= inner] in ``dtype`` (rows ldz, ldo); state float [n_seats, >= inner N].
-extern "C" int fe_selective_scan(const void* x, const float* dt, const float* dt_bias, const float* minus_a, const void* bc, long long ldbc,
+// How many tokens a segment has; a step's ``folds`` and ``sums`` have tokens / that + requests rows.
+extern "C" int fe_selective_segment_tokens() { return SEGMENT; }
+
+// x [T, inner] in ``dtype``; dt float [T, inner] before its bias and softplus (overwritten where ``segments`` is above 1); minus_a float
+// [inner, N]; bc [T, >= 2 N] = B | C in ``dtype`` (rows ldbc entries long); z, out [T, >= inner] in ``dtype`` (rows ldz, ldo); state float
+// [n_seats, >= inner N].  segments: how many the longest portion has, or 1 to walk every portion as a whole (folds and sums may then
+// be null; else float [rows, inner N] and [rows, inner]).
+extern "C" int fe_selective_scan(const void* x, float* dt, const float* dt_bias, const float* minus_a, const void* bc, long long ldbc,
                                  const float* skip, const void* z, long long ldz, float* state, long long state_stride, const int* seats,
-                                 const int* cu_q, void* out, long long ldo, float scale, int requests, int inner, int N, int n_seats, int dtype,
-                                 cudaStream_t stream) {
+                                 const int* cu_q, void* out, long long ldo, float scale, float* folds, float* sums, int segments, int requests,
+                                 int inner, int N, int n_seats, int dtype, cudaStream_t stream) {
     FE_REQUIRE(requests >= 0 && requests <= 65535 && inner > 0 && N > 0 && N <= 512 && ldbc >= 2LL * N && ldz >= inner && ldo >= inner && n_seats >= 0 &&
-                   (long long)inner * N <= state_stride,
+                   (long long)inner * N <= state_stride && ((long long)inner * N + 255) / 256 <= 65535,
                "selective_scan: bad sizes (%d channels, %d state entries of at most 512)", inner, N);
     FE_REQUIRE(dtype == FE_F32 || dtype == FE_BF16, "selective_scan: unknown dtype %d", dtype);
+    FE_REQUIRE(segments <= 65535 && (segments <= 1 || (folds && sums)), "selective_scan: segments need their scratch");
     if (requests == 0) return 0;
-    if (dtype == FE_F32)
-        return dispatch_selective<float>(x, dt, dt_bias, minus_a, bc, ldbc, skip, z, ldz, state, state_stride, seats, cu_q, out, ldo, scale,
-                                         requests, inner, N, n_seats, stream);
-    return dispatch_selective<bf16>(x, dt, dt_bias, minus_a, bc, ldbc, skip, z, ldz, state, state_stride, seats, cu_q, out, ldo, scale, requests,
-                                    inner, N, n_seats, stream);
+    const SelectiveScan sc{dt, dt_bias, minus_a, skip, state, state_stride, seats, cu_q, folds, sums, scale, inner, N, n_seats};
+    if (dtype == FE_F32) return dispatch_selective<float>(x, bc, ldbc, z, ldz, out, ldo, sc, requests, segments, stream);
+    return dispatch_selective<bf16>(x, bc, ldbc, z, ldz, out, ldo, sc, requests, segments, stream);
 }
 
 // One token a request: low [requests, >= rank + 2 N] = low | B | C (rows ldl), dt_weight [inner, rank] in ``dtype``.

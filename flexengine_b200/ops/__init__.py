@@ -1368,7 +1368,7 @@ def conv_silu(u, conv, bias, state, history_at, state_slots, cu_q, out_float32=F
     return out, gates
 
 
-def memory_gates(rows, bias, cap, state, maxima_at, state_slots, cu_q, heads):
+def memory_gates(rows, bias, cap, state, maxima_at, state_slots, cu_q, heads, max_q_len=0):
     """The gates of a matrix memory: rows float32 [T, i | f] (any row stride), bias float32 [2 heads]; i = cap tanh((i + b) / cap),
     f = log sigmoid(cap tanh((f + b) / cap)), m' = max(f + m, i) from token to token with m in state[seat, maxima_at:] (0 and
     nothing kept for a seat below 0).  float32 [3, T, heads]: f + m - m', exp(i - m'), exp(-m') (csrc/head_scan.cu)."""
@@ -1378,9 +1378,12 @@ def memory_gates(rows, bias, cap, state, maxima_at, state_slots, cu_q, heads):
             or state.stride(-1) != 1 or state.shape[-1] < maxima_at + heads:
         raise ValueError("memory_gates: rows float32 [T, 2 heads] with unit column stride, bias float32 [2 heads], a float32 state row")
     gates = torch.empty((3, T, heads), dtype=torch.float32, device=rows.device)
-    _run(_core(), "fe_memory_gates", _ptr(rows), _c_ll(rows.stride(0)), _ptr(bias), _c_float(cap), _ptr(state), _c_ll(state.stride(0)),
-         _c_ll(maxima_at), _ptr(state_slots), _ptr(cu_q), _ptr(gates), _c_ll(T * heads), _c_int(cu_q.numel() - 1), _c_int(heads),
-         _c_int(state.shape[0]), _stream())
+    lib, requests = _core(), cu_q.numel() - 1
+    blocks = T // lib.fe_head_scan_chunk_tokens() + requests
+    scratch_rows = torch.empty((2 * blocks + requests, heads), dtype=torch.float32, device=rows.device)
+    _run(lib, "fe_memory_gates", _ptr(rows), _c_ll(rows.stride(0)), _ptr(bias), _c_float(cap), _ptr(state), _c_ll(state.stride(0)),
+         _c_ll(maxima_at), _ptr(state_slots), _ptr(cu_q), _ptr(gates), _c_ll(T * heads), _ptr(scratch_rows),
+         _ptr(scratch_rows[2 * blocks:]), _c_int(requests), _c_int(max_q_len or T), _c_int(heads), _c_int(state.shape[0]), _stream())
     return gates
 
 
@@ -1458,19 +1461,31 @@ def _selective_out(what, x, dt_bias, minus_a, skip, z, state, into):
     return out
 
 
-def selective_scan(x, dt, dt_bias, minus_a, bc, skip, z, state, state_slots, cu_q, scale=1.0, into=None):
+SELECTIVE_SEGMENTS_FROM = 256       # portions at least this long may be cut into segments that are walked side by side ...
+SELECTIVE_WARPS_ENOUGH = 16         # ... unless whole portions are this many warps a multiprocessor
+
+
+def selective_scan(x, dt, dt_bias, minus_a, bc, skip, z, state, state_slots, cu_q, scale=1.0, into=None, max_q_len=0):
     """dt <- softplus(dt + dt_bias); S[c, n] <- exp(dt_c minus_a[c, n]) S[c, n] + dt_c x_c B_n; y_c = sum_n S[c, n] C_n + skip_c x_c; y silu(z)
     times ``scale``, per request over the step's tokens (csrc/state_space.cu); S [inner, N] float32 lives in state[seat, : inner N] (zeros
-    and nothing kept for a seat below 0).  x [T, inner], bc [T, B | C] and z in the compute dtype, dt float32 [T, inner]; ``into``: where
-    the rows go (a view with any row stride)."""
+    and nothing kept for a seat below 0).  x [T, inner], bc [T, B | C] and z in the compute dtype, dt float32 [T, inner] (scratch: it may be
+    overwritten); ``into``: where the rows go (a view with any row stride)."""
     _need_cuda(x, dt, dt_bias, minus_a, bc, skip, z, state, state_slots, cu_q, into)
     out = _selective_out("selective_scan", x, dt_bias, minus_a, skip, z, state, into)
     (T, inner), N = x.shape, minus_a.shape[1]
     if dt.dtype != torch.float32 or tuple(dt.shape) != (T, inner) or not dt.is_contiguous() or not _rows_ok(bc, 2 * N, x.dtype):
         raise ValueError("selective_scan: dt is contiguous float32 [T, inner], bc [T, 2 N] in the compute dtype")
-    _run(_core(), "fe_selective_scan", _ptr(x), _ptr(dt), _ptr(dt_bias), _ptr(minus_a), _ptr(bc), _c_ll(bc.stride(0)), _ptr(skip), _ptr(z),
+    lib, requests = _core(), cu_q.numel() - 1
+    longest, segments, folds, sums = max_q_len or T, 1, None, None
+    warps = requests * -(-inner // 128) * (4 if N <= 16 else 8 if N <= 32 else 16 if N <= 64 else 32)
+    if longest >= SELECTIVE_SEGMENTS_FROM and warps < SELECTIVE_WARPS_ENOUGH * sm_count(x.device):
+        per = lib.fe_selective_segment_tokens()
+        segments, rows = -(-longest // per), T // per + requests
+        folds = torch.empty((rows, inner * N), dtype=torch.float32, device=x.device)
+        sums = torch.empty((rows, inner), dtype=torch.float32, device=x.device)
+    _run(lib, "fe_selective_scan", _ptr(x), _ptr(dt), _ptr(dt_bias), _ptr(minus_a), _ptr(bc), _c_ll(bc.stride(0)), _ptr(skip), _ptr(z),
          _c_ll(z.stride(0)), _ptr(state), _c_ll(state.stride(0)), _ptr(state_slots), _ptr(cu_q), _ptr(out), _c_ll(out.stride(0)), _c_float(scale),
-         _c_int(cu_q.numel() - 1), _c_int(inner), _c_int(N), _c_int(state.shape[0]), _c_int(_code(x.dtype)), _stream())
+         _ptr(folds), _ptr(sums), _c_int(segments), _c_int(requests), _c_int(inner), _c_int(N), _c_int(state.shape[0]), _c_int(_code(x.dtype)), _stream())
     return out
 
 
@@ -1543,6 +1558,20 @@ def latent_prepare(q, q_latent, down, norm_weight, eps, positions, inv_freq, rot
 
 
 # ---- a routed feed-forward ---------------------------------------------------------------------------------------
+ROUTER_LOGITS_MAX_EXPERTS = 64       # beyond this the float32 product with its wider tiles
+
+
+def router_logits(h, w):
+    """h [T, H] (any compute dtype) times the router's float32 matrix w [outputs, H]: float32 [T, outputs], in true 32-bit."""
+    _need_cuda(h, w)
+    T, H = h.shape
+    if w.dtype != torch.float32 or w.shape[1] != H or w.shape[0] > ROUTER_LOGITS_MAX_EXPERTS or H % 4 or not (h.is_contiguous() and w.is_contiguous()):
+        return linear(h, w, None, out_float32=True)
+    out = torch.empty((T, w.shape[0]), dtype=torch.float32, device=h.device)
+    _run(_core(), "fe_router_logits", _ptr(h), _ptr(w), _ptr(out), _c_int(T), _c_int(w.shape[0]), _c_int(H), _c_int(_code(h.dtype)), _stream())
+    return out
+
+
 def route_top(logits, top, scale, over_chosen=False, correction=None, groups=(1, 1), sigmoid=False):
     """(int32 [T, top], float32 [T, top]): per token the ``top`` largest softmax scores over all experts (float32, ties
     to the lower index) times ``scale``, and their experts.  ``over_chosen``: the ``top`` largest logits are chosen and the

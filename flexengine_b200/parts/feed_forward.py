@@ -163,7 +163,7 @@ class RoutedExperts(FeedForward):
     def forward(self, ctx, h):
         ops = ctx.ops
         e, f, d = self.experts, self.expert_size, self.hidden_size
-        logits = ops.linear(h, self.router_weight, None, out_float32=True)
+        logits = ops.router_logits(h, self.router_weight)
         shared = None
         if self.shared_size and self.single:
             shared = ops.linear(ops.linear_activated(h, self.shared_up_weight, self.activation), self.shared_down_weight)

@@ -63,7 +63,7 @@ class MatrixMemoryMixer(Mixer):
             return ops.linear(out, self.o_weight)
         qk, inner = H * d, H * dv
         gates = ops.memory_gates(projected[:, 2 * qk + 2 * inner:], self.gates_bias, self.gate_cap, state, H * (d * dv + d), ctx.state_slots,
-                                 ctx.cu_q, H)
+                                 ctx.cu_q, H, max_q_len=ctx.max_q_len)
         o = ops.head_scan(projected[:, :qk], projected[:, qk:2 * qk], projected[:, 2 * qk:2 * qk + inner], gates, state, ctx.state_slots,
                           ctx.cu_q, H, H, d, dv, query_scale=self.query_scale, divided=self.floor, max_q_len=ctx.max_q_len)
         out = ops.head_rmsnorm_gate(o, self.norm_weight, projected[:, 2 * qk + inner:2 * qk + 2 * inner], self.eps, H, ctx.dtype, gate="sigmoid")

@@ -146,7 +146,7 @@ class SelectiveScanMixer(_ConvolvedState):
                                         into=out)
         dt = ops.linear(low[:, :self.dt_rank], self.dt_weight, None, out_float32=True)
         return ops.selective_scan(x, dt, self.dt_bias, self._minus_a, low[:, self.dt_rank:], self.D, z, state, ctx.state_slots, ctx.cu_q,
-                                  scale=scale, into=out)
+                                  scale=scale, into=out, max_q_len=ctx.max_q_len)
 
 
 register_mixer("head_state_space", HeadStateSpaceMixer)

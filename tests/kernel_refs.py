@@ -717,7 +717,7 @@ def conv_silu(u, conv, bias, state, history_at, state_slots, cu_q, out_float32=F
     return y, torch.stack([minus_a.float() * dt, dt])
 
 
-def memory_gates(rows, bias, cap, state, maxima_at, state_slots, cu_q, heads):
+def memory_gates(rows, bias, cap, state, maxima_at, state_slots, cu_q, heads, max_q_len=0):
     """float32 [3, T, heads] from the rows i | f: the logarithms of the decays f + m - m', the weights exp(i - m') and exp(-m'),
     with the running maximum m in state[seat, maxima_at:]."""
     T = rows.shape[0]
@@ -786,7 +786,7 @@ def gated_group_rmsnorm(y, z, weight, eps, groups, out_dtype):
     return (x.reshape(T, inner) * weight.float()).to(out_dtype)
 
 
-def selective_scan(x, dt, dt_bias, minus_a, bc, skip, z, state, state_slots, cu_q, scale=1.0, into=None):
+def selective_scan(x, dt, dt_bias, minus_a, bc, skip, z, state, state_slots, cu_q, scale=1.0, into=None, max_q_len=0):
     """dt <- softplus(dt + dt_bias); S[c, n] <- exp(dt_c minus_a[c, n]) S + dt_c x_c B_n; y = S C + skip x; y silu(z) scale.  ``bc`` [T, B | C]."""
     T, inner = x.shape
     N = minus_a.shape[1]
@@ -858,6 +858,10 @@ def latent_prepare(q, q_latent, down, norm_weight, eps, positions, inv_freq, rot
 
 
 # ---- routed feed-forward ------------------------------------------------------------------------------
+def router_logits(h, w):
+    return linear(h, w, None, out_float32=True)
+
+
 def route_top(logits, top, scale, over_chosen=False, correction=None, groups=(1, 1), sigmoid=False):
     """``sigmoid``: the scores are sigmoid(z), not normalised.  ``correction`` (float32, one number per router output) is added to the scores for the choice only; ``groups`` =
     (count, keep): only outputs of the ``keep`` groups (of ``count`` equal groups of neighbours) with the largest corrected
