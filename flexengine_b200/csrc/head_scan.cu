@@ -9,7 +9,7 @@
 //   head_scan      the scan over the step's portions in blocks of C = 64 tokens.  With L_n = l_1 + .. + l_n inside a block,
 //                    o_n = exp(L_n) S_0^T q_n + sum_(b <= n) exp(L_n - L_b) w_b (q_n . k_b) v_b
 //                    S_C = exp(L_C) S_0 + sum_b exp(L_C - L_b) w_b k_b v_b^T
-//                  so three launches do a step: every block's own sum of k v^T (independent of the others), the chain S_0 -> S_C -> ...
+//                  so three launches (four where heads share queries and keys) do a step: every block's own sum of k v^T (independent of the others), the chain S_0 -> S_C -> ...
 //                  over a portion's blocks (elementwise), and every block's outputs from the state before it (independent again)
 //   head_step      a step of one token a request; with MEMORY everything of a matrix memory between its two products: gates,
 //                  running maximum, recurrence, divisor, head norm and output gate
@@ -251,17 +251,59 @@ head_scan_chain_kernel(const float* __restrict__ totals, float* state, long long
     if (mine) *mine = S;
 }
 
+// The products of a block's queries and keys where several heads read one group of them: qk[row][group] [b][n] = query_scale q_n . k_b.
+// Grid (block of tokens, request, group), 256 threads as 16 x 16.
+__global__ void __launch_bounds__(256)
+head_scan_products_kernel(const float* __restrict__ q, long long ldq, float query_scale, const float* __restrict__ k, long long ldk,
+                          const int* __restrict__ cu_q, float* __restrict__ qk, int groups, int d, int nd) {
+    griddep_wait();
+    griddep_launch_dependents();
+    __shared__ __align__(16) float qT[TILE * PITCH];
+    __shared__ __align__(16) float kT[TILE * PITCH];
+    const int c = blockIdx.x, r = blockIdx.y, group = blockIdx.z;
+    const int begin = cu_q[r] + c * CHUNK, end = cu_q[r + 1];
+    if (begin >= end) return;
+    const int len = min(CHUNK, end - begin);
+    const int tid = threadIdx.x, ty = tid >> 4, tx = tid & 15;
+    float W[4][4] = {};
+    for (int dt = 0; dt < nd; ++dt) {
+        __syncthreads();
+        for (int e = tid; e < CHUNK * TILE; e += 256) {
+            const int n = e / TILE, i = e - n * TILE, gi = dt * TILE + i;
+            const bool in = n < len && gi < d;
+            qT[i * PITCH + n] = in ? query_scale * q[(size_t)(begin + n) * ldq + (size_t)group * d + gi] : 0.f;
+            kT[i * PITCH + n] = in ? k[(size_t)(begin + n) * ldk + (size_t)group * d + gi] : 0.f;
+        }
+        __syncthreads();
+#pragma unroll 4
+        for (int i = 0; i < TILE; ++i) {
+            const float4 q4 = *reinterpret_cast<const float4*>(qT + i * PITCH + ty * 4);
+            const float4 k4 = *reinterpret_cast<const float4*>(kT + i * PITCH + tx * 4);
+            const float qq[4] = {q4.x, q4.y, q4.z, q4.w}, kk[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+            for (int x = 0; x < 4; ++x)
+#pragma unroll
+                for (int y = 0; y < 4; ++y) W[x][y] = fmaf(qq[x], kk[y], W[x][y]);
+        }
+    }
+    float* to = qk + ((chunk_row(cu_q, r) + c) * groups + group) * (size_t)(CHUNK * CHUNK);
+#pragma unroll
+    for (int y = 0; y < 4; ++y) *reinterpret_cast<float4*>(to + (tx * 4 + y) * CHUNK + ty * 4) = make_float4(W[0][y], W[1][y], W[2][y], W[3][y]);
+}
+
 // A block's outputs for a tile of value channels: W = (Q K^T) with entry (n, b) times exp(L_n - L_b) w_b where b <= n, else 0, and
 // ``skip`` added on the diagonal; out = diag(exp(L_n)) Q S_0 + W V.  Q, K and S_0 pass through shared memory in tiles of key
 // channels; W takes the keys' place.  Grid (block of tokens, request, head x tile of value channels), 256 threads as 16 x 16, a
-// thread 4 tokens x 4 columns.
+// thread 4 tokens x 4 columns.  SHARED: Q K^T comes from head_scan_products (``qk``) instead.
 constexpr size_t CHUNK_OUT_SMEM = ((size_t)2 * TILE * PITCH + (size_t)TILE * TILE + (size_t)CHUNK * TILE + 5 * CHUNK + 4) * sizeof(float) +
                                   CHUNK * sizeof(double);
 
+template <bool SHARED>
 __global__ void __launch_bounds__(256)
 head_scan_out_kernel(const float* __restrict__ q, long long ldq, float query_scale, const float* __restrict__ k, long long ldk,
                      const float* __restrict__ v, long long ldv, const float* __restrict__ gates, long long plane,
-                     const float* __restrict__ skip, const int* __restrict__ cu_q, const float* __restrict__ sums, long long per,
+                     const float* __restrict__ skip, const float* __restrict__ qk, const int* __restrict__ cu_q,
+                     const float* __restrict__ sums, long long per,
                      float* __restrict__ out, int heads, int groups, int d, int dv, int nd, int nv, int divided, float floor) {
     griddep_wait();
     griddep_launch_dependents();
@@ -298,7 +340,7 @@ head_scan_out_kernel(const float* __restrict__ q, long long ldq, float query_sca
             const int n = e / TILE, i = e - n * TILE, gi = dt * TILE + i;
             const bool in = n < len && gi < d;
             qT[i * PITCH + n] = in ? query_scale * q[(size_t)(begin + n) * ldq + (size_t)group * d + gi] : 0.f;
-            kT[i * PITCH + n] = in ? k[(size_t)(begin + n) * ldk + (size_t)group * d + gi] : 0.f;
+            if (!SHARED) kT[i * PITCH + n] = in ? k[(size_t)(begin + n) * ldk + (size_t)group * d + gi] : 0.f;
             const int gj = vt * TILE + i;                                       // here n walks key channels, i value channels
             sS[e] = (dt * TILE + n < d && gj < dv) ? before[(size_t)(dt * TILE + n) * dv + gj] : 0.f;
         }
@@ -307,14 +349,14 @@ head_scan_out_kernel(const float* __restrict__ q, long long ldq, float query_sca
 #pragma unroll 4
         for (int i = 0; i < TILE; ++i) {
             const float4 q4 = *reinterpret_cast<const float4*>(qT + i * PITCH + ty * 4);
-            const float4 k4 = *reinterpret_cast<const float4*>(kT + i * PITCH + tx * 4);
+            const float4 k4 = SHARED ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(kT + i * PITCH + tx * 4);
             const float4 s4 = *reinterpret_cast<const float4*>(sS + i * TILE + tx * 4);
             const float qq[4] = {q4.x, q4.y, q4.z, q4.w}, kk[4] = {k4.x, k4.y, k4.z, k4.w}, ss[4] = {s4.x, s4.y, s4.z, s4.w};
 #pragma unroll
             for (int x = 0; x < 4; ++x)
 #pragma unroll
                 for (int y = 0; y < 4; ++y) {
-                    W[x][y] = fmaf(qq[x], kk[y], W[x][y]);
+                    if (!SHARED) W[x][y] = fmaf(qq[x], kk[y], W[x][y]);
                     O[x][y] = fmaf(qq[x], ss[y], O[x][y]);
                 }
         }
@@ -322,6 +364,14 @@ head_scan_out_kernel(const float* __restrict__ q, long long ldq, float query_sca
             for (int i = part; i < TILE; i += 4) nq = fmaf(qT[i * PITCH + mine], nS[i], nq);
     }
     __syncthreads();
+    if (SHARED) {
+        const float* from = qk + ((chunk_row(cu_q, r) + c) * groups + group) * (size_t)(CHUNK * CHUNK);
+#pragma unroll
+        for (int y = 0; y < 4; ++y) {
+            const float4 w4 = *reinterpret_cast<const float4*>(from + (tx * 4 + y) * CHUNK + ty * 4);
+            W[0][y] = w4.x, W[1][y] = w4.y, W[2][y] = w4.z, W[3][y] = w4.w;
+        }
+    }
     const float skip_of = skip ? skip[head] : 0.f;
 #pragma unroll
     for (int y = 0; y < 4; ++y) {
@@ -535,10 +585,10 @@ extern "C" int fe_head_scan_chunk_tokens() { return CHUNK; }
 // q, k float [T, >= groups d], v float [T, >= heads dv] (rows ldq, ldk, ldv entries long); gates float [2 or 3][plane] ([T, heads] each:
 // logarithms of the decays, weights, with ``divided`` the numbers e_t); skip float [heads] or null (not with ``divided``); state
 // float [n_seats, >= per] with per = heads d dv (+ heads d with ``divided``); sums float [tokens / 64 + requests, per] and totals
-// [the same, heads] are scratch; out float [T, heads dv]; most_tokens: the longest portion of the step or more.
+// [the same, heads] are scratch, and where several heads read a group (heads > groups) products [the same, groups, 64, 64]; out float [T, heads dv]; most_tokens: the longest portion of the step or more.
 extern "C" int fe_head_scan(const float* q, long long ldq, float query_scale, const float* k, long long ldk, const float* v, long long ldv,
                             const float* gates, long long plane, const float* skip, float* state, long long state_stride, const int* seats,
-                            const int* cu_q, float* out, float* sums, float* totals, int requests, int most_tokens, int heads, int groups, int d,
+                            const int* cu_q, float* out, float* sums, float* totals, float* products, int requests, int most_tokens, int heads, int groups, int d,
                             int dv, int n_seats, int divided, float floor, cudaStream_t stream) {
     const int nd = (d + TILE - 1) / TILE, nv = (dv + TILE - 1) / TILE;
     const long long per = (long long)heads * d * dv + (divided ? (long long)heads * d : 0);
@@ -550,7 +600,8 @@ extern "C" int fe_head_scan(const float* q, long long ldq, float query_scale, co
     if (requests == 0 || most_tokens == 0) return 0;
     static bool opted = false;
     if (!opted) {
-        const cudaError_t err = cudaFuncSetAttribute(head_scan_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)CHUNK_OUT_SMEM);
+        cudaError_t err = cudaFuncSetAttribute(head_scan_out_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)CHUNK_OUT_SMEM);
+        if (err == cudaSuccess) err = cudaFuncSetAttribute(head_scan_out_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)CHUNK_OUT_SMEM);
         FE_REQUIRE(err == cudaSuccess, "head_scan: %s", cudaGetErrorString(err));
         opted = true;
     }
@@ -559,8 +610,13 @@ extern "C" int fe_head_scan(const float* q, long long ldq, float query_scale, co
                totals, per, heads, groups, d, dv, nd, nv, divided);
     fe::launch(head_scan_chain_kernel, dim3(requests, (unsigned)((per + 255) / 256)), 256, 0, stream, (const float*)totals, state, state_stride,
                seats, cu_q, sums, per, heads, d, dv, n_seats);
-    fe::launch(head_scan_out_kernel, dim3(most_blocks, requests, heads * nv), 256, CHUNK_OUT_SMEM, stream, q, ldq, query_scale, k, ldk, v, ldv,
-               gates, plane, skip, cu_q, (const float*)sums, per, out, heads, groups, d, dv, nd, nv, divided, floor);
+    const bool shared = heads > groups && products != nullptr;
+    if (shared)
+        fe::launch(head_scan_products_kernel, dim3(most_blocks, requests, groups), 256, 0, stream, q, ldq, query_scale, k, ldk, cu_q, products,
+                   groups, d, nd);
+    fe::launch(shared ? head_scan_out_kernel<true> : head_scan_out_kernel<false>, dim3(most_blocks, requests, heads * nv), 256, CHUNK_OUT_SMEM,
+               stream, q, ldq, query_scale, k, ldk, v, ldv, gates, plane, skip, (const float*)products, cu_q, (const float*)sums, per, out, heads,
+               groups, d, dv, nd, nv, divided, floor);
     return fe_check_launch("head_scan");
 }
 

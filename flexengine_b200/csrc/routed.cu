@@ -759,6 +759,56 @@ __global__ void routed_combine_kernel(const float* __restrict__ y, const int* __
         out[(size_t)t * D + j] = from_float<T>(total);
     }
 }
+
+// The same four columns a thread (D a multiple of four, rows on 16-byte boundaries): the sums are the same, term by term.
+template <typename T>
+__global__ void __launch_bounds__(256)
+routed_combine_four_kernel(const float* __restrict__ y, const int* __restrict__ row_of_pair, const float* __restrict__ weights,
+                           const T* __restrict__ shared, T* __restrict__ out, int top, int D, const T* __restrict__ h) {
+    griddep_wait();
+    griddep_launch_dependents();
+    const int t = blockIdx.x;
+    for (int j = (blockIdx.y * 256 + threadIdx.x) * 4; j < D; j += gridDim.y * 1024) {
+        float4 total = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int c = 0; c < top; ++c) {
+            const int row = row_of_pair[(size_t)t * top + c];
+            const float w = weights ? weights[(size_t)t * top + c] : 1.f;
+            float4 v;
+            if (row >= 0) v = load_four<float>(y + (size_t)row * D + j);
+            else if (row == -2 && h && weights) v = load_four<T>(h + (size_t)t * D + j);
+            else continue;
+            total.x = fmaf(w, v.x, total.x), total.y = fmaf(w, v.y, total.y), total.z = fmaf(w, v.z, total.z), total.w = fmaf(w, v.w, total.w);
+        }
+        if (shared) {
+            const float4 v = load_four<T>(shared + (size_t)t * D + j);
+            total.x += v.x, total.y += v.y, total.z += v.z, total.w += v.w;
+        }
+        T* to = out + (size_t)t * D + j;
+        if (sizeof(T) == 4) {
+            *reinterpret_cast<float4*>(to) = total;
+        } else {
+            const __nv_bfloat162 a = __floats2bfloat162_rn(total.x, total.y), b = __floats2bfloat162_rn(total.z, total.w);
+            uint2 raw;
+            raw.x = *reinterpret_cast<const unsigned*>(&a), raw.y = *reinterpret_cast<const unsigned*>(&b);
+            *reinterpret_cast<uint2*>(to) = raw;
+        }
+    }
+}
+
+template <typename T>
+void launch_combine(const float* y, const int* row_of_pair, const float* weights, const T* shared, T* out, int tokens, int top, int D, const T* h,
+                    cudaStream_t stream) {
+    if (D % 4 == 0 && (((size_t)y | (size_t)shared | (size_t)out | (size_t)h) & 15) == 0) {
+        const int stretches = (D + 1023) / 1024;
+        fe::launch(routed_combine_four_kernel<T>, dim3(tokens, stretches < 65535 ? stretches : 65535), 256, 0, stream, y,
+                   row_of_pair, weights, shared, out, top, D, h);
+        return;
+    }
+    const int threads = D >= 1024 ? 256 : 128;
+    const int stretches = tokens >= 512 ? 1 : (D + threads - 1) / threads;          // few tokens: one column a thread
+    fe::launch(routed_combine_kernel<T>, dim3(tokens, stretches < 65535 ? stretches : 65535), threads, 0, stream, y, row_of_pair, weights, shared,
+               out, top, D, h);
+}
 }  // namespace
 
 extern "C" long long fe_routed_experts_workspace(int T, int top, int experts, int D, int F, int dtype) {
@@ -800,7 +850,6 @@ extern "C" int fe_routed_experts(const void* h, const int* chosen, const float* 
     char* act = (char*)workspace + (ints * 4 + 255) / 256 * 256;
     const long long width = dtype == FE_F32 ? 4 : 2;
     float* y = (float*)(act + (pairs * F * width + 255) / 256 * 256);
-    const int threads = D >= 1024 ? 256 : 128;
     const long long width_bytes = dtype == FE_F32 ? 4 : 2;
     const int few_rows = pairs <= (long long)FEW_ROWS_SMALL * experts ? FEW_ROWS_SMALL : FEW_ROWS;
     const size_t few_smem1 = (size_t)few_rows * D * width_bytes, few_smem2 = (size_t)few_rows * F * width_bytes;
@@ -809,7 +858,7 @@ extern "C" int fe_routed_experts(const void* h, const int* chosen, const float* 
     const bool piped = !few && dtype == FE_BF16 && D % 8 == 0 && F % 8 == 0;
     FE_REQUIRE(identity >= 0 && single >= 0 && single <= 2 && (single == 0 || limit == 0.f), "routed_experts: bad options");
     const float act_of = single == 0 ? limit : (single == 2 ? SINGLE_GELU : SINGLE_RELU2);
-    fe::launch(route_plan_kernel, 1, 256, 0, stream, chosen, (int)pairs, experts, identity, few ? few_rows : (piped ? PBM : BM), offsets,
+    fe::launch(route_plan_kernel, 1, pairs > 512 ? 1024 : 256, 0, stream, chosen, (int)pairs, experts, identity, few ? few_rows : (piped ? PBM : BM), offsets,
                row_of_pair, pair_of_row, tiles, tile_expert, tile_row0, status);
     const int* c_pairs = pair_of_row;
     const int* c_none = nullptr;
@@ -868,14 +917,8 @@ extern "C" int fe_routed_experts(const void* h, const int* chosen, const float* 
         }
     }
 #undef FE_ROUTED_PRODUCTS
-    const int stretches = T >= 512 ? 1 : (D + threads - 1) / threads;          // few tokens: one column a thread
-    const dim3 combine(T, stretches < 65535 ? stretches : 65535);
-    if (dtype == FE_F32)
-        fe::launch(routed_combine_kernel<float>, combine, threads, 0, stream, (const float*)y, (const int*)row_of_pair, out_weights,
-                   (const float*)shared, (float*)out, top, D, identity ? (const float*)h : (const float*)nullptr);
-    else
-        fe::launch(routed_combine_kernel<bf16>, combine, threads, 0, stream, (const float*)y, (const int*)row_of_pair, out_weights,
-                   (const bf16*)shared, (bf16*)out, top, D, identity ? (const bf16*)h : (const bf16*)nullptr);
+    if (dtype == FE_F32) launch_combine<float>(y, row_of_pair, out_weights, (const float*)shared, (float*)out, T, top, D, identity ? (const float*)h : nullptr, stream);
+    else launch_combine<bf16>(y, row_of_pair, out_weights, (const bf16*)shared, (bf16*)out, T, top, D, identity ? (const bf16*)h : nullptr, stream);
     return fe_check_launch("routed_experts");
 }
 
@@ -885,7 +928,7 @@ extern "C" int fe_routed_experts(const void* h, const int* chosen, const float* 
 extern "C" int fe_routed_plan(const int* chosen, int pairs, int experts, int tile_rows, int* offsets, int* row_of_pair,
                               int* pair_of_row, int* tiles, int* tile_expert, int* tile_row0, int* status, int identity, cudaStream_t stream) {
     FE_REQUIRE(pairs >= 1 && experts >= 1 && experts <= ROUTE_MAX_EXPERTS && tile_rows >= 1 && identity >= 0, "routed_plan: bad sizes");
-    fe::launch(route_plan_kernel, 1, 256, 0, stream, chosen, pairs, experts, identity, tile_rows, offsets, row_of_pair, pair_of_row, tiles,
+    fe::launch(route_plan_kernel, 1, pairs > 512 ? 1024 : 256, 0, stream, chosen, pairs, experts, identity, tile_rows, offsets, row_of_pair, pair_of_row, tiles,
                tile_expert, tile_row0, status);
     return fe_check_launch("routed_plan");
 }
@@ -916,15 +959,8 @@ extern "C" int fe_routed_gather(const void* h, const int* pair_of_row, int top, 
 extern "C" int fe_routed_combine(const float* y, const int* row_of_pair, const float* weights, const void* shared, void* out, int T,
                                  int top, int D, int dtype, const void* identity_rows, cudaStream_t stream) {
     FE_REQUIRE(T >= 1 && top >= 1 && D >= 1, "routed_combine: bad sizes");
-    const int threads = D >= 1024 ? 256 : 128;
-    const int stretches = T >= 512 ? 1 : (D + threads - 1) / threads;
-    const dim3 grid(T, stretches < 65535 ? stretches : 65535);
-    if (dtype == FE_F32)
-        fe::launch(routed_combine_kernel<float>, grid, threads, 0, stream, y, row_of_pair, weights, (const float*)shared, (float*)out, top, D,
-                   (const float*)identity_rows);
-    else if (dtype == FE_BF16)
-        fe::launch(routed_combine_kernel<bf16>, grid, threads, 0, stream, y, row_of_pair, weights, (const bf16*)shared, (bf16*)out, top, D,
-                   (const bf16*)identity_rows);
+    if (dtype == FE_F32) launch_combine<float>(y, row_of_pair, weights, (const float*)shared, (float*)out, T, top, D, (const float*)identity_rows, stream);
+    else if (dtype == FE_BF16) launch_combine<bf16>(y, row_of_pair, weights, (const bf16*)shared, (bf16*)out, T, top, D, (const bf16*)identity_rows, stream);
     else
         FE_REQUIRE(false, "routed_combine: unknown dtype %d", dtype);
     return fe_check_launch("routed_combine");

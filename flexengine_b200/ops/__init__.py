@@ -1411,9 +1411,11 @@ def head_scan(q, k, v, gates, state, state_slots, cu_q, heads, groups, dim, vdim
     rows = T // lib.fe_head_scan_chunk_tokens() + requests
     sums = torch.empty((rows, per), dtype=torch.float32, device=v.device)
     totals = torch.empty((rows, heads), dtype=torch.float32, device=v.device)
+    block = lib.fe_head_scan_chunk_tokens()
+    products = torch.empty((rows, groups, block, block), dtype=torch.float32, device=v.device) if heads > groups else None
     _run(lib, "fe_head_scan", _ptr(q), _c_ll(q.stride(0)), _c_float(query_scale), _ptr(k), _c_ll(k.stride(0)), _ptr(v), _c_ll(v.stride(0)),
          _ptr(gates), _c_ll(T * heads), _ptr(skip), _ptr(state), _c_ll(state.stride(0)), _ptr(state_slots), _ptr(cu_q), _ptr(out), _ptr(sums),
-         _ptr(totals), _c_int(requests), _c_int(max_q_len or T), _c_int(heads), _c_int(groups), _c_int(dim), _c_int(vdim),
+         _ptr(totals), _ptr(products), _c_int(requests), _c_int(max_q_len or T), _c_int(heads), _c_int(groups), _c_int(dim), _c_int(vdim),
          _c_int(state.shape[0]), _c_int(0 if divided is None else 1), _c_float(divided or 0.0), _stream())
     return out
 
