@@ -17,6 +17,8 @@ namespace {
 constexpr float LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ float silu(float z) { return z / (1.f + expf(-z)); }
+// The same with the hardware's division (two units in the last place; a z so far down that the divisor overflows gives 0, as it should).
+__device__ __forceinline__ float silu_near(float z) { return __fdividef(z, 1.f + expf(-z)); }
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 template <typename T, int V> __device__ __forceinline__ void load_v(const T* p, float* out);
@@ -111,7 +113,7 @@ conv_silu_kernel(const TI* __restrict__ u, long long ld, const float* __restrict
                 acc[c] = b[c];
 #pragma unroll
                 for (int j = 0; j < K; ++j) acc[c] = fmaf(w[j][c], x[y + j][c], acc[c]);
-                acc[c] = silu(acc[c]);
+                acc[c] = silu_near(acc[c]);
             }
             store_v<TO, V>(to + (size_t)y * C, acc);
         }
@@ -130,7 +132,7 @@ conv_silu_kernel(const TI* __restrict__ u, long long ld, const float* __restrict
                 for (int c = 0; c < V; ++c) acc[c] = fmaf(w[c], x[c], acc[c]);
             }
 #pragma unroll
-            for (int c = 0; c < V; ++c) acc[c] = silu(acc[c]);
+            for (int c = 0; c < V; ++c) acc[c] = silu_near(acc[c]);
             store_v<TO, V>(to + (size_t)y * C, acc);
         }
     }

@@ -910,6 +910,21 @@ def test_kept_first_tokens_in_every_attention_kernel(dtype, shape, lengths):
 
 
 @pytest.mark.gpu
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("T,width,experts", [(1, 64, 5), (8, 2048, 8), (301, 132, 16), (37, 4, 1), (50, 1028, 64), (9, 66, 7), (20, 128, 65)])
+def test_router_logits_kernel_against_the_reference(T, width, experts, dtype):
+    """Also what goes to the float32 product instead: widths that do not come in fours, more than 64 experts.  A token's logits do
+    not depend on what else is in the batch."""
+    from flexengine_b200 import ops
+    h = randn(T, width, seed=12).to(device="cuda:0", dtype=getattr(torch, dtype))
+    w = randn(experts, width, seed=13, scale=width ** -0.5).cuda()
+    got = ops.router_logits(h, w)
+    near(got, (h.double() @ w.double().T).float(), 1e-5, "logits")
+    for row in (0, T // 2, T - 1):
+        assert torch.equal(ops.router_logits(h[row:row + 1].contiguous(), w), got[row:row + 1])
+
+
+@pytest.mark.gpu
 @pytest.mark.parametrize("T,D,F,experts,top", [(700, 1024, 1024, 4, 2), (1500, 1024, 1536, 3, 1), (300, 256, 128, 6, 3), (6, 128, 64, 8, 2), (3, 72, 36, 5, 2), (200, 68, 36, 5, 2)])
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("activation", ["silu", "clamped", "relu2", "gelu"])
