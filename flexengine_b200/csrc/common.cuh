@@ -96,10 +96,10 @@ template <> __device__ __forceinline__ void store8<bf16>(bf16* p, const float* v
 // The exact form of GELU: z/2 (1 + erf(z / sqrt(2))).
 __device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
 
-// e^x for x <= 0 to about half an ulp: x = k ln 2 + r with k whole and |r| <= ln 2 / 2 (ln 2 in two parts, Cody and Waite's
+// e^x for x <= 0 to about an ulp at worst, and without a bias next to 1: x = k ln 2 + r with k whole and |r| <= ln 2 / 2 (ln 2 in two parts, Cody and Waite's
 // reduction), the Taylor polynomial of e^r - 1 to the seventh power (the next term is below 6e-9), and k added to the exponent.  A
 // recurrence multiplies the same decay into its state token after token: errors of a rounding or two that always fall to the same
-// side, as the hardware's 2^x has them next to 1, add up over a long sequence; half an ulp either way does not.
+// side, as the hardware's 2^x has them next to 1, add up over a long sequence; errors to either side hardly do.
 __device__ __forceinline__ float exp_decay(float x) {
     x = fmaxf(x, -87.f);
     const float magic = 12582912.f;                       // 1.5 2^23: adding it rounds to a whole number

@@ -188,7 +188,7 @@ __global__ void gated_group_rmsnorm_kernel(const float* __restrict__ y, const fl
 
 // ---------------------------------------------------------------------------------------------
 // The selective scan.  LANES neighbouring lanes share a channel, each with NPT neighbouring entries of its state in registers
-// (entries beyond N have B = C = 0 and stay zero); the true 32-bit path takes the decays to half an ulp (exp_decay), the other one
+// (entries beyond N have B = C = 0 and stay zero); the true 32-bit path takes the decays from exp_decay, the other one
 // with the hardware's 2^x; a block has 128 / LANES channels of one request and walks its tokens in tiles of TT staged in shared
 // memory; the rows of the next tile are on their way (in registers, as they lie in memory) while one is walked.  Four tokens at a
 // time share the rounds of the sum over the lanes.
